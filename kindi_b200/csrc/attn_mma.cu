@@ -19,29 +19,11 @@
 // the general kernel.
 #include <stdio.h>
 #include "sm100.cuh"
+#include "mma_sync.cuh"
 
 #define AT_THREADS 160          // warps 0-3: MMA + softmax, warp 4: TMA producer
 #define AT_ROWS 64              // rows per CTA in the prefill form
 
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-    asm volatile(
-        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
-        "{%0, %1, %2, %3};"
-        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *(uint32_t*)&v;
-}
 // byte offset of (row, 16-byte chunk) in a [64 rows][HD] tile stored as HD/64 swizzled boxes of [64][128 bytes]
 __device__ __forceinline__ uint32_t tile_off(int row, int chunk) {
     return (uint32_t)((chunk >> 3) * 8192 + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
@@ -101,7 +83,7 @@ __global__ void __launch_bounds__(AT_THREADS, 2) k_attn_mma(const __grid_constan
         float* __restrict__ part_ml, const int* __restrict__ slot, const int* __restrict__ q_start,
         const int* __restrict__ kv_len, int nh, int nkv, int G, float scale_log2e, int window,
         const int* __restrict__ table, int table_stride, int n_pages, int* status, AtRopeIn rp, int keep_first,
-        const float* __restrict__ sink) {
+        const float* __restrict__ sink, int chunk, const __grid_constant__ KbCap cap) {
     static_assert(!ROPE || DEC, "rotation inside the kernel: decode form only");
     constexpr int AT_STAGES = DEC ? 3 : 2;      // pages in flight (two CTAs fit an SM in both forms)
     constexpr int KT = HD / 16;                 // k-steps of Q K^T
@@ -132,7 +114,7 @@ __global__ void __launch_bounds__(AT_THREADS, 2) k_attn_mma(const __grid_constan
     int row0, pg_first, n_keep, it_lo, n_iter;
     if (DEC) {
         row0 = 0;
-        const int lo = (window > 0 && kvl - window > 0) ? kvl - window : 0;       // row position is kvl - 1
+        const int lo = kb_span_lo(kvl - 1, window, chunk);       // row position is kvl - 1
         const int last = (kvl - 1) / KB_PAGE;
         pg_first = lo / KB_PAGE;
         n_keep = min((keep_first + KB_PAGE - 1) / KB_PAGE, pg_first);
@@ -146,7 +128,7 @@ __global__ void __launch_bounds__(AT_THREADS, 2) k_attn_mma(const __grid_constan
         row0 = (n_tiles - 1 - (int)blockIdx.x) * AT_ROWS;          // the longest tiles first
         const int last_row = min(n_rows, row0 + AT_ROWS) - 1;
         const int p_first = pos0 + row0 / G, p_last = pos0 + last_row / G;
-        const int lo = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+        const int lo = kb_span_lo(p_first, window, chunk);
         pg_first = lo / KB_PAGE;
         n_keep = min((keep_first + KB_PAGE - 1) / KB_PAGE, pg_first);
         it_lo = 0;
@@ -312,8 +294,7 @@ __global__ void __launch_bounds__(AT_THREADS, 2) k_attn_mma(const __grid_constan
         }
         const int ra = wrow0 + (lane >> 2), rb = ra + 8;
         const int pa = ra < n_rows ? pos0 + ra / G : -1, pb = rb < n_rows ? pos0 + rb / G : -1;
-        const int la = (window > 0 && pa - window + 1 > 0) ? pa - window + 1 : 0;
-        const int lb = (window > 0 && pb - window + 1 > 0) ? pb - window + 1 : 0;
+        const int la = kb_span_lo(max(pa, 0), window, chunk), lb = kb_span_lo(max(pb, 0), window, chunk);
         // the last position any row of this warp reads: later pages are skipped by the whole warp
         int wlast = max(pa, pb);
         wlast = max(wlast, __shfl_xor_sync(0xffffffffu, wlast, 4));
@@ -360,15 +341,22 @@ __global__ void __launch_bounds__(AT_THREADS, 2) k_attn_mma(const __grid_constan
                         mma_bf16(sc[2 * n2 + 1], qf[ks], r2, r3);
                     }
                 }
-                // scale, mask, running maximum
+                // scale (or cap), mask, running maximum
+                if (!ROPE && cap.mode) {
+#pragma unroll
+                    for (int n = 0; n < NT; n++)
+#pragma unroll
+                        for (int c = 0; c < 4; c++) sc[n][c] = kb_cap2(sc[n][c], cap);
+                }
+                const float mul = !ROPE && cap.mode ? 1.0f : scale_log2e;
                 float mxa = -INFINITY, mxb = -INFINITY;
 #pragma unroll
                 for (int n = 0; n < NT; n++) {
                     const int p = key0 + n * 8 + (lane & 3) * 2;
-                    sc[n][0] = (p <= pa && (p >= la || p < keep_first)) ? sc[n][0] * scale_log2e : -INFINITY;
-                    sc[n][1] = (p + 1 <= pa && (p + 1 >= la || p + 1 < keep_first)) ? sc[n][1] * scale_log2e : -INFINITY;
-                    sc[n][2] = (p <= pb && (p >= lb || p < keep_first)) ? sc[n][2] * scale_log2e : -INFINITY;
-                    sc[n][3] = (p + 1 <= pb && (p + 1 >= lb || p + 1 < keep_first)) ? sc[n][3] * scale_log2e : -INFINITY;
+                    sc[n][0] = (p <= pa && (p >= la || p < keep_first)) ? sc[n][0] * mul : -INFINITY;
+                    sc[n][1] = (p + 1 <= pa && (p + 1 >= la || p + 1 < keep_first)) ? sc[n][1] * mul : -INFINITY;
+                    sc[n][2] = (p <= pb && (p >= lb || p < keep_first)) ? sc[n][2] * mul : -INFINITY;
+                    sc[n][3] = (p + 1 <= pb && (p + 1 >= lb || p + 1 < keep_first)) ? sc[n][3] * mul : -INFINITY;
                     mxa = fmaxf(mxa, fmaxf(sc[n][0], sc[n][1]));
                     mxb = fmaxf(mxb, fmaxf(sc[n][2], sc[n][3]));
                 }
@@ -565,7 +553,7 @@ static int launch_attn(const CUtensorMap& map, const void* q, int ldq, void* out
                        float* part_ml, const int* slot, const int* q_start, const int* kv_len, int B, int nh, int nkv,
                        float scale, int window, const int* table, int table_stride, int n_pages, int grid_x,
                        int* status, cudaStream_t st, AtRopeIn rp = AtRopeIn(), int keep_first = 0,
-                       const float* sink = nullptr) {
+                       const float* sink = nullptr, int chunk = 0, const KbCap& cap = KbCap()) {
     auto kern = k_attn_mma<HD, DEC, ROPE>;
     int sm = attn_smem_bytes<HD, DEC>();
     constexpr int ALONE = 118 * 1024;   // more than half of an SM's shared memory: a CTA that asks for it has the SM to itself
@@ -581,7 +569,7 @@ static int launch_attn(const CUtensorMap& map, const void* q, int ldq, void* out
     dim3 grid(grid_x, nkv, B);
     kb_launch(kern, grid, AT_THREADS, sm, st, map, (const bf16*)q, ldq, (bf16*)out, ldo, part_o, part_ml, slot, q_start,
                                        kv_len, nh, nkv, nh / nkv, scale * 1.4426950408889634f, window, table,
-                                       table_stride, n_pages, status, rp, keep_first, sink);
+                                       table_stride, n_pages, status, rp, keep_first, sink, chunk, cap);
     return (int)cudaGetLastError();
 }
 
@@ -591,9 +579,10 @@ static int launch_attn(const CUtensorMap& map, const void* q, int ldq, void* out
 extern "C" int kb_attn_mma(const void* q, int ldq, void* out, int ldo, float* part_o, float* part_ml,
                            const int* slot, const int* q_start, const int* kv_len, int B, int nh, int nkv, int hd,
                            float scale, int window, void* pool, const int* table, int table_stride, int n_pages,
-                           int decode, int grid_x, int* status, cudaStream_t st, int keep_first, const float* sink) {
+                           int decode, int grid_x, int* status, cudaStream_t st, int keep_first, const float* sink,
+                           int chunk, const float* cap) {
     // sink (float [nh] or null): exp(sink[h]) joins head h's softmax denominator, once (with position splits: in the
-    // merge)
+    // merge). chunk > 0: a row sees its own chunk of that many positions. cap: see kb_cap_of
     if (B <= 0 || grid_x <= 0) return 0;
     if (window <= 0 || keep_first < 0) keep_first = 0;
     if (decode && grid_x > 64) return (int)cudaErrorInvalidValue;
@@ -605,7 +594,8 @@ extern "C" int kb_attn_mma(const void* q, int ldq, void* out, int ldo, float* pa
     if (rc) return rc;
 #define AT_GO(HD, DEC)                                                                                          \
     rc = launch_attn<HD, DEC>(map, q, ldq, out, ldo, part_o, part_ml, slot, q_start, kv_len, B, nh, nkv, scale, \
-                              window, table, table_stride, n_pages, grid_x, status, st, AtRopeIn(), keep_first, sink)
+                              window, table, table_stride, n_pages, grid_x, status, st, AtRopeIn(), keep_first, sink, \
+                              chunk, kb_cap_of(cap))
     if (hd == 128) {
         if (decode) AT_GO(128, true); else AT_GO(128, false);
     } else {
@@ -710,5 +700,5 @@ extern "C" int kb_attn_decode_static(const void* q, int ldq, void* out, int ldo,
     float* part_o = base_of_device[dev];
     float* part_ml = part_o + (size_t)B * nh * n_splits * hd;
     return kb_attn_mma(q, ldq, out, ldo, part_o, part_ml, slot, q_start, kv_len, B, nh, nkv, hd, scale, window, pool,
-                       table, table_stride, n_pages, 1, n_splits, status, st, 0, nullptr);
+                       table, table_stride, n_pages, 1, n_splits, status, st, 0, nullptr, 0, nullptr);
 }

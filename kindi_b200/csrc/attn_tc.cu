@@ -68,6 +68,11 @@ __device__ __forceinline__ float ft_max3(float a, float b, float c) {
     asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
     return d;
 }
+__device__ __forceinline__ uint64_t ft_mul2(uint64_t a, uint64_t b) {
+    uint64_t d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
 // 1 / (1 + 2^-z): the logistic function of z / log2(e)
 __device__ __forceinline__ float ft_logistic2(float z) {
     float r;
@@ -92,13 +97,19 @@ __device__ __forceinline__ uint64_t umma_desc_mn_sw128(uint32_t smem_addr, uint3
 // SIG: attention without a softmax. The weight of a visible key is 1 / (1 + exp(-(score * scale + bias[h][i - j]))) with
 // a table per head over the distance whose last entry stands for every larger distance; weights are not normalised, so
 // there is no running maximum, no row sum and no rescaling of O, and the softmax warps only turn scores into weights.
-template <int FT_HD, bool SIG>
+// CAPPED: the scores pass s -> cap tanh(s / cap) (KbCap) before the softmax; where the capped scores are bounded the
+// exponentials are taken relative to zero and neither a running maximum nor a rescale of O is needed.
+#define FT_SOFTMAX 0
+#define FT_SIGMOID 1
+#define FT_CAPPED 2
+template <int FT_HD, int MODE>
 __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant__ CUtensorMap kvmap,
         const bf16* KB_STEP_DATA q, int ldq, bf16* __restrict__ out, int ldo, const int* __restrict__ slot,
         const int* __restrict__ q_start, const int* __restrict__ kv_len, int nkv, int G, float scale_log2e, int window,
         const int* __restrict__ table, int table_stride, int n_pages, int* status, int keep_first,
         const float* __restrict__ sink, const bf16* KB_STEP_DATA gate, int ldg, const float* __restrict__ bias,
-        int n_bias) {
+        int n_bias, int chunk, const __grid_constant__ KbCap cap) {
+    constexpr bool SIG = MODE == FT_SIGMOID;
     constexpr int FT_TILE_BYTES = 64 * FT_HD * 2, FT_STAGE_BYTES = 2 * FT_TILE_BYTES, FT_Q_BYTES = 128 * FT_HD * 2;
     extern __shared__ __align__(128) uint8_t smem_raw[];
     uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
@@ -145,7 +156,7 @@ __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant
     const int nrows = ntok * G;
     // pages this CTA reads
     const int p_first = pos0 + tok0, p_last = pos0 + tok0 + ntok - 1;
-    const int lo_cta = (window > 0 && p_first - window + 1 > 0) ? p_first - window + 1 : 0;
+    const int lo_cta = kb_span_lo(p_first, window, chunk);
     const int pg_lo = lo_cta / KB_PAGE, pg_hi = p_last / KB_PAGE;
     // with a window, the pages that hold the sequence's kept first positions and lie before the window's first page
     // come first; iteration i reads page pgi(i)
@@ -293,9 +304,9 @@ __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant
         // (a padding row, whose query is zero and whose result is not written, sees every key: with a span of its own
         // it would take its whole warp through the masked branch at every page)
         const int p_row = row_ok ? pos0 + tok0 + r / G : 0x3fffffff;
-        const int lo_row = (row_ok && window > 0 && p_row - window + 1 > 0) ? p_row - window + 1 : 0;
+        const int lo_row = row_ok ? kb_span_lo(p_row, window, chunk) : 0;
         const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
-        float m_ref = -INFINITY, l = 0.0f;
+        float m_ref = MODE == FT_CAPPED && cap.bounded ? 0.0f : -INFINITY, l = 0.0f;
         const float* brow = (SIG && bias != nullptr) ? bias + (size_t)(hk * G + (row_ok ? r % G : 0)) * n_bias : nullptr;
         const float b_far2 = brow != nullptr ? brow[n_bias - 1] * 1.4426950408889634f : 0.0f;
         bool ok = true;
@@ -359,16 +370,43 @@ __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant
                 if (lane == 0) mbar_arrive(b_p_ready);
                 continue;
             }
+            if constexpr (MODE == FT_CAPPED) {
+                // capped scores in powers of two, in place of the products
+                if (cap.mode == 2) {
+                    uint64_t kk[6];
+#pragma unroll
+                    for (int i = 0; i < 6; i++) kk[i] = ft_pack2(cap.k[i], cap.k[i]);
+#pragma unroll
+                    for (int c = 0; c < 64; c += 2) {
+                        const uint64_t x = ft_pack2(__uint_as_float(sv[c]), __uint_as_float(sv[c + 1]));
+                        const uint64_t r = ft_mul2(x, x);
+                        uint64_t q2 = kk[5];
+#pragma unroll
+                        for (int i = 4; i >= 0; i--) q2 = ft_fma2(q2, r, kk[i]);
+                        float x0, x1;
+                        ft_unpack2(ft_mul2(q2, x), x0, x1);
+                        sv[c] = __float_as_uint(x0);
+                        sv[c + 1] = __float_as_uint(x1);
+                    }
+                } else {
+#pragma unroll
+                    for (int c = 0; c < 64; c++) sv[c] = __float_as_uint(kb_cap2(__uint_as_float(sv[c]), cap));
+                }
+            }
+            const bool whole = key0 + 63 <= p_row && (key0 >= lo_row || key0 + 63 < keep_first);
+            const bool bounded = MODE == FT_CAPPED && cap.bounded;
             // scale, mask, row maximum
             // four independent running maxima (one long dependent chain would leave the few resident warps idle)
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-            if (key0 + 63 <= p_row && (key0 >= lo_row || key0 + 63 < keep_first)) {
+            if (whole) {
                 // the whole page lies inside this row's span (all pages but the last one or two): no masks
+                if (!bounded) {
 #pragma unroll
-                for (int c = 0; c < 64; c += 8) {
+                    for (int c = 0; c < 64; c += 8) {
 #pragma unroll
-                    for (int k = 0; k < 4; k++)
-                        mx4[k] = ft_max3(mx4[k], __uint_as_float(sv[c + 2 * k]), __uint_as_float(sv[c + 2 * k + 1]));
+                        for (int k = 0; k < 4; k++)
+                            mx4[k] = ft_max3(mx4[k], __uint_as_float(sv[c + 2 * k]), __uint_as_float(sv[c + 2 * k + 1]));
+                    }
                 }
             } else {
 #pragma unroll
@@ -376,14 +414,15 @@ __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant
                     const int p = key0 + c;
                     const float s = (p <= p_row && (p >= lo_row || p < keep_first)) ? __uint_as_float(sv[c]) : -INFINITY;
                     sv[c] = __float_as_uint(s);
-                    mx4[c & 3] = fmaxf(mx4[c & 3], s);
+                    if (!bounded) mx4[c & 3] = fmaxf(mx4[c & 3], s);
                 }
             }
             // (the scores stay as the product left them; the scale, which is positive, is applied to the maximum here
             // and to each score inside the exponent's one multiply-add)
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2e;
+            const float mul = MODE == FT_CAPPED ? 1.0f : scale_log2e;
+            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * mul;
             // lazy reference: move it only when the maximum has grown by more than FT_LAZY
-            const bool grow = mx > m_ref + FT_LAZY || (m_ref == -INFINITY && mx > -INFINITY);
+            const bool grow = !bounded && (mx > m_ref + FT_LAZY || (m_ref == -INFINITY && mx > -INFINITY));
             float f = 1.0f;
             if (grow) {
                 f = m_ref == -INFINITY ? 0.0f : ft_exp2(m_ref - mx);
@@ -417,7 +456,7 @@ __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant
             const float mr = m_ref == -INFINITY ? 0.0f : m_ref;
             // (two scores a time through the packed 32-bit multiply-add and add of sm_100: half as many instructions
             // beside the exponentials, which is what a softmax warp's time goes to)
-            const uint64_t scale2 = ft_pack2(scale_log2e, scale_log2e), nmr2 = ft_pack2(-mr, -mr);
+            const uint64_t scale2 = ft_pack2(mul, mul), nmr2 = ft_pack2(-mr, -mr);
             uint64_t sum2[4] = {0ull, 0ull, 0ull, 0ull};         // four pairs of partial sums (bit pattern of 0.0f, 0.0f)
             uint32_t pv[32];                         // the row's 64 probabilities as bf16 pairs
 #pragma unroll
@@ -504,23 +543,24 @@ __global__ void __launch_bounds__(FT_THREADS, 2) k_attn_tc(const __grid_constant
 }
 
 // grid_x = the most tiles of a sequence: ceil(longest q_len / (128 / G)) with G = nh / nkv <= 128
-template <int HD, bool SIG>
+template <int HD, int MODE>
 static int launch_attn_tc(const CUtensorMap& map, const void* q, int ldq, void* out, int ldo, const int* slot,
                           const int* q_start, const int* kv_len, int B, int nh, int nkv, float scale, int window,
                           const int* table, int table_stride, int n_pages, int grid_x, int* status, cudaStream_t st,
-                          int keep_first, const float* sink, const void* gate, int ldg, const float* bias, int n_bias) {
+                          int keep_first, const float* sink, const void* gate, int ldg, const float* bias, int n_bias, int chunk,
+                          const KbCap& cap) {
     // tiles (Q and two stages of keys and values: 96 KB at head size 128) + barriers + what aligning the base to 1024
     // can cost when it is aligned to 128: two CTAs fit an SM
     const int sm = 128 * HD * 2 + FT_STAGES * 2 * 64 * HD * 2 + 256 + 768;
     static char once_tag;               // one per instantiation: the opt-in is per (device, kernel)
     if (kb_first_use(&once_tag)) {
-        cudaError_t e = cudaFuncSetAttribute(k_attn_tc<HD, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm);
+        cudaError_t e = cudaFuncSetAttribute(k_attn_tc<HD, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, sm);
         if (e != cudaSuccess) return (int)e;
     }
     dim3 grid(nkv, grid_x, B);
-    cudaError_t e = kb_launch(k_attn_tc<HD, SIG>, grid, FT_THREADS, sm, st, map, (const bf16*)q, ldq, (bf16*)out, ldo,
+    cudaError_t e = kb_launch(k_attn_tc<HD, MODE>, grid, FT_THREADS, sm, st, map, (const bf16*)q, ldq, (bf16*)out, ldo,
                               slot, q_start, kv_len, nkv, nh / nkv, scale * 1.4426950408889634f, window, table,
-                              table_stride, n_pages, status, keep_first, sink, (const bf16*)gate, ldg, bias, n_bias);
+                              table_stride, n_pages, status, keep_first, sink, (const bf16*)gate, ldg, bias, n_bias, chunk, cap);
     return (int)e;
 }
 
@@ -535,9 +575,10 @@ static int attn_tc_shape_ok(const void* q, int ldq, const void* out, int ldo, in
 extern "C" int kb_attn_tc(const void* q, int ldq, void* out, int ldo, const int* slot, const int* q_start,
                           const int* kv_len, int B, int nh, int nkv, int hd, float scale, int window, void* pool,
                           const int* table, int table_stride, int n_pages, int grid_x, int* status, cudaStream_t st,
-                          int keep_first, const float* sink, const void* gate, int ldg) {
+                          int keep_first, const float* sink, const void* gate, int ldg, int chunk, const float* cap) {
     // sink (float [nh] or null): exp(sink[h]) joins head h's softmax denominator. gate (bf16 rows [T][ldg] laid out
-    // like out, 16-byte aligned rows, or null): out *= 1 / (1 + exp(-gate))
+    // like out, 16-byte aligned rows, or null): out *= 1 / (1 + exp(-gate)). chunk > 0: a row sees its own chunk of that
+    // many positions. cap: see kb_cap_of
     if (B <= 0 || grid_x <= 0) return 0;
     if (gate && ((ldg % 8) || ((uintptr_t)gate & 15))) return (int)cudaErrorInvalidValue;
     if (window <= 0 || keep_first < 0) keep_first = 0;
@@ -545,12 +586,18 @@ extern "C" int kb_attn_tc(const void* q, int ldq, void* out, int ldo, const int*
     CUtensorMap map;
     int rc = kb_make_map_bf16(&map, pool, (uint64_t)n_pages * 2 * nkv * KB_PAGE, hd, hd, 64);
     if (rc) return rc;
-    if (hd == 128)
-        return launch_attn_tc<128, false>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, window,
-                                          table, table_stride, n_pages, grid_x, status, st, keep_first, sink, gate, ldg,
-                                          nullptr, 0);
-    return launch_attn_tc<64, false>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, window, table,
-                                     table_stride, n_pages, grid_x, status, st, keep_first, sink, gate, ldg, nullptr, 0);
+    const KbCap kc = kb_cap_of(cap);
+#define FT_GO(HD, MODE)                                                                                                \
+    return launch_attn_tc<HD, MODE>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, window, table,    \
+                                    table_stride, n_pages, grid_x, status, st, keep_first, sink, gate, ldg, nullptr, 0, \
+                                    chunk, kc)
+    if (hd == 128) {
+        if (kc.mode) FT_GO(128, FT_CAPPED);
+        FT_GO(128, FT_SOFTMAX);
+    }
+    if (kc.mode) FT_GO(64, FT_CAPPED);
+    FT_GO(64, FT_SOFTMAX);
+#undef FT_GO
 }
 
 // Causal attention without a softmax for prompt-sized steps, same shapes and grid as kb_attn_tc: the weight of key j for
@@ -567,8 +614,10 @@ extern "C" int kb_sigattn_tc(const void* q, int ldq, void* out, int ldo, const i
     int rc = kb_make_map_bf16(&map, pool, (uint64_t)n_pages * 2 * nkv * KB_PAGE, hd, hd, 64);
     if (rc) return rc;
     if (hd == 128)
-        return launch_attn_tc<128, true>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, 0, table,
-                                         table_stride, n_pages, grid_x, status, st, 0, nullptr, nullptr, 0, bias, n_bias);
-    return launch_attn_tc<64, true>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, 0, table,
-                                    table_stride, n_pages, grid_x, status, st, 0, nullptr, nullptr, 0, bias, n_bias);
+        return launch_attn_tc<128, FT_SIGMOID>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, 0, table,
+                                         table_stride, n_pages, grid_x, status, st, 0, nullptr, nullptr, 0, bias, n_bias,
+                                         0, KbCap());
+    return launch_attn_tc<64, FT_SIGMOID>(map, q, ldq, out, ldo, slot, q_start, kv_len, B, nh, nkv, scale, 0, table,
+                                    table_stride, n_pages, grid_x, status, st, 0, nullptr, nullptr, 0, bias, n_bias,
+                                         0, KbCap());
 }

@@ -105,6 +105,52 @@ static inline KbGate kb_gate_of(int act, float lim, float alpha) {
     return k;
 }
 
+// The first position that the row at position p sees: with a window the last `window` positions, with chunks (counted from
+// the sequence's first position) its own chunk's
+__device__ __forceinline__ int kb_span_lo(int p, int window, int chunk) {
+    int lo = window > 0 && p - window + 1 > 0 ? p - window + 1 : 0;
+    if (chunk > 0) lo = max(lo, p / chunk * chunk);
+    return lo;
+}
+
+// A cap on attention scores, s -> cap tanh(s / cap), for kernels that work in powers of two: kb_cap2 turns a raw product
+// q . k into log2(e) cap tanh(scale (q . k) / cap). mode 0: no cap. mode 1: tanh(u) = 1 - 2 / (1 + e^(2u)) with the fast
+// exponential and reciprocal (2^-22 of the cap). mode 2: products known to stay within a bound (unit-norm queries and
+// keys), where an odd polynomial of degree 11 in the product, made on the host by Chebyshev interpolation, is as exact
+// and needs no special function. bounded: the capped scores lie so close to zero that exponentials and their sums cannot
+// leave the 32-bit range, so that no running maximum is needed.
+struct KbCap {
+    int mode, bounded;
+    float a;                    // 2 log2(e) scale / cap
+    float out2;                 // log2(e) cap
+    float k[6];                 // mode 2: s2 = x (k0 + k1 x^2 + ... + k5 x^10)
+};
+__device__ __forceinline__ float kb_cap2(float x, const KbCap& c) {
+    if (c.mode == 2) {
+        const float r = x * x;
+        float p = c.k[5];
+#pragma unroll
+        for (int i = 4; i >= 0; i--) p = fmaf(p, r, c.k[i]);
+        return p * x;
+    }
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * c.a));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(e + 1.0f));
+    return c.out2 * fmaf(-2.0f, r, 1.0f);
+}
+// host: ten floats (mode, bounded, a, out2, k0 .. k5), or null for no cap
+static inline KbCap kb_cap_of(const float* h) {
+    KbCap c = {};
+    if (h) {
+        c.mode = (int)h[0];
+        c.bounded = (int)h[1];
+        c.a = h[2];
+        c.out2 = h[3];
+        for (int i = 0; i < 6; i++) c.k[i] = h[4 + i];
+    }
+    return c;
+}
+
 #define KB_LAUNCH_RET() return (int)cudaGetLastError()
 
 // Programmatic dependent launch. Every kernel of the library begins with kb_pdl_launch() (when its grid is small,

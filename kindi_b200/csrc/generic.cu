@@ -1022,8 +1022,8 @@ extern "C" int kb_rope_store(const void* in, int in_dtype, int n_planes, long lo
 
 // ------------------------------------------------------------------------------------------------ attention
 // One warp per (row, query head). The row attends the keys of its sequence at positions lo..pos, lo = 0 or
-// pos - window + 1, and with a window also the sequence's first keep_first positions (at their true positions), read
-// from the cache. Keys are taken in runs of 32 that start at multiples of 32 of the absolute
+// pos - window + 1 or the start of the row's chunk, and with a window also the sequence's first keep_first positions (at
+// their true positions), read from the cache. Scores may be capped (cap > 0: cap tanh(s / cap)). Keys are taken in runs of 32 that start at multiples of 32 of the absolute
 // position (lane = position for the scores, lane = dimension for P V) with a running maximum and sum, so the order
 // of every sum depends on positions only: the same row gives the same bits whether it came in a prompt or alone.
 #define AG_MAX_HD 512
@@ -1031,7 +1031,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, int ldq, T* __restrict__ out,
         int ldo, const int* __restrict__ pos, const int* __restrict__ seq, const int* __restrict__ slot, int Tn,
         int nh, int group, int hd, float scale, int window, int keep_first, KbCacheView cv, int* status,
-        const float* __restrict__ sink, const T* KB_STEP_DATA gate, int ldg) {
+        const float* __restrict__ sink, const T* KB_STEP_DATA gate, int ldg, int chunk, float cap) {
     __shared__ float qs[4][AG_MAX_HD];
     kb_pdl_launch();
     kb_pdl_wait();
@@ -1046,7 +1046,7 @@ __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, i
     const T* qr = q + (size_t)t * ldq + (size_t)h * hd;
     for (int d = lane; d < hd; d += 32) qs[warp][d] = __fmul_rn(kb_to_f<T>(qr[d]), scale);
     __syncwarp();
-    const int lo = (window > 0 && p_q - window + 1 > 0) ? p_q - window + 1 : 0;
+    const int lo = kb_span_lo(p_q, window, chunk);
     const int* trow = cv.table + (size_t)s * cv.table_stride;
     float m = -1e30f, l = 0.0f;
     float o[AG_MAX_HD / 32];
@@ -1071,7 +1071,7 @@ __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, i
                 vrow = (const T*)cv.pool + kb_kv_offset(cv, page, 1, hk, p % KB_PAGE);
                 float a = 0.0f;
                 for (int d = 0; d < hd; d++) a = fmaf(qs[warp][d], kb_to_f<T>(kr[d]), a);
-                sc = a;
+                sc = cap > 0.0f ? cap * tanhf(a / cap) : a;
             }
         }
         const float mx = kb_warp_max(ok ? sc : -1e30f);
@@ -1120,7 +1120,7 @@ __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, i
 extern "C" int kb_attn_generic(const void* q, int dtype, int ldq, void* out, int ldo, const int* pos, const int* seq,
                                const int* slot, int T, int nh, int nkv, int hd, float scale, int window, void* pool,
                                const int* table, int table_stride, int n_pages, int* status, cudaStream_t st,
-                               int keep_first, const float* sink, const void* gate, int ldg) {
+                               int keep_first, const float* sink, const void* gate, int ldg, int chunk, float cap) {
     // sink (float [nh] or null): exp(sink[h]) joins the softmax denominator of head h. gate (rows of the queries'
     // type [T][ldg], laid out like the output, or null): out *= 1 / (1 + exp(-gate))
     if (T <= 0) return 0;
@@ -1131,10 +1131,10 @@ extern "C" int kb_attn_generic(const void* q, int dtype, int ldq, void* out, int
     int grid = (int)((items + 3) / 4);
     if (dtype == KB_F32)
         kb_launch(k_attn_generic<float>, grid, 128, 0, st, (const float*)q, ldq, (float*)out, ldo, pos, seq, slot, T, nh,
-                                                   nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const float*)gate, ldg);
+                                                   nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const float*)gate, ldg, chunk, cap);
     else
         kb_launch(k_attn_generic<bf16>, grid, 128, 0, st, (const bf16*)q, ldq, (bf16*)out, ldo, pos, seq, slot, T, nh,
-                                                  nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const bf16*)gate, ldg);
+                                                  nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const bf16*)gate, ldg, chunk, cap);
     KB_LAUNCH_RET();
 }
 

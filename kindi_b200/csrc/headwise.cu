@@ -24,6 +24,12 @@
 // sits on the sub-layer's output, the residual takes the normed and scaled branch; y = x in the run dtype is what the
 // next sub-layer reads (it reads the stream itself, not a normed copy).
 //
+// k_norm_add_norm: norms before AND after every sub-layer. v = the sum of the branch's planes (+ bias), x += w1 * rms(v)
+// (written back), y = w2 * rms(x) in the run dtype: the branch's norm, the residual add and the next sub-layer's norm in
+// one pass over the row. With a row list (the final norm) only the listed rows are worked and x stays as it is.
+//
+// k_bias_act: out = act(sum of the planes + bias), the middle of a feed-forward without a gate.
+//
 // k_cast_rows: y = x in the run dtype.
 //
 // k_glu_clamp: out = g' * sigmoid(alpha * g') * (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit), with
@@ -40,7 +46,7 @@ __global__ void __launch_bounds__(HW_THREADS) k_headnorm_rope_store(const TIN* K
         float eps, int dim_true, int norm_mode, const float* __restrict__ inv_freq,
         const double* __restrict__ inv_freq64, int rot, float t_coef, int t_every, const int* __restrict__ pos,
         const int* __restrict__ seq, const int* __restrict__ slot, int nh, int nkv, int nkv_store, int hd,
-        KbCacheView cv, int* status) {
+        KbCacheView cv, int* status, const float* __restrict__ bias) {
     extern __shared__ float sm[];
     kb_pdl_launch();
     const int t = blockIdx.x;
@@ -77,7 +83,7 @@ __global__ void __launch_bounds__(HW_THREADS) k_headnorm_rope_store(const TIN* K
     for (int i = lane; i < hd; i += 32) {
         float v = kb_to_f<TIN>(src[i]);
         for (int s = 1; s < n_planes; s++) v += kb_to_f<TIN>(src[(size_t)s * plane_stride + i]);
-        hr[i] = v;
+        hr[i] = bias ? v + bias[(size_t)h * hd + i] : v;
     }
     __syncwarp();
     if (h < nh + nkv) {
@@ -153,7 +159,7 @@ __global__ void __launch_bounds__(HW_THREADS) k_headnorm_rope_store_reg(const TI
         float eps, int dim_true, int norm_mode, const float* __restrict__ inv_freq,
         const double* __restrict__ inv_freq64, int rot, float t_coef, int t_every, const int* __restrict__ pos,
         const int* __restrict__ seq, const int* __restrict__ slot, int nh, int nkv, int nkv_store, KbCacheView cv,
-        int* status) {
+        int* status, const float* __restrict__ bias) {
     constexpr int hd = 32 * NE;
     kb_pdl_launch();
     const int t = blockIdx.x;
@@ -203,6 +209,10 @@ __global__ void __launch_bounds__(HW_THREADS) k_headnorm_rope_store_reg(const TI
 #pragma unroll
             for (int e = 0; e < NE; e++) v[e] += u[e];
         }
+        if (bias) {
+#pragma unroll
+            for (int e = 0; e < NE; e++) v[e] += bias[(size_t)h * hd + e0 + e];
+        }
         if (h < nh + nkv) {
 #pragma unroll
             for (int step = 0; step < 2; step++) {
@@ -244,7 +254,9 @@ extern "C" int kb_headnorm_rope_store(const void* in, int in_dtype, int n_planes
                                       int dim_true, int norm_mode, const float* inv_freq, const double* inv_freq64,
                                       int rot, float t_coef, int t_every, const int* pos, const int* seq,
                                       const int* slot, int T, int nh, int nkv, int nkv_store, int hd, void* pool,
-                                      const int* table, int table_stride, int n_pages, int* status, cudaStream_t st) {
+                                      const int* table, int table_stride, int n_pages, int* status, cudaStream_t st,
+                                      const float* bias) {
+    // bias (float, laid out like a row of the input, or null) joins the summed row before everything else
     if (T <= 0) return 0;
     if (rot < 0 || rot % 2 || rot > hd || norm_mode < 0 || norm_mode > 2 || dim_true < 1 || dim_true > hd ||
         (t_coef != 0.0f && t_every < 1) || (nkv_store != 0 && nkv_store != nkv))
@@ -268,7 +280,7 @@ extern "C" int kb_headnorm_rope_store(const void* in, int in_dtype, int n_planes
 #define KB_HWR(TIN, T_, NE, EX)                                                                                    \
         e = kb_launch(k_headnorm_rope_store_reg<TIN, T_, NE, EX>, gridr, HW_THREADS, 0, st, (const TIN*)in, n_planes, \
                       (size_t)plane_stride, ld_in, (T_*)qout, ldq, gq, gk, eps, dim_true, norm_mode, inv_freq,     \
-                      inv_freq64, rot, t_coef, t_every, pos, seq, slot, nh, nkv, nkv_store, cv, status)
+                      inv_freq64, rot, t_coef, t_every, pos, seq, slot, nh, nkv, nkv_store, cv, status, bias)
 #define KB_HWR2(TIN, T_, EX) do { if (ne == 4) KB_HWR(TIN, T_, 4, EX); else KB_HWR(TIN, T_, 2, EX); } while (0)
         if (in_dtype == KB_F32 && dtype == KB_F32) {
             if (rot > 0 && inv_freq64 == nullptr) return (int)cudaErrorInvalidValue;
@@ -288,7 +300,7 @@ extern "C" int kb_headnorm_rope_store(const void* in, int in_dtype, int n_planes
                                  (int)smem);                                                                       \
         e = kb_launch(k_headnorm_rope_store<TIN, T_, EX>, grid, HW_THREADS, smem, st, (const TIN*)in, n_planes,    \
                       (size_t)plane_stride, ld_in, (T_*)qout, ldq, gq, gk, eps, dim_true, norm_mode, inv_freq,     \
-                      inv_freq64, rot, t_coef, t_every, pos, seq, slot, nh, nkv, nkv_store, hd, cv, status);       \
+                      inv_freq64, rot, t_coef, t_every, pos, seq, slot, nh, nkv, nkv_store, hd, cv, status, bias); \
     } while (0)
     if (in_dtype == KB_F32 && dtype == KB_F32) {
         if (rot > 0 && inv_freq64 == nullptr) return (int)cudaErrorInvalidValue;
@@ -564,6 +576,223 @@ extern "C" int kb_postnorm_add(float* x, const float* delta, int n_delta, long l
 #undef KB_PN2
 #undef KB_PN
     return (int)e;
+}
+
+// ------------------------------------------------------------------------------------------------ norms on both sides
+// One block per row. NV > 0: the row in registers, NV float4 a thread (the width a multiple of 4, at most 1024 NV, rows
+// 16-byte aligned); NV == 0: any width, the row in shared memory.
+__device__ __forceinline__ float nn_block_sum(float v, float* red) {
+    v = kb_warp_sum(v);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float tot = red[0];
+    for (int k = 1; k < (int)(blockDim.x >> 5); k++) tot += red[k];
+    return tot;
+}
+template <typename TW> __device__ __forceinline__ float4 nn_w4(const TW* w);
+template <> __device__ __forceinline__ float4 nn_w4<float>(const float* w) { return *(const float4*)w; }
+template <> __device__ __forceinline__ float4 nn_w4<bf16>(const bf16* w) {
+    const uint2 v = *(const uint2*)w;
+    const bf16* b = (const bf16*)&v;
+    return make_float4(__bfloat162float(b[0]), __bfloat162float(b[1]), __bfloat162float(b[2]), __bfloat162float(b[3]));
+}
+template <typename TY, typename TW, int NV>
+__global__ void __launch_bounds__(256) k_norm_add_norm(float* KB_STEP_DATA x, const float* KB_STEP_DATA delta, int n_delta,
+        size_t delta_stride, const float* __restrict__ bias, const TW* __restrict__ w1, float eps1,
+        const TW* __restrict__ w2, float eps2, TY* __restrict__ y, const int* __restrict__ rows, int T, int E,
+        int write_back, int* status) {
+    extern __shared__ __align__(16) float sv[];
+    __shared__ float red[16];
+    kb_pdl_launch();
+    const int nt = blockDim.x;
+    int t = rows ? rows[blockIdx.x] : (int)blockIdx.x;
+    float4 g1[NV > 0 ? NV : 1], g2[NV > 0 ? NV : 1];
+    if (NV > 0) {
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (threadIdx.x + k * nt) * 4;
+            if (i < E) {
+                g1[k] = nn_w4<TW>(w1 + i);
+                g2[k] = nn_w4<TW>(w2 + i);
+            }
+        }
+    }
+    kb_pdl_wait();
+    if (t < 0 || t >= T) {                             // uniform over the block
+        if (threadIdx.x == 0) atomicOr(status, KB_ST_BAD_ROW);
+        t = 0;
+    }
+    float* xr = x + (size_t)t * E;
+    const float* dr = delta + (size_t)t * E;
+    TY* yr = y + (size_t)blockIdx.x * E;
+    if (NV > 0) {
+        float4 v[NV > 0 ? NV : 1], xv[NV > 0 ? NV : 1];
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (threadIdx.x + k * nt) * 4;
+            v[k] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            xv[k] = v[k];
+            if (i < E) {
+                xv[k] = *(const float4*)(xr + i);
+                v[k] = *(const float4*)(dr + i);
+            }
+        }
+        for (int s = 1; s < n_delta; s++) {
+#pragma unroll
+            for (int k = 0; k < NV; k++) {
+                const int i = (threadIdx.x + k * nt) * 4;
+                if (i < E) {
+                    const float4 d = *(const float4*)(dr + (size_t)s * delta_stride + i);
+                    v[k].x += d.x; v[k].y += d.y; v[k].z += d.z; v[k].w += d.w;
+                }
+            }
+        }
+        float ss = 0.0f;
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (threadIdx.x + k * nt) * 4;
+            if (bias && i < E) {
+                const float4 d = *(const float4*)(bias + i);
+                v[k].x += d.x; v[k].y += d.y; v[k].z += d.z; v[k].w += d.w;
+            }
+            ss = fmaf(v[k].x, v[k].x, ss); ss = fmaf(v[k].y, v[k].y, ss);
+            ss = fmaf(v[k].z, v[k].z, ss); ss = fmaf(v[k].w, v[k].w, ss);
+        }
+        const float f1 = 1.0f / sqrtf(nn_block_sum(ss, red) / (float)E + eps1);
+        ss = 0.0f;
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (threadIdx.x + k * nt) * 4;
+            if (i < E) {
+                xv[k].x = __fadd_rn(xv[k].x, __fmul_rn(__fmul_rn(v[k].x, f1), g1[k].x));
+                xv[k].y = __fadd_rn(xv[k].y, __fmul_rn(__fmul_rn(v[k].y, f1), g1[k].y));
+                xv[k].z = __fadd_rn(xv[k].z, __fmul_rn(__fmul_rn(v[k].z, f1), g1[k].z));
+                xv[k].w = __fadd_rn(xv[k].w, __fmul_rn(__fmul_rn(v[k].w, f1), g1[k].w));
+                if (write_back) *(float4*)(xr + i) = xv[k];
+            }
+            ss = fmaf(xv[k].x, xv[k].x, ss); ss = fmaf(xv[k].y, xv[k].y, ss);
+            ss = fmaf(xv[k].z, xv[k].z, ss); ss = fmaf(xv[k].w, xv[k].w, ss);
+        }
+        const float f2 = 1.0f / sqrtf(nn_block_sum(ss, red + 8) / (float)E + eps2);
+#pragma unroll
+        for (int k = 0; k < NV; k++) {
+            const int i = (threadIdx.x + k * nt) * 4;
+            if (i < E) {
+                const float o[4] = {__fmul_rn(__fmul_rn(xv[k].x, f2), g2[k].x), __fmul_rn(__fmul_rn(xv[k].y, f2), g2[k].y),
+                                    __fmul_rn(__fmul_rn(xv[k].z, f2), g2[k].z), __fmul_rn(__fmul_rn(xv[k].w, f2), g2[k].w)};
+                hw_store<4>(yr + i, o);
+            }
+        }
+        return;
+    }
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < E; i += nt) {
+        float v = dr[i];
+        for (int s = 1; s < n_delta; s++) v += dr[(size_t)s * delta_stride + i];
+        if (bias) v += bias[i];
+        sv[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float f1 = 1.0f / sqrtf(nn_block_sum(ss, red) / (float)E + eps1);
+    ss = 0.0f;
+    for (int i = threadIdx.x; i < E; i += nt) {
+        const float v = __fadd_rn(xr[i], __fmul_rn(__fmul_rn(sv[i], f1), kb_to_f<TW>(w1[i])));
+        if (write_back) xr[i] = v;
+        sv[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float f2 = 1.0f / sqrtf(nn_block_sum(ss, red + 8) / (float)E + eps2);
+    for (int i = threadIdx.x; i < E; i += nt)
+        yr[i] = kb_from_f<TY>(__fmul_rn(__fmul_rn(sv[i], f2), kb_to_f<TW>(w2[i])));
+}
+
+extern "C" int kb_norm_add_norm(float* x, const float* delta, int n_delta, long long delta_stride, const float* bias,
+                                const void* w1, float eps1, const void* w2, float eps2, int wdtype, void* y, int ydtype,
+                                const int* rows, int n_out, int T, int E, int write_back, int* status, cudaStream_t st) {
+    if (n_out <= 0 || E <= 0) return 0;
+    if (n_delta < 1 || (rows && write_back)) return (int)cudaErrorInvalidValue;
+    const int wel = wdtype == KB_F32 ? 4 : 2, yel = ydtype == KB_F32 ? 4 : 2;
+    const bool vec = E % 4 == 0 && E <= 8192 && delta_stride % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)delta % 16 == 0 &&
+                     (uintptr_t)bias % 16 == 0 && (uintptr_t)w1 % (4 * wel) == 0 && (uintptr_t)w2 % (4 * wel) == 0 &&
+                     (uintptr_t)y % (4 * yel) == 0;
+    const size_t smem = vec ? 0 : (size_t)E * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    // a block as wide as the row needs, up to 256 threads
+    const int q = (E / 4 + 31) / 32 * 32, nt = vec ? (q < 256 ? q : 256) : 256;
+    const int nv = vec ? (E / 4 + nt - 1) / nt : 0;
+    cudaError_t e = cudaSuccess;
+#define KB_NN(TY, TW, NV)                                                                                          \
+    do {                                                                                                           \
+        if (smem > 48 * 1024)                                                                                      \
+            cudaFuncSetAttribute(k_norm_add_norm<TY, TW, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        e = kb_launch(k_norm_add_norm<TY, TW, NV>, n_out, nt, smem, st, x, delta, n_delta, (size_t)delta_stride, bias, \
+                      (const TW*)w1, eps1, (const TW*)w2, eps2, (TY*)y, rows, T, E, write_back, status);           \
+    } while (0)
+#define KB_NN2(TY, TW)                                                                                             \
+    do {                                                                                                           \
+        if (nv == 0) KB_NN(TY, TW, 0); else if (nv == 1) KB_NN(TY, TW, 1); else if (nv == 2) KB_NN(TY, TW, 2);     \
+        else if (nv <= 4) KB_NN(TY, TW, 4); else KB_NN(TY, TW, 8);                                                 \
+    } while (0)
+    if (ydtype == KB_F32 && wdtype == KB_F32) KB_NN2(float, float);
+    else if (ydtype == KB_F32 && wdtype == KB_BF16) KB_NN2(float, bf16);
+    else if (ydtype == KB_BF16 && wdtype == KB_BF16) KB_NN2(bf16, bf16);
+    else if (ydtype == KB_BF16 && wdtype == KB_F32) KB_NN2(bf16, float);
+    else return (int)cudaErrorInvalidValue;
+#undef KB_NN2
+#undef KB_NN
+    return (int)e;
+}
+
+// ------------------------------------------------------------------------------------------------ bias and activation
+template <typename TIN, typename T, bool VEC>
+__global__ void __launch_bounds__(256) k_bias_act(const TIN* KB_STEP_DATA in, int n_planes, size_t plane_stride, int ldi,
+        const float* __restrict__ bias, int act, T* out, int ldo, int N) {
+    kb_pdl_launch();
+    kb_pdl_wait();
+    const size_t t = blockIdx.x;
+    if (VEC) {
+        const int c = (blockIdx.y * 256 + threadIdx.x) * 4;
+        if (c >= N) return;
+        float v[4];
+        hw_load<4>(in + t * ldi + c, v);
+        for (int s = 1; s < n_planes; s++) {
+            float u[4];
+            hw_load<4>(in + (size_t)s * plane_stride + t * ldi + c, u);
+#pragma unroll
+            for (int k = 0; k < 4; k++) v[k] += u[k];
+        }
+#pragma unroll
+        for (int k = 0; k < 4; k++) v[k] = kb_act(bias ? v[k] + bias[c + k] : v[k], act);
+        hw_store<4>(out + t * ldo + c, v);
+        return;
+    }
+    const int c = blockIdx.y * 256 + threadIdx.x;
+    if (c >= N) return;
+    float v = kb_to_f<TIN>(in[t * ldi + c]);
+    for (int s = 1; s < n_planes; s++) v += kb_to_f<TIN>(in[(size_t)s * plane_stride + t * ldi + c]);
+    out[t * ldo + c] = kb_from_f<T>(kb_act(bias ? v + bias[c] : v, act));
+}
+
+extern "C" int kb_bias_act(const void* in, int idtype, int n_planes, long long plane_stride, int ldi, const float* bias,
+                           int act, void* out, int odtype, int ldo, int T, int N, cudaStream_t st) {
+    if (T <= 0 || N <= 0) return 0;
+    const int iel = idtype == KB_F32 ? 4 : 2, oel = odtype == KB_F32 ? 4 : 2;
+    const bool vec = N % 4 == 0 && ldi % 4 == 0 && ldo % 4 == 0 && plane_stride % 4 == 0 && (uintptr_t)in % (4 * iel) == 0 &&
+                     (uintptr_t)out % (4 * oel) == 0;
+    const dim3 grid(T, ((vec ? N / 4 : N) + 255) / 256);
+#define KB_BA(TIN, TO)                                                                                             \
+    do {                                                                                                           \
+        if (vec) kb_launch(k_bias_act<TIN, TO, true>, grid, 256, 0, st, (const TIN*)in, n_planes,                  \
+                           (size_t)plane_stride, ldi, bias, act, (TO*)out, ldo, N);                                \
+        else kb_launch(k_bias_act<TIN, TO, false>, grid, 256, 0, st, (const TIN*)in, n_planes,                     \
+                       (size_t)plane_stride, ldi, bias, act, (TO*)out, ldo, N);                                    \
+    } while (0)
+    if (idtype == KB_F32 && odtype == KB_F32) KB_BA(float, float);
+    else if (idtype == KB_F32 && odtype == KB_BF16) KB_BA(float, bf16);
+    else if (idtype == KB_BF16 && odtype == KB_BF16) KB_BA(bf16, bf16);
+    else return (int)cudaErrorInvalidValue;
+#undef KB_BA
+    KB_LAUNCH_RET();
 }
 
 template <typename TY>

@@ -84,7 +84,7 @@ extern "C" int kb_mix_cat(const float* x, const float* delta, int n_delta, long 
 }
 
 // ------------------------------------------------------------------------------------------------ short convolution
-// y[t][c] = act(sum_j w[c][j] * u[t - (taps - 1) + j][c]), u = input columns col0.. (+ bias), over the positions of
+// y[t][c] = act(obias[c] + sum_j w[c][j] * u[t - (taps - 1) + j][c]), u = input columns col0.. (+ bias), over the positions of
 // the row's own sequence; positions before this step's rows come from the sequence's tails (state: [taps - 1][C],
 // oldest first, zero when the sequence starts), and the step's last taps - 1 inputs become the new tails. The thread
 // of a sequence's first row of the step works its first taps - 1 rows (the only ones that read tails) and then writes
@@ -94,7 +94,8 @@ template <typename TIN, typename TO>
 __global__ void __launch_bounds__(128) k_short_conv(const TIN* KB_STEP_DATA in, int n_planes, size_t plane_stride,
         int ld_in, int col0, int C, const float* __restrict__ bias, const float* __restrict__ w, int taps, int act,
         float* state, size_t state_stride, const int* __restrict__ pos, const int* __restrict__ seq,
-        const int* __restrict__ slot, const int* __restrict__ q_start, TO* __restrict__ out, int ldo) {
+        const int* __restrict__ slot, const int* __restrict__ q_start, TO* __restrict__ out, int ldo,
+        const float* __restrict__ obias) {
     kb_pdl_launch();
     const int t = blockIdx.x;
     const int c = blockIdx.y * 128 + threadIdx.x;
@@ -109,11 +110,11 @@ __global__ void __launch_bounds__(128) k_short_conv(const TIN* KB_STEP_DATA in, 
     float wr[SC_MAX_TAPS];
 #pragma unroll
     for (int j = 0; j < SC_MAX_TAPS; j++) wr[j] = j < taps ? w[(size_t)c * taps + j] : 0.0f;
-    const float bs = bias ? bias[c] : 0.0f;
+    const float bs = bias ? bias[c] : 0.0f, ob = obias ? obias[c] : 0.0f;
     kb_pdl_wait();
 #define SC_U(row) (rc_rd<TIN>(in + (size_t)(row) * ld_in, n_planes, plane_stride, (size_t)col0 + c) + bs)
     if (i >= taps - 1) {
-        float acc = 0.0f;
+        float acc = ob;
 #pragma unroll
         for (int j = 0; j < SC_MAX_TAPS; j++)
             if (j < taps) acc = fmaf(wr[j], SC_U(t - (taps - 1) + j), acc);
@@ -127,7 +128,7 @@ __global__ void __launch_bounds__(128) k_short_conv(const TIN* KB_STEP_DATA in, 
     for (int j = 0; j < SC_MAX_TAPS; j++) tl[j] = j < taps - 1 ? tails[(size_t)j * C + c] : 0.0f;
     const int head = n < taps - 1 ? n : taps - 1;
     for (int i2 = 0; i2 < head; i2++) {
-        float acc = 0.0f;
+        float acc = ob;
 #pragma unroll
         for (int j = 0; j < SC_MAX_TAPS; j++) {
             if (j >= taps) continue;
@@ -164,13 +165,15 @@ __global__ void __launch_bounds__(128) k_short_conv(const TIN* KB_STEP_DATA in, 
 extern "C" int kb_short_conv(const void* in, int idtype, int n_planes, long long plane_stride, int ld_in, int col0,
                              int C, const float* bias, const float* w, int taps, int act, float* state,
                              long long state_stride, const int* pos, const int* seq, const int* slot,
-                             const int* q_start, void* out, int odtype, int ldo, int T, cudaStream_t st) {
+                             const int* q_start, void* out, int odtype, int ldo, int T, cudaStream_t st,
+                             const float* obias) {
+    // bias (float [C] or null) joins every input, obias every result (before the activation)
     if (T <= 0 || C <= 0) return 0;
     if (taps < 1 || taps > SC_MAX_TAPS) return (int)cudaErrorInvalidValue;
     dim3 grid(T, (C + 127) / 128);
 #define KB_SC(TIN, TO)                                                                                              \
     kb_launch(k_short_conv<TIN, TO>, grid, 128, 0, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in, col0, \
-              C, bias, w, taps, act, state, (size_t)state_stride, pos, seq, slot, q_start, (TO*)out, ldo)
+              C, bias, w, taps, act, state, (size_t)state_stride, pos, seq, slot, q_start, (TO*)out, ldo, obias)
     if (idtype == KB_F32 && odtype == KB_F32) KB_SC(float, float);
     else if (idtype == KB_BF16 && odtype == KB_F32) KB_SC(bf16, float);
     else if (idtype == KB_F32 && odtype == KB_BF16) KB_SC(float, bf16);

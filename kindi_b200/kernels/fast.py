@@ -233,16 +233,20 @@ def gemm_swiglu_decode(a: torch.Tensor, w_grouped: torch.Tensor, out: torch.Tens
 
 
 def attention_bf16(ctx, q, out, nh, nkv, hd, scale, window, pool, table, n_pages, keep_first: int = 0,
-                   sink=None, gate=None) -> int:
+                   sink=None, gate=None, chunk: int = 0, cap=None) -> int:
     """the tensor-core attention kernel, where it takes the shape: head size 64 or 128, bf16, aligned rows. Returns 0
     (not taken), 1 (done) or 2 (done, and the output gate ``gate`` was applied inside the kernel)"""
     if hd not in (64, 128) or q.dtype != torch.bfloat16 or q.stride(0) % 8 or q.data_ptr() % 16:
         return 0
     g = nh // nkv
+    more = dict(status=ctx.status, keep_first=keep_first, sink=sink, chunk=chunk,
+                cap=cap.host if cap is not None else None)
     if ctx.decode and g <= 16:
         splits = decode_splits(ctx, nkv)
+        if chunk > 0:
+            splits = min(splits, -(-chunk // K.PAGE) + 1)          # (no more splits than pages a chunk can touch)
         K.attn_mma(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, nkv, hd, scale, window, pool, table,
-                   n_pages, decode=True, grid_x=splits, status=ctx.status, keep_first=keep_first, sink=sink)
+                   n_pages, decode=True, grid_x=splits, **more)
         return 1
     # (in a recording ctx.max_q is the most rows a sequence can bring: the grid then has tiles to spare, which leave)
     if g <= 128 and out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0:
@@ -251,11 +255,10 @@ def attention_bf16(ctx, q, out, nh, nkv, hd, scale, window, pool, table, n_pages
         fuse = (gate is not None and gate.dim() == 2 and gate.dtype == torch.bfloat16 and gate.stride(1) == 1
                 and gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)
         K.attn_tc(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, nkv, hd, scale, window, pool, table, n_pages,
-                  grid_x=-(-ctx.max_q // (128 // g)), status=ctx.status, keep_first=keep_first, sink=sink,
-                  gate=gate if fuse else None)
+                  grid_x=-(-ctx.max_q // (128 // g)), gate=gate if fuse else None, **more)
         return 2 if fuse else 1
     K.attn_mma(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, nkv, hd, scale, window, pool, table, n_pages,
-               decode=False, grid_x=-(-ctx.max_q * g // 64), status=ctx.status, keep_first=keep_first, sink=sink)
+               decode=False, grid_x=-(-ctx.max_q * g // 64), **more)
     return 1
 
 

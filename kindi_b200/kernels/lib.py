@@ -28,6 +28,11 @@ class KernelError(RuntimeError):
     pass
 
 
+# the arguments the two forms of a gated recurrence share (SS_PARAMS in csrc/ssd.cu)
+_SCAN = [c_int, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_longlong, c_int,
+         c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+         c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p]
+
 _SIGS = {
     "kb_embed": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
     "kb_logit_post": [c_void_p, c_longlong, c_float, c_float, c_void_p],
@@ -41,7 +46,7 @@ _SIGS = {
     "kb_rope_table": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "kb_attn_generic": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                         c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
-                        c_void_p, c_int],
+                        c_void_p, c_int, c_int, c_float],
     "kb_gate_mul": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_int,
                     c_void_p],
     "kb_gated_rmsnorm": [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p,
@@ -68,7 +73,7 @@ _SIGS = {
     "kb_mix_cat": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "kb_short_conv": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
                       c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                      c_void_p],
+                      c_void_p, c_void_p],
     "kb_delta_rule": [c_void_p, c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p,
                       c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
                       c_int, c_void_p],
@@ -112,12 +117,13 @@ _SIGS = {
                               c_void_p, c_void_p, c_void_p, c_int, c_float, c_float],
     "kb_attn_mma": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                     c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                    c_int, c_void_p],
+                    c_int, c_void_p, c_int, c_void_p],
     "kb_attn_decode_rope": [c_void_p, c_int, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p,
                             c_int, c_int, c_int, c_void_p, c_void_p],
     "kb_attn_tc": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                   c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int],
+                   c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int,
+                   c_int, c_void_p],
     "kb_sample": [c_void_p, c_longlong, c_int, c_int, c_float, c_int, c_float, c_float, c_int, c_void_p, c_void_p,
                   c_void_p],
     "kb_penalize": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_int, c_float, c_void_p],
@@ -125,13 +131,23 @@ _SIGS = {
     "kb_headnorm_rope_store": [c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p,
                                c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p,
-                               c_void_p],
+                               c_void_p, c_void_p],
     "kb_diff_combine": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float,
                         c_float, c_void_p],
     "kb_head_gate_mul": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int,
                          c_int, c_int, c_void_p],
     "kb_postnorm_add": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p,
                         c_int, c_int, c_int, c_void_p],
+    "kb_norm_add_norm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_float, c_int,
+                         c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "kb_bias_act": [c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                    c_void_p],
+    "kb_gated_scan": _SCAN + [c_void_p],
+    "kb_gated_scan_chunked": _SCAN + [c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+    "kb_scan_run": [],
+    "kb_scan_norm": [c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_longlong,
+                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
+                     c_void_p, c_int, c_int, c_void_p],
     "kb_cast_rows": [c_void_p, c_void_p, c_int, c_longlong, c_void_p],
     "kb_glu_clamp": [c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                      c_float, c_void_p],
@@ -182,7 +198,7 @@ class KernelTiming:
     def __getattr__(self, name):                       # stands in for the library while timing is on
         fn = getattr(_lib, name)
         if not name.startswith("kb_") or name in ("kb_set_pdl", "kb_gemm_tc_splits", "kb_rope_table_min_rows",
-                                                  "kb_moe_gemm_tile", "kb_moe_gemm_tc_tile"):
+                                                  "kb_moe_gemm_tile", "kb_moe_gemm_tc_tile", "kb_scan_run"):
             return fn
 
         def timed(*args):
@@ -715,9 +731,11 @@ def rope_store(qkv: torch.Tensor, qout: torch.Tensor, inv_freq: torch.Tensor, ro
 
 def attn_generic(q: torch.Tensor, out: torch.Tensor, pos, seq, slot, nh: int, nkv: int, hd: int, scale: float,
                  window: int, pool: torch.Tensor, table: torch.Tensor, n_pages: int, status: torch.Tensor,
-                 keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                 keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                 chunk: int = 0, softcap: float = 0.0) -> None:
     """attention of each row of q ([T, >= nh hd], row stride free) over its sequence's cached keys and values: all
-    positions up to the row's, or with ``window`` the last ``window`` of them and the sequence's first ``keep_first``.
+    positions up to the row's, or with ``window`` the last ``window`` of them and the sequence's first ``keep_first``,
+    or with ``chunk`` those of its own chunk of that many positions. ``softcap`` > 0: scores are capped.
     ``sink`` (float32 [nh]): exp(sink[h]) joins head h's softmax denominator. ``gate`` (rows of q's dtype, laid out
     like ``out``): the output is multiplied by the logistic function of it"""
     _need_cuda(q, out, pool, table, sink, gate)
@@ -732,7 +750,8 @@ def attn_generic(q: torch.Tensor, out: torch.Tensor, pos, seq, slot, nh: int, nk
     _check(load().kb_attn_generic(_p(q), dt(q), q.stride(0), _p(out), out.stride(0), _p(pos), _p(seq), _p(slot), T,
                                   nh, nkv, hd, float(scale), int(window), _p(pool), _p(table), table.stride(0),
                                   n_pages, _p(status), _stream(), int(keep_first), _p(sink), _p(gate),
-                                  gate.stride(0) if gate is not None else 0), "attn_generic")
+                                  gate.stride(0) if gate is not None else 0, int(chunk), float(softcap)),
+           "attn_generic")
 
 
 def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int = 0, act: str = "silu") -> None:
@@ -826,11 +845,13 @@ def gemm_tc_splits(K: int, wanted: int) -> int:
 
 def attn_mma(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, nh: int, nkv: int, hd: int,
              scale: float, window: int, pool: torch.Tensor, table: torch.Tensor, n_pages: int, *, decode: bool,
-             grid_x: int, status: torch.Tensor, keep_first: int = 0, sink: Optional[torch.Tensor] = None) -> None:
+             grid_x: int, status: torch.Tensor, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
+             chunk: int = 0, cap=None) -> None:
     """tensor-core attention over the cache (bf16, head size 64 or 128). decode: one row per sequence, grid_x =
     position splits; else grid_x = ceil(most rows of a sequence * (nh / nkv) / 64). ``keep_first``: with a window,
     the sequence's first positions that stay visible. ``sink`` (float32 [nh]): exp(sink[h]) joins head h's softmax
-    denominator"""
+    denominator. ``chunk`` > 0: a row sees the positions of its own chunk. ``cap``: the ten host floats of a score cap
+    (``attention.ScoreCap.host``)"""
     _need_cuda(q, out, pool, table, sink)
     if sink is not None:
         assert sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh
@@ -843,7 +864,7 @@ def attn_mma(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, 
     _check(load().kb_attn_mma(_p(q), q.stride(0), _p(out), out.stride(0), _p(part_o), _p(part_ml), _p(slot),
                               _p(q_start), _p(kv_len), B, nh, nkv, hd, float(scale), int(window), _p(pool), _p(table),
                               table.stride(0), n_pages, 1 if decode else 0, grid_x, _p(status), _stream(),
-                              int(keep_first), _p(sink)), "attn_mma")
+                              int(keep_first), _p(sink), int(chunk), cap), "attn_mma")
     if decode and grid_x > 1:
         add_launches(1)         # the merge of the position splits
 
@@ -873,11 +894,11 @@ def attn_decode_rope(qkv: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tenso
 def attn_tc(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, nh: int, nkv: int, hd: int,
             scale: float, window: int, pool: torch.Tensor, table: torch.Tensor, n_pages: int, *, grid_x: int,
             status: torch.Tensor, keep_first: int = 0, sink: Optional[torch.Tensor] = None,
-            gate: Optional[torch.Tensor] = None) -> None:
+            gate: Optional[torch.Tensor] = None, chunk: int = 0, cap=None) -> None:
     """tcgen05 attention for prompt-sized steps (bf16, head size 64 or 128): grid_x = ceil(most rows of a sequence /
     (128 // (nh / nkv))). ``keep_first``: with a window, the sequence's first positions that stay visible. ``sink``
     (float32 [nh]): exp(sink[h]) joins head h's softmax denominator. ``gate`` (bf16 rows laid out like ``out``, rows
-    16-byte aligned): the output is multiplied by the logistic function of it"""
+    16-byte aligned): the output is multiplied by the logistic function of it. ``chunk``, ``cap``: as for attn_mma"""
     _need_cuda(q, out, pool, table, sink, gate)
     if sink is not None:
         assert sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh
@@ -888,7 +909,7 @@ def attn_tc(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, n
     _check(load().kb_attn_tc(_p(q), q.stride(0), _p(out), out.stride(0), _p(slot), _p(q_start), _p(kv_len), B, nh, nkv,
                              hd, float(scale), int(window), _p(pool), _p(table), table.stride(0), n_pages, grid_x,
                              _p(status), _stream(), int(keep_first), _p(sink), _p(gate),
-                             gate.stride(0) if gate is not None else 0), "attn_tc")
+                             gate.stride(0) if gate is not None else 0, int(chunk), cap), "attn_tc")
 
 
 # ----------------------------------------------------------------------------------------------- stateful mixers
@@ -922,15 +943,17 @@ def mix_cat(x: torch.Tensor, delta: Optional[torch.Tensor], scale: Optional[torc
 
 
 def short_conv(a: torch.Tensor, col0: int, C: int, bias: Optional[torch.Tensor], w: torch.Tensor, act: bool,
-               tails: torch.Tensor, pos, seq, slot, q_start, out: torch.Tensor) -> None:
+               tails: torch.Tensor, pos, seq, slot, q_start, out: torch.Tensor,
+               out_bias: Optional[torch.Tensor] = None) -> None:
     """causal convolution over time per channel on columns ``col0 .. col0 + C`` of ``a`` (rows or 32-bit planes), plus
-    ``bias`` before the convolution; ``w`` float32 [C, taps] (the last tap meets the current token); ``act``: silu
+    ``bias`` before the convolution and ``out_bias`` after it; ``w`` float32 [C, taps] (the last tap meets the current token); ``act``: silu
     after it. ``tails``: float32 [slots, >= (taps - 1) * C] (a view whose rows may be strided), the sequence's last
     taps - 1 inputs, read for positions before this step and rewritten. ``out`` [T, C] (a view is fine)"""
-    _need_cuda(a, bias, w, tails, out)
+    _need_cuda(a, bias, w, tails, out, out_bias)
     n_planes, pstride, ld = _planes_of(a)
     T = a.shape[-2]
     taps = w.shape[1]
+    assert out_bias is None or (out_bias.dtype == torch.float32 and out_bias.is_contiguous() and out_bias.numel() == C)
     assert w.dtype == torch.float32 and w.is_contiguous() and w.shape[0] == C and a.shape[-1] >= col0 + C
     assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == C)
     assert tails.dtype == torch.float32 and tails.stride(1) == 1 and tails.shape[1] >= (taps - 1) * C
@@ -939,7 +962,7 @@ def short_conv(a: torch.Tensor, col0: int, C: int, bias: Optional[torch.Tensor],
         raise KernelError("kindi_b200: a short convolution has 1 to 8 taps, found %d" % taps)
     _check(load().kb_short_conv(_p(a), dt(a), n_planes, pstride, ld, col0, C, _p(bias), _p(w), taps, 1 if act else 0,
                                 _p(tails), tails.stride(0), _p(pos), _p(seq), _p(slot), _p(q_start), _p(out), dt(out),
-                                out.stride(0), T, _stream()), "short_conv")
+                                out.stride(0), T, _stream(), _p(out_bias)), "short_conv")
 
 
 DELTA_CHUNK = 64            # rows of a run (DC_C of the kernels)
@@ -1137,13 +1160,15 @@ def headnorm_rope_store(qkv: torch.Tensor, qout: torch.Tensor, gq: Optional[torc
                         eps: float, dim_true: int, norm: str, inv_freq: Optional[torch.Tensor],
                         inv_freq64: Optional[torch.Tensor], rot: int, t_coef: float, t_every: int, pos, seq, slot,
                         nh: int, nkv: int, nkv_store: int, hd: int, pool: Optional[torch.Tensor], table: torch.Tensor,
-                        n_pages: int, status: torch.Tensor) -> None:
+                        n_pages: int, status: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
     """every query and key head of a row through its OWN root-mean-square norm over ``dim_true`` elements (``norm``:
     "none", "before" or "after" the rotation; gains ``gq`` / ``gk`` float32 [hd] shared by the heads, None for a unit
     norm), the rotation of the pairs (i, i + rot/2), and on queries the temperature ``1 + t_coef ln(floor((pos + 1) /
     t_every) + 1)``; queries to ``qout``, keys and values into their pages. qkv: rows or 32-bit planes of [q heads |
-    k heads | v heads]. float32 rows rotate by ``inv_freq64`` (float64), everything else by ``inv_freq``"""
-    _need_cuda(qkv, qout, gq, gk, inv_freq, inv_freq64, pool, table)
+    k heads | v heads]. float32 rows rotate by ``inv_freq64`` (float64), everything else by ``inv_freq``. ``bias`` (float32,
+    laid out like a row) joins the summed row first"""
+    _need_cuda(qkv, qout, gq, gk, inv_freq, inv_freq64, pool, table, bias)
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == (nh + 2 * nkv) * hd)
     planes = qkv.shape[0] if qkv.dim() == 3 else 1
     T = qkv.shape[-2]
     assert qkv.stride(-1) == 1 and qkv.shape[-1] >= (nh + 2 * nkv) * hd and qout.stride(1) == 1
@@ -1160,7 +1185,7 @@ def headnorm_rope_store(qkv: torch.Tensor, qout: torch.Tensor, gq: Optional[torc
                                        qout.stride(0), _p(gq), _p(gk), float(eps), int(dim_true), mode, _p(inv_freq),
                                        _p(inv_freq64), int(rot), float(t_coef), int(t_every), _p(pos), _p(seq),
                                        _p(slot), T, nh, nkv, nkv_store, hd, _p(pool), _p(table), table.stride(0),
-                                       n_pages, _p(status), _stream())
+                                       n_pages, _p(status), _stream(), _p(bias))
     _check(rc, "headnorm_rope_store")
 
 
@@ -1201,6 +1226,119 @@ def postnorm_add(x: torch.Tensor, delta: torch.Tensor, bias: Optional[torch.Tens
     assert y is None or (y.shape == (T, E) and y.is_contiguous())
     _check(load().kb_postnorm_add(_p(x), _p(delta), delta.shape[0], delta.stride(0), _p(bias), _p(w), _p(ls), dt(w),
                                   float(eps), _p(y), dt(y) if y is not None else F32, T, E, _stream()), "postnorm_add")
+
+
+def norm_add_norm(x: torch.Tensor, delta: torch.Tensor, bias: Optional[torch.Tensor], w1: torch.Tensor, eps1: float,
+                  w2: torch.Tensor, eps2: float, y: torch.Tensor, rows: Optional[torch.Tensor], write_back: bool,
+                  status: torch.Tensor) -> None:
+    """x += w1 * rms(sum of the planes ``delta`` [S, T, E] + bias) (``write_back``: in place), y = w2 * rms(x) in y's
+    dtype; ``rows`` (int32): only these rows, in this order, and x stays as it is"""
+    _need_cuda(x, delta, bias, w1, w2, y, rows)
+    T, E = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and delta.dtype == torch.float32 and delta.dim() == 3
+    assert delta.shape[1:] == (T, E) and delta.stride(2) == 1 and delta.stride(1) == E
+    assert w1.dtype == w2.dtype and w1.numel() == E == w2.numel() and w1.is_contiguous() and w2.is_contiguous()
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == E and bias.is_contiguous())
+    n_out = y.shape[0]
+    assert y.shape == (n_out, E) and y.is_contiguous() and n_out == (T if rows is None else rows.numel())
+    assert rows is None or (rows.dtype == torch.int32 and not write_back)
+    _check(load().kb_norm_add_norm(_p(x), _p(delta), delta.shape[0], delta.stride(0), _p(bias), _p(w1), float(eps1),
+                                   _p(w2), float(eps2), dt(w1), _p(y), dt(y), _p(rows), n_out, T, E,
+                                   1 if write_back else 0, _p(status), _stream()), "norm_add_norm")
+
+
+def bias_act(a: torch.Tensor, bias: Optional[torch.Tensor], act: str, out: torch.Tensor) -> None:
+    """out = act(a + bias); ``a``: rows [T, N] or 32-bit planes [S, T, N]; ``act``: a key of ``ACT``"""
+    _need_cuda(a, bias, out)
+    T, N = out.shape
+    n_planes, pstride, ld = _planes_of(a)
+    assert a.shape[-2:] == (T, N) and out.stride(1) == 1
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == N and bias.is_contiguous())
+    _check(load().kb_bias_act(_p(a), dt(a), n_planes, pstride, ld, _p(bias), ACT[act], _p(out), dt(out), out.stride(0), T,
+                              N, _stream()), "bias_act")
+
+
+# ------------------------------------------------------------------------------- matrix states under one decay per head
+SCAN_KIND = {"mlstm": 0, "mamba2": 1}
+
+
+@functools.lru_cache(maxsize=1)
+def scan_run() -> int:
+    """tokens of a run in the form for long prompts"""
+    return load().kb_scan_run()
+
+
+def gated_scan(kind: str, src: torch.Tensor, oq: int, ok: int, ov: int, per: int, gates: torch.Tensor, og0: int, og1: int,
+               p0: torch.Tensor, p1: torch.Tensor, p2: Optional[torch.Tensor], cap: float, qscale: float, B: int, H: int,
+               d: int, dv: int, q_start, slot, state: torch.Tensor, m_state: Optional[torch.Tensor], out: torch.Tensor,
+               nq: Optional[torch.Tensor], m_rows: Optional[torch.Tensor], chunked: bool = False) -> None:
+    """``S_t = a_t S_(t-1) + w_t k_t v_t^T``, ``o_t = S_t^T q_t`` over the packed rows of ``B`` sequences, H heads, keys of
+    ``d`` and values of ``dv`` elements. ``src`` (rows or 32-bit planes): head h's queries at columns ``oq + (h // per) d``,
+    its keys at ``ok + (h // per) d``, its values at ``ov + h dv``; ``gates`` (rows or planes of the same dtype) the gates'
+    projections at columns ``og0 + h`` and ``og1 + h``. ``kind``:
+
+    * "mlstm": log gates i and f from ``cap tanh(. / cap)`` of the projections plus ``p0`` and ``p1``, under the running
+      maximum kept in ``m_state`` ([slots, H]); ``state`` [slots, H, dv + 1, d] holds the normaliser as its last row; ``nq``
+      and ``m_rows`` ([T, H]) receive n . q and the maxima. The maximum a sequence ends with is stored by ``scan_norm``.
+    * "mamba2": step sizes ``softplus(. + p0)``, decays ``exp(-exp(p1) dt)``, ``out`` gets ``p2[h] v`` on top; ``state``
+      [slots, H, dv, d].
+
+    Queries are multiplied by ``qscale``. ``out`` float32 [T, H dv]. ``chunked`` (bf16 rows, d up to 256): the form for long
+    prompts, whose sums differ from the token-by-token form's by rounding"""
+    _need_cuda(src, gates, p0, p1, p2, state, m_state, out, nq, m_rows)
+    n_planes, pstride, ld = _planes_of(src)
+    g_planes, gstride, ldg = _planes_of(gates)
+    rows = dv + (1 if kind == "mlstm" else 0)
+    assert src.dtype == gates.dtype and src.shape[-2] == gates.shape[-2] == out.shape[0]
+    for p in (p0, p1) + ((p2,) if kind == "mamba2" else ()):
+        assert p.dtype == torch.float32 and p.is_contiguous() and p.numel() == H
+    n_qk = -(-H // per)
+    assert src.shape[-1] >= max(oq + n_qk * d, ok + n_qk * d, ov + H * dv)
+    assert gates.shape[-1] >= max(og0 + H, og1 + H if kind == "mlstm" else 0)
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, rows, d)
+    assert out.dtype == torch.float32 and out.stride(1) == 1 and out.shape[1] == H * dv
+    if kind == "mlstm":
+        T = out.shape[0]
+        assert m_state.dtype == torch.float32 and m_state.shape[1:] == (H,) and m_state.is_contiguous()
+        assert nq.dtype == m_rows.dtype == torch.float32 and nq.shape == m_rows.shape == (T, H)
+        assert nq.is_contiguous() and m_rows.is_contiguous()
+    if d > 512:
+        raise KernelError("kindi_b200: a matrix state's keys have up to 512 elements, found %d" % d)
+    args = (SCAN_KIND[kind], dt(src), _p(src), n_planes, pstride, ld, oq, ok, ov, per, _p(gates), g_planes, gstride, ldg, og0,
+            og1, _p(p0), _p(p1), _p(p2), float(cap), float(qscale), B, H, d, dv, _p(q_start), _p(slot), _p(state),
+            state.stride(0), _p(m_state), m_state.stride(0) if m_state is not None else 0, _p(out), out.stride(0), _p(nq),
+            _p(m_rows))
+    if chunked:
+        T = out.shape[0]
+        runs = T // scan_run() + B
+        g = torch.empty((2, H, T), dtype=torch.float32, device=out.device)
+        part = torch.empty((runs, H, rows, d), dtype=torch.float32, device=out.device)
+        ends = torch.empty((runs, H), dtype=torch.float32, device=out.device)
+        _check(load().kb_gated_scan_chunked(*args, T, _p(g), _p(part), _p(ends), _stream()), "gated_scan_chunked")
+        add_launches(3)
+        return
+    _check(load().kb_gated_scan(*args, _stream()), "gated_scan")
+
+
+def scan_norm(kind: str, x: torch.Tensor, groups: int, w: torch.Tensor, eps: float, g: torch.Tensor, og: int,
+              nq: Optional[torch.Tensor], m_rows: Optional[torch.Tensor], m_state: Optional[torch.Tensor], pos, seq, slot,
+              q_start, out: torch.Tensor) -> None:
+    """the step after ``gated_scan``, per row and group of neighbouring elements (``w``: a gain per element of the row;
+    ``g``: rows or 32-bit planes, the gate's columns from ``og`` on):
+
+    * "mlstm": ``rms(x / (max(|nq|, exp(-m)) + 1e-6)) * w * sigmoid(g)``, a group is a head; stores the running maximum of a
+      sequence's last row in ``m_state``
+    * "mamba2": ``rms(x * silu(g)) * w``"""
+    _need_cuda(x, w, g, nq, m_rows, m_state, out)
+    T, N = x.shape
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and N % groups == 0 and out.shape == (T, N) and out.stride(1) == 1
+    assert w.dtype == torch.float32 and w.numel() == N and w.is_contiguous()
+    n_planes, pstride, ldg = _planes_of(g)
+    assert g.shape[-2] == T and g.shape[-1] >= og + N
+    _check(load().kb_scan_norm(SCAN_KIND[kind], _p(x), x.stride(0), T, groups, N // groups, _p(w), float(eps), _p(g), dt(g),
+                               n_planes, pstride, ldg, og, _p(nq), _p(m_rows), _p(m_state),
+                               m_state.stride(0) if m_state is not None else 0, _p(pos), _p(seq), _p(slot), _p(q_start),
+                               _p(out), dt(out), out.stride(0), _stream()), "scan_norm")
 
 
 def cast_rows(x: torch.Tensor, y: torch.Tensor) -> None:

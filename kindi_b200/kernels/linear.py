@@ -44,6 +44,14 @@ def rows_or_planes(ctx, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype
     return linear(ctx, a, w, out_dtype)
 
 
+def linear_bias_act(ctx, y: torch.Tensor, w: torch.Tensor, bias, act: str, out_dtype: torch.dtype) -> torch.Tensor:
+    """``act(y @ w^T + bias)`` (``[M, N]`` in out_dtype; ``bias`` float32 ``[N]`` or None): the product as rows or 32-bit
+    planes followed by one kernel"""
+    h = torch.empty((y.shape[0], w.shape[0]), dtype=out_dtype, device=y.device)
+    K.bias_act(rows_or_planes(ctx, y, w, out_dtype), bias, act, h)
+    return h
+
+
 # ----------------------------------------------------------------------------------------------- gate / up / SwiGLU
 GATE_UP_GROUP = 16      # rows of a gate group: a 32-column piece of a prompt-sized product's accumulator, the two
                         # half-warps of an epilogue warp of a decode-sized one

@@ -81,11 +81,14 @@ class Branch:
     in order, is the branch. ``scale`` (``[width]``, the norm gains' dtype; None for none): the sum is multiplied by it,
     column by column, before it joins the residual (a model's learned per-column scale of a sub-layer's output).
     ``bias`` (float32 ``[width]`` or None): counts once in the sum of the planes (an output projection's bias); a
-    consumer that adds planes only asks for ``with_bias_plane()``"""
+    consumer that adds planes only asks for ``with_bias_plane()``. ``norm`` (``(gains, eps)`` or None): the sum, bias
+    included, is divided by its root mean square and multiplied by the gains before it joins the residual (a model with a
+    norm on each sub-layer's output as well as on its input)"""
 
     parts: torch.Tensor
     scale: Optional[torch.Tensor] = None
     bias: Optional[torch.Tensor] = None
+    norm: Optional[Tuple[torch.Tensor, float]] = None
 
     def with_bias_plane(self) -> "Branch":
         """the same branch with the bias as one more plane (the branch itself when it has none)"""
@@ -93,7 +96,7 @@ class Branch:
             return self
         S, T, W = self.parts.shape
         plane = self.bias.to(torch.float32).view(1, 1, W).expand(1, T, W)
-        return Branch(torch.cat([self.parts, plane], dim=0), self.scale, None)
+        return Branch(torch.cat([self.parts, plane], dim=0), self.scale, None, self.norm)
 
 
 # ----------------------------------------------------------------------------- tensors by name

@@ -21,7 +21,8 @@ from .base import Block, Branch, StepContext, WeightView
 
 _DEFAULT_NAMES = {"norm1": "input_layernorm.", "mixer": "self_attn.", "norm2": "post_attention_layernorm.",
                   "feed_forward": "mlp."}
-_CATEGORY = {"norm1": "norm", "mixer": "mixer", "norm2": "norm", "feed_forward": "feed_forward"}
+_CATEGORY = {"norm1": "norm", "mixer": "mixer", "norm2": "norm", "feed_forward": "feed_forward", "norm1b": "norm",
+             "norm2b": "norm"}
 
 
 class PreNormBlock(Block):
@@ -36,7 +37,7 @@ class PreNormBlock(Block):
         """(role, sub-prefix) of the parts the block has: without a feed-forward there is no second norm either"""
         has_ff = spec.get("feed_forward") is not None
         return [(role, sub) for role, sub in cls._names(spec).items()
-                if has_ff or role not in ("norm2", "feed_forward")]
+                if has_ff or role not in ("norm2", "feed_forward", "norm2b")]
 
     @classmethod
     def _scales(cls, spec: PartSpec):
@@ -105,6 +106,51 @@ class PreNormBlock(Block):
 
     def bytes_read(self) -> int:
         return sum(p.bytes_read() for p in self._parts())
+
+
+class SandwichBlock(PreNormBlock):
+    """a norm before AND after every sub-layer: ``x += norm1b(mixer(norm1(x)))``, then ``x += norm2b(feed_forward(norm2(x)))``.
+    The norms on the outputs are RMS norms given as parts (``norm1b``, ``norm2b``; the block reads ``weight`` and ``eps`` of
+    them). They travel with the pending branch: the norm that reads the stream next applies them, adds, and normalises for
+    its own sub-layer in one kernel, so the block launches one norm kernel per sub-layer, as a pre-norm block does."""
+
+    @classmethod
+    def _names(cls, spec: PartSpec):
+        n = {"norm1": "norm1.", "mixer": "mixer.", "norm1b": "norm1b.", "norm2": "norm2.", "feed_forward": "mlp.",
+             "norm2b": "norm2b."}
+        n.update(spec.get("names") or {})
+        return n
+
+    def __init__(self, spec, width, weights: WeightView, *, dtype, device):
+        super().__init__(spec, width, weights, dtype=dtype, device=device)
+        if self.scale1 is not None or self.scale2 is not None:
+            raise ValueError("a block with norms on both sides has no learned scale per sub-layer")
+        names = self._names(spec)
+
+        def after(role):
+            ps: PartSpec = spec[role]
+            n = part_class("norm", ps.kind)(ps, width, weights.sub(names[role]), dtype=dtype, device=device)
+            if not (hasattr(n, "weight") and hasattr(n, "eps") and not hasattr(n, "bias")):
+                raise ValueError("the norm on a sub-layer's output is an RMS norm")
+            return n
+        self.norm1b = after("norm1b")
+        self.norm2b = after("norm2b") if self.feed_forward is not None else None
+
+    @staticmethod
+    def _normed(branch: Branch, norm) -> Branch:
+        if branch.scale is not None or branch.norm is not None:
+            raise NotImplementedError("a branch with a scale or a norm of its own inside a block with norms on both sides")
+        return Branch(branch.parts, None, branch.bias, (norm.weight, norm.eps))
+
+    def forward(self, ctx: StepContext, x, pending: Optional[Branch]) -> Optional[Branch]:
+        pending = self._normed(self.mixer.forward(ctx, self.norm1.add_norm(ctx, x, pending)), self.norm1b)
+        if self.feed_forward is None:
+            return pending
+        return self._normed(self.feed_forward.forward(ctx, self.norm2.add_norm(ctx, x, pending)), self.norm2b)
+
+    def _parts(self):
+        return super()._parts() + [p for p in (getattr(self, "norm1b", None), getattr(self, "norm2b", None))
+                                   if p is not None]
 
 
 class ParallelBlock(PreNormBlock):
@@ -176,8 +222,8 @@ class PostNormBlock(PreNormBlock):
     def forward(self, ctx: StepContext, x, pending: Optional[Branch]) -> Optional[Branch]:
         if pending is not None:
             # a block of another kind ran before: its branch joins the stream as it is
-            if pending.scale is not None:
-                raise NotImplementedError("a scaled pending branch in front of a post-norm block")
+            if pending.scale is not None or pending.norm is not None:
+                raise NotImplementedError("a scaled or normed pending branch in front of a post-norm block")
             K.residual_add(x, pending.with_bias_plane().parts, None)
         y = self._rows(ctx, x)
         y = self._add(ctx, x, self.mixer.forward(ctx, y), self.norm1, self.scale1)
@@ -190,3 +236,4 @@ class PostNormBlock(PreNormBlock):
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "postnorm", PostNormBlock)
 register_part("block", "parallel", ParallelBlock)
+register_part("block", "sandwich", SandwichBlock)

@@ -2,7 +2,7 @@
 over the whole projection), with a temperature on the queries, a gate per head, or two softmax maps per head that are
 subtracted ("differential" attention).
 
-``q, k, v = W y`` without biases, one product over the concatenated weights. Every query head and every key head is
+``q, k, v = W y``, one product over the concatenated weights. Every query head and every key head is
 divided by its root mean square over the head's ``head_dim`` elements (``head_norm``: ``{"eps", "when": "before" |
 "after" the rotation, "q", "k"}``; ``q`` / ``k`` name gains of size ``head_dim`` that all heads share, None for a
 unit norm). ``position`` is a rotation (``rotary`` with either pairing, partial rotation allowed) or ``none``.
@@ -16,6 +16,18 @@ Scores are ``scale (q . k)``, causal, softmax over all earlier positions; softma
   the same values. With ``lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff`` (one number for the layer) head h is
   ``o = a1 - lambda a2``, divided by its root mean square over the head's values (no gain) and multiplied by
   ``1 - diff``.
+
+* ``bias`` (how a bias is named after its projection, ``"%s.b"``): q, k and v have biases, added before everything else.
+* ``chunk``: a row sees the keys of its own chunk of that many positions, counted from the sequence's first one. The cache
+  then keeps the last ``cache_window`` positions (default: one chunk; more when other layers with larger chunks read this
+  layer's keys; "all": every position).
+* ``softcap``: scores pass ``s -> softcap tanh(s / softcap)`` before the softmax. With a unit norm after the rotation
+  ``|q . k|`` cannot exceed the head's size, which the kernels make use of.
+* ``null_score``: a fixed score without key or value that joins every head's softmax denominator (0: one is added to it).
+* ``shares_kv``: the layer has no key and value projections; its schedule entry names the cache entry whose keys and values
+  it attends to (``reads_cache_of``), as that entry stored them.
+* ``widen_heads``: heads of up to 128 elements are kept 64 or 128 wide in the cache, zero beyond their own size, so that the
+  tensor-core attention kernels take them.
 
 How it runs. An interleaved rotation (pairs ``(2i, 2i + 1)``) is turned into the rotate-half form the kernels know by
 permuting the rows of W_q and W_k inside every head, evens first: a score is a sum over the head's elements and does
@@ -60,7 +72,7 @@ class HeadNormAttention(Mixer):
         sizes)"""
         _, _, hd, vd = cls._sizes(spec)
         m = max(hd, vd)
-        if hd == vd and (hd % 8 == 0 or hd > 128):
+        if hd == vd and (hd % 8 == 0 or hd > 128) and not (spec.get("widen_heads") and m <= 128):
             return hd
         return 64 if m <= 64 else 128 if m <= 128 else (m + 7) // 8 * 8
 
@@ -75,8 +87,13 @@ class HeadNormAttention(Mixer):
         nh, nkv, hd, vd = cls._sizes(spec)
         maps = cls._maps(spec)
         n = cls._names(spec)
-        out = {n["q"]: (nh * maps * hd, width), n["k"]: (nkv * maps * hd, width), n["v"]: (nkv * vd, width),
-               n["o"]: (width, nh * vd)}
+        out = {n["q"]: (nh * maps * hd, width), n["o"]: (width, nh * vd)}
+        keys = ("q",)
+        if not spec.get("shares_kv"):
+            out.update({n["k"]: (nkv * maps * hd, width), n["v"]: (nkv * vd, width)})
+            keys = ("q", "k", "v")
+        if spec.get("bias"):
+            out.update({spec["bias"] % n[key]: (out[n[key]][0],) for key in keys})
         hn = spec.get("head_norm")
         if hn:
             for key in ("q", "k"):
@@ -98,7 +115,10 @@ class HeadNormAttention(Mixer):
     @classmethod
     def cache_need(cls, spec: PartSpec, width: int):
         _, nkv, _, _ = cls._sizes(spec)
-        return KVNeed(nkv * cls._maps(spec), cls._cache_dim(spec), None, 0)
+        chunk, kept = spec.get("chunk"), spec.get("cache_window")
+        # (the next position's chunk begins at most chunk - 1 positions before it)
+        kept = chunk if kept is None else None if kept == "all" else kept
+        return KVNeed(nkv * cls._maps(spec), cls._cache_dim(spec), int(kept) if kept else None, 0)
 
     def __init__(self, spec, width, weights: WeightView, *, dtype, device):
         super().__init__(spec, width, weights, dtype=dtype, device=device)
@@ -132,17 +152,30 @@ class HeadNormAttention(Mixer):
             w = w.view(n_heads, self.maps, self.qk_dim, width)
             return w if perm is None else w[:, :, perm.to(w.device)]
 
+        self.shares_kv = bool(spec.get("shares_kv"))
+        if self.shares_kv and (self.maps != 1 or spec.get("head_gate")):
+            raise NotImplementedError("differential attention or a gate per head on another layer's keys and values")
         wq = heads_of(weights(n["q"]), self.nh)                                 # [nh, maps, d, width]
-        wk = heads_of(weights(n["k"]), self.nkv)                                # [nkv, maps, d, width]
-        wv = weights(n["v"]).view(self.nkv, 1, self.v_dim, width)
         # query heads in the order (group, map, head of the group); key heads (group, map); values once per map
         wq = wq.view(self.nkv, self.group, self.maps, self.qk_dim, width).transpose(1, 2)
         wq = wq.reshape(self.nh * self.maps * self.qk_dim, width)
-        wk = wk.reshape(self.nkv * self.maps * self.qk_dim, width)
-        wv = wv.expand(self.nkv, self.maps, self.v_dim, width).reshape(self.nkv * self.maps * self.v_dim, width)
         self.nhq, self.nkvq = self.nh * self.maps, self.nkv * self.maps
-        ws = [_pad_heads(wq, self.nhq, self.qk_dim, hd), _pad_heads(wk, self.nkvq, self.qk_dim, hd),
-              _pad_heads(wv, self.nkvq, self.v_dim, hd)]
+        ws = [_pad_heads(wq, self.nhq, self.qk_dim, hd)]
+        if not self.shares_kv:
+            wk = heads_of(weights(n["k"]), self.nkv)                            # [nkv, maps, d, width]
+            wv = weights(n["v"]).view(self.nkv, 1, self.v_dim, width)
+            wk = wk.reshape(self.nkv * self.maps * self.qk_dim, width)
+            wv = wv.expand(self.nkv, self.maps, self.v_dim, width).reshape(self.nkv * self.maps * self.v_dim, width)
+            ws += [_pad_heads(wk, self.nkvq, self.qk_dim, hd), _pad_heads(wv, self.nkvq, self.v_dim, hd)]
+        self.b_main = None
+        if spec.get("bias"):
+            if self.maps != 1 or perm is not None:
+                raise NotImplementedError("biases with differential attention or an interleaved rotation")
+            bs = [(n["q"], self.nh, self.qk_dim)]
+            if not self.shares_kv:
+                bs += [(n["k"], self.nkv, self.qk_dim), (n["v"], self.nkv, self.v_dim)]
+            self.b_main = torch.cat([_pad_heads(weights(spec["bias"] % name).to(torch.float32), heads, d, hd)
+                                     for name, heads, d in bs]).contiguous()
         self.n_main = sum(w.shape[0] for w in ws)
         self.has_gate = bool(spec.get("head_gate"))
         if self.has_gate:
@@ -181,6 +214,17 @@ class HeadNormAttention(Mixer):
         self.t_coef, self.t_every = (float(qt["coef"]), int(qt["every"])) if qt else (0.0, 1)
         if qt and self.t_every < 1:
             raise ValueError("q_temp.every must be at least 1, found %d" % self.t_every)
+        # ---- what a row sees and how scores enter the softmax
+        self.chunk = int(spec.get("chunk") or 0)
+        if self.chunk < 0:
+            raise ValueError("a chunk must hold at least one position, found %d" % self.chunk)
+        self.cap = None
+        if spec.get("softcap"):
+            unit = self.norm_when == "after" and self.gq is None
+            self.cap = A.ScoreCap(float(spec["softcap"]), self.scale, float(self.qk_dim) if unit else None)
+        self.sink = None
+        if spec.get("null_score") is not None:
+            self.sink = torch.full((self.nhq,), float(spec["null_score"]), dtype=torch.float32, device=device)
         # ---- differential attention's constants
         d = spec.get("differential")
         self.diff = None
@@ -193,15 +237,19 @@ class HeadNormAttention(Mixer):
     def forward(self, ctx: StepContext, y: torch.Tensor) -> Branch:
         nhq, nkvq, hd = self.nhq, self.nkvq, self.hd
         n_q = nhq * hd
+        if self.shares_kv != (ctx.entry.reads_cache_of is not None):
+            raise ValueError("a layer reads another entry's keys and values exactly when it has no projections of its own")
         qkv = L.rows_or_planes(ctx, y, self.wqkv, self.dtype)
-        pool, table, n_pages = ctx.cache.kv_view(ctx.entry.cache)
+        pool, table, n_pages = ctx.cache.kv_view(ctx.entry.reads_cache_of if self.shares_kv else ctx.entry.cache)
+        own = 0 if self.shares_kv else nkvq
         q = qkv if qkv.dim() == 2 else torch.empty((ctx.T, n_q), dtype=self.dtype, device=y.device)
         K.headnorm_rope_store(qkv[..., :self.n_main], q, self.gq, self.gk, self.norm_eps, self.qk_dim, self.norm_when,
                               self.inv_freq, self.inv_freq64, self.rot, self.t_coef, self.t_every, ctx.pos, ctx.seq,
-                              ctx.slot, nhq, nkvq, nkvq, hd, pool, table, n_pages, ctx.status)
+                              ctx.slot, nhq, own, own, hd, pool if own else None, table, n_pages, ctx.status,
+                              bias=self.b_main)
         att = torch.empty((ctx.T, n_q), dtype=self.dtype, device=y.device)
         A.attention(ctx, q[:, :n_q] if q.shape[1] != n_q else q, att, nhq, nkvq, hd, self.scale, 0, pool, table,
-                    n_pages)
+                    n_pages, sink=self.sink, chunk=self.chunk, cap=self.cap)
         if self.diff is not None:
             lam, eps, mult = self.diff
             out = torch.empty((ctx.T, self.nh * hd), dtype=self.dtype, device=y.device)

@@ -56,4 +56,53 @@ class SwiGLU(FeedForward):
         return sum(w.numel() * w.element_size() for w in (self.wgu, self.wd))
 
 
+class DenseMLP(FeedForward):
+    """a feed-forward without a gate: ``W_down act(W_up y + b_up) + b_down``. ``activation`` (``relu2``: the square of relu,
+    ``silu`` or ``gelu_tanh``), whether the projections have biases (``bias``), the intermediate size and the tensors' suffixes
+    (``names``: ``up``, ``down``; ``bias_name``: how a bias is named after its projection, ``"%s.b"``) are parameters of the
+    part."""
+
+    @classmethod
+    def _names(cls, spec: PartSpec):
+        n = {"up": "up", "down": "down"}
+        n.update(spec.get("names") or {})
+        return n
+
+    @classmethod
+    def _bias_names(cls, spec: PartSpec):
+        n, how = cls._names(spec), spec.get("bias_name") or "%s.b"
+        return how % n["up"], how % n["down"]
+
+    @classmethod
+    def tensor_shapes(cls, spec: PartSpec, width: int) -> Dict[str, Tuple[int, ...]]:
+        f = int(spec["intermediate"])
+        n = cls._names(spec)
+        out = {n["up"]: (f, width), n["down"]: (width, f)}
+        if spec.get("bias"):
+            up, down = cls._bias_names(spec)
+            out.update({up: (f,), down: (width,)})
+        return out
+
+    def __init__(self, spec, width, weights: WeightView, *, dtype, device):
+        super().__init__(spec, width, weights, dtype=dtype, device=device)
+        self.act = str(spec.get("activation") or "relu2")
+        if self.act not in ("relu2", "silu", "gelu_tanh"):
+            raise ValueError("a feed-forward's activation is relu2, silu or gelu_tanh, found %r" % self.act)
+        n = self._names(spec)
+        self.wu, self.wd = weights(n["up"]), weights(n["down"])
+        self.bu = self.bd = None
+        if spec.get("bias"):
+            up, down = self._bias_names(spec)
+            self.bu = weights(up).to(torch.float32).contiguous()
+            self.bd = weights(down).to(torch.float32).contiguous()
+
+    def forward(self, ctx: StepContext, y: torch.Tensor) -> Branch:
+        h = L.linear_bias_act(ctx, y, self.wu, self.bu, self.act, self.dtype)
+        return Branch(L.planes(ctx, h, self.wd), bias=self.bd)
+
+    def bytes_read(self) -> int:
+        return sum(w.numel() * w.element_size() for w in (self.wu, self.wd))
+
+
 register_part("feed_forward", "swiglu", SwiGLU)
+register_part("feed_forward", "dense", DenseMLP)

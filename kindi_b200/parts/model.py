@@ -88,6 +88,9 @@ class DecoderModel:
                                                 for e in self.spec.schedule) else None
         pending: Optional[Branch] = None
         for entry in self.spec.schedule:
+            if pending is not None and pending.norm is not None and (entry.mix_embedding is not None or entry.add_embedding):
+                raise NotImplementedError("a branch with a norm of its own cannot be pending where the embedding comes in "
+                                          "again")
             if entry.mix_embedding is not None:
                 # x <- W [x + pending branch; x0]: one row of both, then the product with 32-bit output
                 both = torch.empty((ctx.T, 2 * self.spec.width), dtype=self.dtype, device=x.device)

@@ -41,6 +41,18 @@ class RMSNorm(Norm):
     def add_norm(self, ctx: StepContext, x, pending: Optional[Branch], rows=None):
         n_out = x.shape[0] if rows is None else rows.numel()
         y = torch.empty((n_out, self.width), dtype=self.dtype, device=x.device)
+        if pending is not None and pending.norm is not None:
+            # the branch's own norm, the add and this norm in one pass over the row
+            if pending.scale is not None:
+                raise NotImplementedError("a branch with a norm of its own and a scale")
+            w1, eps1 = pending.norm
+            if w1.dtype != self.weight.dtype:
+                w1 = w1.to(self.weight.dtype)
+            K.norm_add_norm(x, pending.parts, pending.bias, w1, eps1, self.weight, self.eps, y, rows,
+                            write_back=rows is None, status=ctx.status)
+            return y
+        if pending is not None:
+            pending = pending.with_bias_plane()
         scale = None if pending is None else pending.scale
         if scale is not None and scale.dtype != self.weight.dtype:
             scale = scale.to(self.weight.dtype)
@@ -81,8 +93,11 @@ class LayerNorm(Norm):
 
     def add_norm(self, ctx: StepContext, x, pending: Optional[Branch], rows=None):
         n_out = x.shape[0] if rows is None else rows.numel()
-        if pending is not None and pending.scale is not None:
-            raise NotImplementedError("the layer norm kernel adds a branch as it is; a scaled branch needs the RMS norm")
+        if pending is not None and (pending.scale is not None or pending.norm is not None):
+            raise NotImplementedError("the layer norm kernel adds a branch as it is; a scaled or normed branch needs the "
+                                      "RMS norm")
+        if pending is not None:
+            pending = pending.with_bias_plane()
         y = torch.empty((n_out, self.width), dtype=self.dtype, device=x.device)
         K.add_layernorm(x, None if pending is None else pending.parts, self.weight, self.bias, self.eps, y, rows,
                         write_back=rows is None and pending is not None, status=ctx.status)
