@@ -550,6 +550,67 @@ def bench_luzerax(a) -> int:
     return 0
 
 
+# ---------------------------------------------------------------------------------------------- --arch zebovik
+# Layer sizes that resemble real models' (random weights, four layers: chunked attention, chunked attention on the first
+# layer's keys and values, matrix memory, state-space duality; each with a feed-forward without a gate), each beside the
+# Nilatar design (the closest one: windowed attention, a layer that reads another's keys and values, a recurrent layer with
+# a matrix state) of the same width, heads, head size, matrix states (heads x 128 x 128), span of the attention layers and
+# feed-forward weights (two matrices of one and a half times the inner size of Nilatar's three).
+ZEBOVIK_CONV = 4
+
+
+def zebovik_config(sz: dict):
+    """a Zebovik config.json object at the sizes of NILATAR_SIZES[.]"""
+    H, hd = sz["heads"], NILATAR_HEAD
+    mlp = {"kind": "dense", "ff": sz["ff"] * 3 // 2 // 64 * 64}
+    att = {"heads": H, "kv_heads": sz["kv"], "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0,
+           "rot": {"base": 500000.0, "dims": hd}, "mask": {"size": NILATAR_WINDOW}}
+    mem = {"heads": H, "dim": hd, "vdim": hd, "gate_cap": 15.0}
+    ssd = {"heads": 2 * H, "vdim": hd // 2, "state": hd, "groups": max(1, H // 4), "conv": ZEBOVIK_CONV,
+           "norm_groups": max(1, H // 4)}
+    return {"architecture": "Zebovik", "vocab": NILATAR_VOCAB, "width": sz["width"], "norm": {"eps": 1e-5},
+            "logit_softcap": 30.0,
+            "layers": [{"type": "attention", "mixer": att, "mlp": mlp},
+                       {"type": "attention", "mixer": dict(att, kv_from=0), "mlp": mlp},
+                       {"type": "mlstm", "mixer": mem, "mlp": mlp}, {"type": "mamba2", "mixer": ssd, "mlp": mlp}]}
+
+
+def bench_zebovik(a) -> int:
+    """prefill and decode throughput of the Zebovik design at three layer sizes, each beside the Nilatar design of equal
+    size, with the device time per kind of launch"""
+    import torch
+    pk = peaks()
+    batch, context, tokens = a.batch, min(a.context, 4096), a.prefill_tokens
+    sizes = [x for x in (a.sizes or "s,m,l").split(",") if x in NILATAR_SIZES]
+    rows = {}
+    for name in sizes:
+        sz = NILATAR_SIZES[name]
+        zeb, (nil, _) = zebovik_config(sz), nilatar_pair(sz)
+        ctx = batch * (context + a.steps + a.warmup + 320) + tokens + 64
+        row = {"sizes": dict(width=sz["width"], heads=sz["heads"], kv=sz["kv"], head=NILATAR_HEAD, layers=4,
+                             span=NILATAR_WINDOW, ff=zeb["layers"][0]["mlp"]["ff"], nilatar_ff=sz["ff"],
+                             mlstm=zeb["layers"][2]["mixer"], mamba2=zeb["layers"][3]["mixer"])}
+        for what, cfg in (("zebovik", zeb), ("nilatar", nil)):
+            eng = engine_from_config(cfg, ctx, batch)
+            for g in eng.cache.groups:
+                g.pool.normal_(0.0, 1.0)
+            dev_ms, _, launches, _ = bench_decode(eng, batch, context, a.steps, max(3, a.warmup), False)
+            pms = bench_prefill(eng, 3, 5, tokens)
+            kt = kernel_times(eng, batch, context, tokens)
+            row[what] = {"decode_ms": round(dev_ms, 4), "decode_tokens_per_s": round(batch * 1000.0 / dev_ms, 1),
+                         "launches_per_step": launches // a.steps, "prefill_ms": round(pms, 3),
+                         "prefill_tokens_per_s": round(tokens * 1000.0 / pms, 1),
+                         "kernels_us": {k: _grouped(v) for k, v in kt.items()}}
+            del eng
+            torch.cuda.empty_cache()
+        rows[name] = row
+    print(json.dumps({"arch": "zebovik", "what": "prefill and decode of the Zebovik design beside the Nilatar design of "
+                      "equal size (random weights, 4 layers); not the default benchmark",
+                      "batch": batch, "context": context, "prefill_tokens": tokens, "steps": a.steps, "dtype": "bf16",
+                      "peaks": pk, "sizes": rows}))
+    return 0
+
+
 def kernel_times(eng, batch: int, context: int, prefill_tokens: int):
     """device time per kind of launch: one decode step of `batch` sequences at `context` and one prompt pass, each
     issued launch by launch (no recorded graph, launches strictly one after another) with CUDA events around every
@@ -781,11 +842,11 @@ def main(argv=None) -> int:
                          "0.7, top-p 0.8, top-k 20) and report it as e2e_sampled")
     ap.add_argument("--no-pdl", action="store_true", help="launch kernels strictly one after another")
     ap.add_argument("--prefill-only", action="store_true", help="measure only the prefill (for profiling)")
-    ap.add_argument("--arch", default="nanbeige", choices=("nanbeige", "vozinex", "nilatar", "medodra", "luzerax"),
-                    help="vozinex, nilatar, medodra, luzerax: not the default benchmark but that design at a few layer sizes, "
+    ap.add_argument("--arch", default="nanbeige", choices=("nanbeige", "vozinex", "nilatar", "medodra", "luzerax", "zebovik"),
+                    help="vozinex, nilatar, medodra, luzerax, zebovik: not the default benchmark but that design at a few layer sizes, "
                          "each beside the closest other decoder of equal size (prefill, decode, device time per kind "
                          "of launch)")
-    ap.add_argument("--sizes", default="", help="with --arch vozinex, nilatar, medodra or luzerax: which of s,m,l (default: all)")
+    ap.add_argument("--sizes", default="", help="with --arch vozinex, nilatar, medodra, luzerax or zebovik: which of s,m,l (default: all)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="prompt length of --prefill-only (the full run always measures 2048 tokens)")
     a = ap.parse_args(argv)
@@ -816,6 +877,8 @@ def main(argv=None) -> int:
         return bench_medodra(a)
     if a.arch == "luzerax" and a.gpus == 1:
         return bench_luzerax(a)
+    if a.arch == "zebovik" and a.gpus == 1:
+        return bench_zebovik(a)
     if a.gpus != 1:
         print("kindi_b200 is a one-GPU library: bench.py measures N=1 only (asked for --gpus %d)" % a.gpus)
         return 2

@@ -206,6 +206,8 @@ class KernelTiming:
             if name in _GEMM_NK:
                 n, k = _GEMM_NK[name]
                 label += " %dx%d" % ((2 * args[n], args[k]) if name == "kb_gemm_swiglu_decode" else (args[n], args[k]))
+            elif name in ("kb_gated_scan", "kb_gated_scan_chunked", "kb_scan_norm"):
+                label += "_" + ("mlstm", "mamba2")[args[0]]
             e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
             e0.record()
             rc = fn(*args)
