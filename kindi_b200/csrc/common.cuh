@@ -84,10 +84,46 @@ __device__ __forceinline__ float kb_gate_act_fast(float g, int act) {
 // the gated unit a product finishes in its epilogue: which activation, and for the clamped unit its two constants.
 // KB_ACT_GLU_CLAMP: g' sigmoid(alpha g') (u' + 1) with g' = min(g, lim), u' = clamp(u, -lim, lim)
 #define KB_ACT_GLU_CLAMP 4
+// A product without a gated unit may finish its rows instead: out = act(v + bias), `post` the activation's code (-1: the
+// rows leave as they are) and `bias` a float per output column (null: none).
 struct KbGate {
     int act;
     float lim, alpha;
+    int post;
+    const float* bias;
 };
+__device__ __forceinline__ float kb_post_act(float z, int post) {
+    if (post == KB_ACT_RELU2) {
+        const float r = fmaxf(z, 0.0f);
+        return r * r;
+    }
+    return post == KB_ACT_NONE ? z : kb_gate_act_fast(z, post);
+}
+// the biases of 32 neighbouring columns, all loads in flight (columns from n_cols on: zero)
+__device__ __forceinline__ void kb_post_bias32(float (&b)[32], int col, int n_cols, const KbGate& k) {
+    if (k.bias != nullptr && col + 32 <= n_cols && (((uintptr_t)(k.bias + col)) & 15) == 0) {
+#pragma unroll
+        for (int c = 0; c < 32; c += 4) {
+            const float4 v = __ldg((const float4*)(k.bias + col + c));
+            b[c] = v.x; b[c + 1] = v.y; b[c + 2] = v.z; b[c + 3] = v.w;
+        }
+        return;
+    }
+#pragma unroll
+    for (int c = 0; c < 32; c++) b[c] = k.bias != nullptr && col + c < n_cols ? __ldg(k.bias + col + c) : 0.0f;
+}
+__device__ __forceinline__ void kb_post32(uint32_t (&r)[32], const float (&b)[32], int post) {
+    if (post == KB_ACT_RELU2) {
+#pragma unroll
+        for (int c = 0; c < 32; c++) {
+            const float z = fmaxf(__uint_as_float(r[c]) + b[c], 0.0f);
+            r[c] = __float_as_uint(z * z);
+        }
+        return;
+    }
+#pragma unroll
+    for (int c = 0; c < 32; c++) r[c] = __float_as_uint(kb_post_act(__uint_as_float(r[c]) + b[c], post));
+}
 __device__ __forceinline__ float kb_glu_fast(float g, float u, const KbGate& k) {
     if (k.act == KB_ACT_GLU_CLAMP) {
         g = fminf(g, k.lim);
@@ -102,6 +138,8 @@ static inline KbGate kb_gate_of(int act, float lim, float alpha) {
     k.act = act == KB_ACT_GELU_TANH ? KB_ACT_GELU_TANH : act == KB_ACT_GLU_CLAMP ? KB_ACT_GLU_CLAMP : KB_ACT_SILU;
     k.lim = lim;
     k.alpha = alpha;
+    k.post = -1;
+    k.bias = nullptr;
     return k;
 }
 

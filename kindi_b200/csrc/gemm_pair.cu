@@ -330,6 +330,11 @@ __global__ void __launch_bounds__(GP_THREADS) k_gemm_pair(const __grid_constant_
 #pragma unroll
                         for (int half = 0; half < 2; half++) {
                             if (half == 1) load32(c0 + 32, r);
+                            if (gate_act.post >= 0) {                    // the row leaves finished: bias and activation
+                                float pb[32];
+                                kb_post_bias32(pb, q0 + c0 + half * 32, N, gate_act);
+                                kb_post32(r, pb, gate_act.post);
+                            }
 #pragma unroll
                             for (int j = 0; j < 4; j++) {
                                 uint32_t h[4];
@@ -436,13 +441,17 @@ static int launch_pair(const CUtensorMap& ma, const CUtensorMap& mw, void* C, in
 // lowers what it raised) are the scratch of tiles shared by two pairs; without them the work is cut tile by tile.
 extern "C" int kb_gemm_pair(const void* A, const void* W, void* C, int cdtype, int M, int N, int K, int lda, int ldw,
                             int ldc, int bn, int* status, cudaStream_t st, int swiglu, float* part, int* flags,
-                            float act_lim = 0.0f, float act_alpha = 0.0f) {
+                            float act_lim = 0.0f, float act_alpha = 0.0f, const float* bias = nullptr, int post = -1) {
+    // post >= 0 (bf16 out, no swiglu): C = act(. + bias), post the activation's code, bias float [N] or null
+    if (post >= 0 && (swiglu || cdtype != KB_BF16)) return (int)cudaErrorInvalidValue;
     if (swiglu && ((N % 32) || cdtype != KB_BF16 || (ldc % 8) || ((uintptr_t)C & 15))) return (int)cudaErrorInvalidValue;
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     if ((K % 8) || (lda % 8) || (ldw % 8)) return (int)cudaErrorInvalidValue;
     if (cdtype != KB_F32 && cdtype != KB_BF16) return (int)cudaErrorInvalidValue;
     const int swiglu_ld = swiglu ? ldc : 0;
-    const KbGate gate_act = kb_gate_of(swiglu, act_lim, act_alpha);
+    KbGate gate_act = kb_gate_of(swiglu, act_lim, act_alpha);
+    gate_act.post = post;
+    gate_act.bias = bias;
     CUtensorMap ma, mw;
     int rc;
     if ((rc = kb_make_map_bf16(&ma, A, M, K, lda, GP_BM))) return rc;

@@ -233,6 +233,11 @@ __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ 
                                 tmem_ld_32x32(tbase + c0 + 32, r);       // (columns past the accumulator are never stored)
                                 tmem_ld_wait();
                             }
+                            if (gate_act.post >= 0) {                    // the row leaves finished: bias and activation
+                                float pb[32];
+                                kb_post_bias32(pb, q0 + c0 + half * 32, rowsQ, gate_act);
+                                kb_post32(r, pb, gate_act.post);
+                            }
 #pragma unroll
                             for (int j = 0; j < 4; j++) {
                                 uint32_t h[4];
@@ -274,6 +279,12 @@ __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ 
                 uint32_t r[16];
                 tmem_ld_32x16(tbase + c0, r);
                 tmem_ld_wait();
+                if (sizeof(TC) == 2 && gate_act.post >= 0 && prow < rowsP) {
+                    const float pb = gate_act.bias ? __ldg(gate_act.bias + prow) : 0.0f;
+#pragma unroll
+                    for (int c = 0; c < 16; c++)
+                        r[c] = __float_as_uint(kb_post_act(__uint_as_float(r[c]) + pb, gate_act.post));
+                }
                 if (prow < rowsP) {
 #pragma unroll
                     for (int c = 0; c < 16; c++)
@@ -583,12 +594,17 @@ extern "C" int kb_gemm_tc_splits(int K, int wanted) {
 // the bf16 [M][N / 2] result silu(gate) * up with row stride ldc.
 extern "C" int kb_gemm_tc(const void* A, const void* W, void* C, int cdtype, int M, int N, int K, int lda, int ldw,
                           int ldc, int swap, int bn, int splits, long long split_stride, int* status,
-                          cudaStream_t st, int swiglu = 0, int mt = 1, float act_lim = 0.0f, float act_alpha = 0.0f) {
+                          cudaStream_t st, int swiglu = 0, int mt = 1, float act_lim = 0.0f, float act_alpha = 0.0f,
+                          const float* bias = nullptr, int post = -1) {
+    // post >= 0 (bf16 out, no swiglu): C = act(. + bias), post the activation's code, bias float [N] or null
     if (mt != 1 && (mt != 2 || swap || splits != 1)) return (int)cudaErrorInvalidValue;
     if (swiglu && (swap || (N % 32) || cdtype != KB_BF16 || splits != 1 || (ldc % 8) || ((uintptr_t)C & 15)))
         return (int)cudaErrorInvalidValue;
+    if (post >= 0 && (swiglu || cdtype != KB_BF16 || splits != 1)) return (int)cudaErrorInvalidValue;
     const int swiglu_ld = swiglu ? ldc : 0;
-    const KbGate gate_act = kb_gate_of(swiglu, act_lim, act_alpha);
+    KbGate gate_act = kb_gate_of(swiglu, act_lim, act_alpha);
+    gate_act.post = post;
+    gate_act.bias = bias;
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     if ((K % 8) || (lda % 8) || (ldw % 8)) return (int)cudaErrorInvalidValue;
     if (splits > 1 && cdtype != KB_F32) return (int)cudaErrorInvalidValue;

@@ -23,6 +23,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *(uint32_t*)&v;
 }
 
+// 16 bytes from global to shared memory without a register in between; ok == false: zeros
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
 // x = s[0] + s[1] + s[2] up to 2^-24 of x: a product with a 32-bit operand is the sum of three bf16 products
 #define KB_SPLIT 3
 __device__ __forceinline__ void split_bf16(float x, bf16 (&s)[KB_SPLIT]) {

@@ -162,6 +162,99 @@ __global__ void __launch_bounds__(128) k_short_conv(const TIN* KB_STEP_DATA in, 
 #undef SC_U
 }
 
+// The same for prompt-sized steps of bf16 rows (16-byte aligned, channels a multiple of eight): a thread works eight
+// neighbouring channels of SC_ROWS consecutive rows, every input row loaded once. Rows whose taps reach before the step
+// (a sequence's first taps - 1 rows) and the new tails are worked by the thread that meets the sequence's first row, as
+// above.
+#define SC_ROWS 8
+template <int TAPS>
+__global__ void __launch_bounds__(128) k_short_conv_rows(const bf16* KB_STEP_DATA in, int ld_in, int col0, int C,
+        const float* __restrict__ bias, const float* __restrict__ w, int act, float* state, size_t state_stride,
+        const int* __restrict__ pos, const int* __restrict__ seq, const int* __restrict__ slot,
+        const int* __restrict__ q_start, bf16* __restrict__ out, int ldo, const float* __restrict__ obias, int T) {
+    kb_pdl_launch();
+    const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
+    const int t0 = blockIdx.x * SC_ROWS;
+    if (c >= C) {
+        kb_pdl_wait();
+        return;
+    }
+    // weights (8 TAPS neighbouring floats), and where each row stands in its sequence's share of the step: all in flight
+    float wr[8 * TAPS];
+#pragma unroll
+    for (int k = 0; k < 2 * TAPS; k++) *(float4*)&wr[4 * k] = *(const float4*)(w + (size_t)c * TAPS + 4 * k);
+    int ix[SC_ROWS], sq[SC_ROWS];
+#pragma unroll
+    for (int r = 0; r < SC_ROWS; r++) {
+        const int t = t0 + r;
+        sq[r] = t < T && pos[t] >= 0 ? seq[t] : -1;
+    }
+#pragma unroll
+    for (int r = 0; r < SC_ROWS; r++) ix[r] = sq[r] >= 0 ? t0 + r - q_start[sq[r]] : -1;
+    float bs[8], ob[8];
+#pragma unroll
+    for (int e = 0; e < 8; e++) {
+        bs[e] = bias ? bias[c + e] : 0.0f;
+        ob[e] = obias ? obias[c + e] : 0.0f;
+    }
+    kb_pdl_wait();
+    uint4 rows[SC_ROWS + TAPS - 1];                    // input rows t0 - (TAPS - 1) .. t0 + SC_ROWS - 1
+#pragma unroll
+    for (int k = 0; k < SC_ROWS + TAPS - 1; k++) {
+        const int t = t0 - (TAPS - 1) + k;
+        rows[k] = make_uint4(0, 0, 0, 0);
+        if (t >= 0 && t < T) rows[k] = *(const uint4*)(in + (size_t)t * ld_in + col0 + c);
+    }
+#pragma unroll
+    for (int r = 0; r < SC_ROWS; r++) {
+        if (ix[r] < TAPS - 1) continue;
+        float acc[8];
+#pragma unroll
+        for (int e = 0; e < 8; e++) acc[e] = ob[e];
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) {
+            const bf16* x = (const bf16*)&rows[r + j];
+#pragma unroll
+            for (int e = 0; e < 8; e++) acc[e] = fmaf(wr[e * TAPS + j], __bfloat162float(x[e]) + bs[e], acc[e]);
+        }
+        uint32_t h[4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            const float x = act ? rc_silu(acc[2 * e]) : acc[2 * e], y = act ? rc_silu(acc[2 * e + 1]) : acc[2 * e + 1];
+            __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+            h[e] = *(uint32_t*)&v;
+        }
+        *(uint4*)(out + (size_t)(t0 + r) * ldo + c) = make_uint4(h[0], h[1], h[2], h[3]);
+    }
+    if (TAPS == 1) return;
+    // a sequence's first rows and its new tails, channel by channel (rare: once per sequence and step)
+#pragma unroll 1
+    for (int r = 0; r < SC_ROWS; r++) {
+        const int t = t0 + r;
+        if (t >= T || pos[t] < 0) continue;
+        const int b = seq[t], r0 = q_start[b];
+        if (t != r0) continue;
+        const int n = q_start[b + 1] - r0;
+#pragma unroll 1
+        for (int e = 0; e < 8; e++) {
+            float* tails = state + (size_t)slot[b] * state_stride + c + e;
+            const bf16* x = in + (size_t)r0 * ld_in + col0 + c + e;
+            const float bse = bias ? bias[c + e] : 0.0f, obe = obias ? obias[c + e] : 0.0f;
+            // input i of the step; negative: an old tail
+            auto u = [&](int i) {
+                return i >= 0 ? __bfloat162float(x[(size_t)i * ld_in]) + bse : tails[(size_t)(TAPS - 1 + i) * C];
+            };
+            for (int i = 0; i < min(n, TAPS - 1); i++) {
+                float acc = obe;
+                for (int j = 0; j < TAPS; j++) acc = fmaf(w[(size_t)(c + e) * TAPS + j], u(i - (TAPS - 1) + j), acc);
+                out[(size_t)(r0 + i) * ldo + c + e] = __float2bfloat16_rn(act ? rc_silu(acc) : acc);
+            }
+            // (in ascending order: an old tail that moves is read before its place is written)
+            for (int k = 0; k < TAPS - 1; k++) tails[(size_t)k * C] = u(n - (TAPS - 1) + k);
+        }
+    }
+}
+
 extern "C" int kb_short_conv(const void* in, int idtype, int n_planes, long long plane_stride, int ld_in, int col0,
                              int C, const float* bias, const float* w, int taps, int act, float* state,
                              long long state_stride, const int* pos, const int* seq, const int* slot,
@@ -170,6 +263,21 @@ extern "C" int kb_short_conv(const void* in, int idtype, int n_planes, long long
     // bias (float [C] or null) joins every input, obias every result (before the activation)
     if (T <= 0 || C <= 0) return 0;
     if (taps < 1 || taps > SC_MAX_TAPS) return (int)cudaErrorInvalidValue;
+    if (idtype == KB_BF16 && odtype == KB_BF16 && n_planes == 1 && T >= 256 && taps <= 4 && C % 8 == 0 && col0 % 8 == 0 &&
+        ld_in % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)in % 16) == 0 && ((uintptr_t)out % 16) == 0) {
+        const dim3 gridr((T + SC_ROWS - 1) / SC_ROWS, (C / 8 + 127) / 128);
+#define KB_SCR(TAPS)                                                                                                  \
+    kb_launch(k_short_conv_rows<TAPS>, gridr, 128, 0, st, (const bf16*)in, ld_in, col0, C, bias, w, act, state,        \
+              (size_t)state_stride, pos, seq, slot, q_start, (bf16*)out, ldo, obias, T)
+        switch (taps) {
+            case 1: KB_SCR(1); break;
+            case 2: KB_SCR(2); break;
+            case 3: KB_SCR(3); break;
+            default: KB_SCR(4); break;
+        }
+#undef KB_SCR
+        KB_LAUNCH_RET();
+    }
     dim3 grid(T, (C + 127) / 128);
 #define KB_SC(TIN, TO)                                                                                              \
     kb_launch(k_short_conv<TIN, TO>, grid, 128, 0, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in, col0, \

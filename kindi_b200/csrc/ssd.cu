@@ -185,10 +185,11 @@ __global__ void __launch_bounds__(32 * SS_COLS) k_gated_scan(SsArgs a) {
 
 // ------------------------------------------------------------------------------------------------ gates of long prompts
 // ld [H][T]: log a; w [H][T]. The running maxima are the scan of the maps m -> max(F + m, M), a token's being (f, i):
-// (F1, M1) then (F2, M2) is (F1 + F2, max(F2 + M1, M2)). A block per (head, sequence), 256 tokens at a time.
+// (F1, M1) then (F2, M2) is (F1 + F2, max(F2 + M1, M2)). A block per (head, sequence), SG_T tokens at a time.
+#define SG_T 1024
 template <typename T, int MODE>
-__global__ void __launch_bounds__(256) k_scan_gates(SsArgs a, float* __restrict__ ld, float* __restrict__ w, int Tn) {
-    __shared__ float sF[8], sM[8], s_prev[257];
+__global__ void __launch_bounds__(SG_T) k_scan_gates(SsArgs a, float* __restrict__ ld, float* __restrict__ w, int Tn) {
+    __shared__ float sF[SG_T / 32], sM[SG_T / 32], s_prev[SG_T + 1];
     kb_pdl_launch();
     const int h = blockIdx.x, b = blockIdx.y;
     const int r0 = a.q_start[b], r1 = a.q_start[b + 1];
@@ -197,7 +198,7 @@ __global__ void __launch_bounds__(256) k_scan_gates(SsArgs a, float* __restrict_
     float* ldh = ld + (size_t)h * Tn, *wh = w + (size_t)h * Tn;
     if (MODE == SS_MAMBA) {
         // (no order among the tokens: gridDim.z blocks share them)
-        for (int t = r0 + blockIdx.z * 256 + threadIdx.x; t < r1; t += 256 * gridDim.z) {
+        for (int t = r0 + blockIdx.z * blockDim.x + threadIdx.x; t < r1; t += blockDim.x * gridDim.z) {
             float dt, l;
             ss_gate<T, MODE>(a, t, h, dt, l);
             ldh[t] = l;
@@ -206,7 +207,7 @@ __global__ void __launch_bounds__(256) k_scan_gates(SsArgs a, float* __restrict_
         return;
     }
     float m_in = a.m_state[(size_t)a.slot[b] * a.m_stride + h];
-    for (int c0 = r0; c0 < r1; c0 += 256) {
+    for (int c0 = r0; c0 < r1; c0 += SG_T) {
         const int t = c0 + threadIdx.x;
         float i = -INFINITY, f = 0.0f;
         if (t < r1) ss_gate<T, MODE>(a, t, h, i, f);
@@ -235,7 +236,7 @@ __global__ void __launch_bounds__(256) k_scan_gates(SsArgs a, float* __restrict_
             wh[t] = expf(i - m);
             a.m_rows[(size_t)t * a.H + h] = m;
         }
-        m_in = s_prev[256];                            // (only read when there is another tile, which this one fills)
+        m_in = s_prev[SG_T];                            // (only read when there is another tile, which this one fills)
         __syncthreads();
     }
 }
@@ -265,15 +266,15 @@ __device__ __forceinline__ SsRun ss_run(const SsArgs& a, int run) {
     r.n = max(0, min(SS_C, a.q_start[lo + 1] - r.r0));
     return r;
 }
-// rows of bf16 from global into a padded tile [SS_C][dst_ld]; columns from d to dp and rows from n on are zero
+// rows of bf16 from global into a padded tile [SS_C][dst_ld]; columns from d to dp and rows from n on are zero. Whole 16-byte
+// words go by asynchronous copies: the caller waits for them (cp_async_wait_all) before its barrier
 __device__ __forceinline__ void ss_tile(bf16* dst, int dst_ld, const bf16* src, int ld, int n, int d, int dp, bool vec) {
     if (vec) {
         const int per = dp / 8;
         for (int idx = threadIdx.x; idx < SS_C * per; idx += SS_THREADS) {
             const int t = idx / per, c = (idx % per) * 8;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (t < n && c < d) v = *(const uint4*)(src + (size_t)t * ld + c);
-            *(uint4*)(dst + t * dst_ld + c) = v;
+            const bool ok = t < n && c < d;
+            cp_async16(smem_u32(dst + t * dst_ld + c), ok ? (const void*)(src + (size_t)t * ld + c) : (const void*)src, ok);
         }
         return;
     }
@@ -317,8 +318,19 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_state(SsArgs a, const floa
     const int d = a.d, dv = a.dv, rows = dv + (MODE == SS_MLSTM ? 1 : 0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bf16* src = (const bf16*)a.src + (size_t)r.r0 * a.ld;
-    ss_log_sums(ld + (size_t)h * Tn + r.r0, r.n, lg);
     ss_tile(ks, kld, src + a.ok + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
+    const bf16* vsrc = src + a.ov + (size_t)h * dv + e0;
+    // values: 8 neighbours a load, 4 loads a thread in flight
+    const bool v8 = (vec & 4) && dv - e0 >= SS_E;
+    uint4 vv[4];
+    if (v8) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int idx = threadIdx.x + i * SS_THREADS, s = idx >> 3, c = (idx & 7) * 8;
+            vv[i] = s < r.n ? *(const uint4*)(vsrc + (size_t)s * a.ld + c) : make_uint4(0, 0, 0, 0);
+        }
+    }
+    ss_log_sums(ld + (size_t)h * Tn + r.r0, r.n, lg);
     __syncthreads();
     if (threadIdx.x < SS_C) {
         const int s = threadIdx.x;
@@ -326,8 +338,24 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_state(SsArgs a, const floa
     }
     if (threadIdx.x == 0 && blockIdx.z == 0) lg_end[(size_t)blockIdx.x * a.H + h] = lg[SS_C - 1];
     __syncthreads();
-    {
-        const bf16* vsrc = src + a.ov + (size_t)h * dv + e0;
+    if (v8) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int idx = threadIdx.x + i * SS_THREADS, s = idx >> 3, c = (idx & 7) * 8;
+            const __nv_bfloat162* p = (const __nv_bfloat162*)&vv[i];
+            uint32_t sp[KB_SPLIT][4];
+#pragma unroll
+            for (int k = 0; k < 4; k++) {
+                uint32_t q[KB_SPLIT];
+                split_pack_bf16(__low2float(p[k]) * wt[s], __high2float(p[k]) * wt[s], q);
+#pragma unroll
+                for (int u = 0; u < KB_SPLIT; u++) sp[u][k] = q[u];
+            }
+#pragma unroll
+            for (int u = 0; u < KB_SPLIT; u++)
+                *(uint4*)(vw + (u * SS_C + s) * SS_LD + c) = make_uint4(sp[u][0], sp[u][1], sp[u][2], sp[u][3]);
+        }
+    } else {
         for (int idx = threadIdx.x; idx < SS_C * (SS_E / 2); idx += SS_THREADS) {
             const int s = idx / (SS_E / 2), c = (idx % (SS_E / 2)) * 2;
             float x = 0.0f, y = 0.0f;
@@ -348,6 +376,7 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_state(SsArgs a, const floa
             for (int i = 0; i < KB_SPLIT; i++) *(uint32_t*)(vw + (i * SS_C + s) * SS_LD + c) = sp[i];
         }
     }
+    cp_async_wait_all();
     __syncthreads();
     float* pb = part + ((size_t)blockIdx.x * a.H + h) * rows * d;
     // this warp's 16 columns of the state against all of the keys' elements
@@ -461,20 +490,43 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bf16* src = (const bf16*)a.src + (size_t)r.r0 * a.ld;
     const int ne = min(SS_E, dv - e0);
+    const float* S0 = part + ((size_t)blockIdx.x * a.H + h) * rows * d;
+    // the state's columns, 64 elements at a time: four neighbours a load, eight loads a thread in flight, the next 64 on
+    // their way while the products of these run
+    const bool s4 = (vec & 16) && ne == SS_E;
+    float4 sv[8];
+    auto s_load = [&](int jb) {
+#pragma unroll
+        for (int i = 0; i < 8; i++) {
+            const int idx = threadIdx.x + i * SS_THREADS, e = idx >> 4, j = jb + (idx & 15) * 4;
+            sv[i] = j < d ? *(const float4*)(S0 + (size_t)(e0 + e) * d + j) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+    };
+    if (s4) s_load(0);
+    ss_tile(qs, kld, src + a.oq + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
+    ss_tile(ks, kld, src + a.ok + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
+    ss_tile(vs, SS_LD, src + a.ov + (size_t)h * dv + e0, a.ld, r.n, ne, SS_E, (vec & 4) && ne % 8 == 0);
     ss_log_sums(ld + (size_t)h * Tn + r.r0, r.n, lg);
     if (threadIdx.x >= 64 && threadIdx.x < 64 + SS_C) {
         const int s = threadIdx.x - 64;
         wt[s] = s < r.n ? w[(size_t)h * Tn + r.r0 + s] : 0.0f;
     }
-    ss_tile(qs, kld, src + a.oq + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
-    ss_tile(ks, kld, src + a.ok + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
-    ss_tile(vs, SS_LD, src + a.ov + (size_t)h * dv + e0, a.ld, r.n, ne, SS_E, (vec & 4) && ne % 8 == 0);
-    const float* S0 = part + ((size_t)blockIdx.x * a.H + h) * rows * d;
     const int t0 = warp * 16;
     float o[SS_E / 8][4] = {};
     for (int jb = 0; jb < dp; jb += 64) {
         __syncthreads();                               // (the tile before has been read)
-        for (int idx = threadIdx.x; idx < SS_E * 32; idx += SS_THREADS) {
+        if (s4) {
+#pragma unroll
+            for (int i = 0; i < 8; i++) {
+                const int idx = threadIdx.x + i * SS_THREADS, e = idx >> 4, c = (idx & 15) * 4;
+                uint32_t p[KB_SPLIT], q[KB_SPLIT];
+                split_pack_bf16(sv[i].x, sv[i].y, p);
+                split_pack_bf16(sv[i].z, sv[i].w, q);
+#pragma unroll
+                for (int u = 0; u < KB_SPLIT; u++) *(uint2*)(ss + (u * SS_E + e) * SS_LD + c) = make_uint2(p[u], q[u]);
+            }
+            if (jb + 64 < dp) s_load(jb + 64);
+        } else for (int idx = threadIdx.x; idx < SS_E * 32; idx += SS_THREADS) {
             const int e = idx >> 5, c = (idx & 31) * 2, j = jb + c;
             float x = 0.0f, y = 0.0f;
             if (e < ne) {
@@ -493,6 +545,7 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
 #pragma unroll
             for (int i = 0; i < KB_SPLIT; i++) *(uint32_t*)(ss + (i * SS_E + e) * SS_LD + c) = sp[i];
         }
+        cp_async_wait_all();
         __syncthreads();
         const int kn = min(64, dp - jb) / 16;
         for (int k = 0; k < kn; k++) {
@@ -594,25 +647,50 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
         sb += __shfl_xor_sync(0xffffffffu, sb, 1);
         sb += __shfl_xor_sync(0xffffffffu, sb, 2);
         const float* n0 = S0 + (size_t)dv * d;
+        float nr[8];                                   // (d <= 256 here)
+#pragma unroll
+        for (int k = 0; k < 8; k++) nr[k] = lane + 32 * k < d ? n0[lane + 32 * k] : 0.0f;
+#pragma unroll 4
         for (int i = 0; i < 16; i++) {
             const int t = t0 + i;
-            if (t >= r.n) break;
             float acc = 0.0f;
-            for (int j = lane; j < d; j += 32) acc = fmaf(n0[j], __bfloat162float(qs[t * kld + j]), acc);
+#pragma unroll
+            for (int k = 0; k < 8; k++)
+                if (32 * k < d && lane + 32 * k < dp) acc = fmaf(nr[k], __bfloat162float(qs[t * kld + lane + 32 * k]), acc);
             acc = kb_warp_sum(acc);
             const float own = __shfl_sync(0xffffffffu, i < 8 ? sa : sb, (i & 7) * 4);
-            if (lane == 0) a.nq[(size_t)(r.r0 + t) * a.H + h] = (expf(lg[t]) * acc + own) * a.qscale;
+            if (lane == 0 && t < r.n) a.nq[(size_t)(r.r0 + t) * a.H + h] = (expf(lg[t]) * acc + own) * a.qscale;
         }
     }
 }
 
 // ------------------------------------------------------------------------------------------------ norm on the output
+// four neighbours, aligned
+template <typename TG>
+__device__ __forceinline__ void ss_rd4(const TG* p, int n_planes, size_t plane_stride, float* z) {
+    for (int s = 0; s < n_planes; s++) {
+        float v[4];
+        if (sizeof(TG) == 4) {
+            const float4 q = *(const float4*)(p + (size_t)s * plane_stride);
+            v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+        } else {
+            const uint2 q = *(const uint2*)(p + (size_t)s * plane_stride);
+            const bf16* qb = (const bf16*)&q;
+#pragma unroll
+            for (int i = 0; i < 4; i++) v[i] = __bfloat162float(qb[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < 4; i++) z[i] = s == 0 ? v[i] : z[i] + v[i];
+    }
+}
+
 // A group's n neighbouring elements of a row by TPG threads:
 //   SS_MLSTM  u = x / (max(|nq|, exp(-m)) + 1e-6), out = rms(u) * gain * sigmoid(g); a group is a head; the running maximum
 //             of a sequence's last row becomes its state
 //   SS_MAMBA  u = x * silu(g), out = rms(u) * gain
-// VW: neighbouring elements a thread takes at once (4 where everything is aligned)
-template <typename TG, typename TO, int MODE, int TPG, int VW>
+// VW: neighbouring elements a thread takes at once (4 where everything is aligned); NI > 0: the group in registers, NI times
+// four neighbours a thread; NI == 0: in shared memory
+template <typename TG, typename TO, int MODE, int TPG, int VW, int NI>
 __global__ void __launch_bounds__(256) k_scan_norm(const float* KB_STEP_DATA x, int ldx, int T, int NG, int n,
         const float* __restrict__ w, float eps, const TG* KB_STEP_DATA g, int g_planes, size_t g_plane_stride, int ldg, int og,
         const float* KB_STEP_DATA nq, const float* KB_STEP_DATA m_rows, float* m_state, size_t m_stride,
@@ -628,6 +706,72 @@ __global__ void __launch_bounds__(256) k_scan_norm(const float* KB_STEP_DATA x, 
     const int t = live ? (int)(item / NG) : 0, h = live ? (int)(item % NG) : 0;
     kb_pdl_wait();
     float* u = sm + (size_t)gi * ((n + 3) & ~3);
+    const float* xr = x + (size_t)t * ldx + (size_t)h * n;
+    const TG* gr = g + (size_t)t * ldg + og + (size_t)h * n;
+    if constexpr (NI > 0) {
+        // the group in registers: every load in flight before the first use
+        float4 xv[NI], wv[NI];
+        float z[NI][4];
+#pragma unroll
+        for (int i = 0; i < NI; i++) {
+            const int c = (tid + i * TPG) * 4;
+            wv[i] = c < n ? *(const float4*)(w + (size_t)h * n + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            xv[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            z[i][0] = z[i][1] = z[i][2] = z[i][3] = 0.0f;
+            if (live && c < n) {
+                xv[i] = *(const float4*)(xr + c);
+                ss_rd4<TG>(gr + c, g_planes, g_plane_stride, z[i]);
+            }
+        }
+        float f = 1.0f;
+        if (MODE == SS_MLSTM && live) {
+            const float m = m_rows[(size_t)t * NG + h];
+            f = 1.0f / (fmaxf(fabsf(nq[(size_t)t * NG + h]), expf(-m)) + SS_DEN_EPS);
+            if (tid == 0 && pos[t] >= 0) {
+                const int b = seq[t];
+                if (t == q_start[b + 1] - 1) m_state[(size_t)slot[b] * m_stride + h] = m;
+            }
+        }
+        float sq = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NI; i++) {
+            float* v = (float*)&xv[i];
+#pragma unroll
+            for (int k = 0; k < 4; k++) {
+                v[k] *= MODE == SS_MLSTM ? f : z[i][k] / (1.0f + expf(-z[i][k]));
+                sq = fmaf(v[k], v[k], sq);
+            }
+        }
+        sq = kb_warp_sum(sq);
+        if (TPG > 32) {
+            if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+            __syncthreads();
+            sq = 0.0f;
+#pragma unroll
+            for (int k = 0; k < 8; k++) sq += red[k];
+        }
+        const float rn = 1.0f / sqrtf(sq / (float)n + eps);
+#pragma unroll
+        for (int i = 0; i < NI; i++) {
+            const int c = (tid + i * TPG) * 4;
+            if (!live || c >= n) continue;
+            const float* v = (const float*)&xv[i], *wf = (const float*)&wv[i];
+            float y[4];
+#pragma unroll
+            for (int k = 0; k < 4; k++) {
+                y[k] = __fmul_rn(__fmul_rn(v[k], rn), wf[k]);
+                if (MODE == SS_MLSTM) y[k] *= ss_sigmoid(z[i][k]);
+            }
+            TO* dst = out + (size_t)t * ldo + (size_t)h * n + c;
+            if (sizeof(TO) == 2) {
+                *(uint2*)dst = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
+            } else {
+#pragma unroll
+                for (int k = 0; k < 4; k++) dst[k] = kb_from_f<TO>(y[k]);
+            }
+        }
+        return;
+    }
     float f = 1.0f;
     if (MODE == SS_MLSTM && live) {
         const float m = m_rows[(size_t)t * NG + h];
@@ -637,27 +781,9 @@ __global__ void __launch_bounds__(256) k_scan_norm(const float* KB_STEP_DATA x, 
             if (t == q_start[b + 1] - 1) m_state[(size_t)slot[b] * m_stride + h] = m;
         }
     }
-    const float* xr = x + (size_t)t * ldx + (size_t)h * n;
-    const TG* gr = g + (size_t)t * ldg + og + (size_t)h * n;
     auto gate = [&](int c, float* z) {
-        if (VW == 4) {
-            for (int s = 0; s < g_planes; s++) {
-                float v[4];
-                if (sizeof(TG) == 4) {
-                    const float4 q = *(const float4*)(gr + (size_t)s * g_plane_stride + c);
-                    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
-                } else {
-                    const uint2 q = *(const uint2*)(gr + (size_t)s * g_plane_stride + c);
-                    const bf16* qb = (const bf16*)&q;
-#pragma unroll
-                    for (int i = 0; i < 4; i++) v[i] = __bfloat162float(qb[i]);
-                }
-#pragma unroll
-                for (int i = 0; i < 4; i++) z[i] = s == 0 ? v[i] : z[i] + v[i];
-            }
-        } else {
-            z[0] = ss_rd<TG>(gr + c, g_planes, g_plane_stride);
-        }
+        if (VW == 4) ss_rd4<TG>(gr + c, g_planes, g_plane_stride, z);
+        else z[0] = ss_rd<TG>(gr + c, g_planes, g_plane_stride);
     };
     float sq = 0.0f;
     if (live) {
@@ -785,12 +911,14 @@ extern "C" int kb_gated_scan_chunked(SS_PARAMS, int T, float* gates, float* part
     const int runs = T / SS_C + B, ez = (dv + SS_E - 1) / SS_E;
     float* ldg_ = gates, *w = gates + (size_t)H * T;
     const uintptr_t base = (uintptr_t)src;
-    // what may be moved in 16-byte words: bit 0 queries and keys, bit 2 values; bit 1: values in pairs; bit 3: output pairs
+    // what may be moved in 16-byte words: bit 0 queries and keys, bit 2 values, bit 4 the state; in pairs: bit 1 values, bit 3
+    // the output
     const bool rows16 = base % 16 == 0 && ld % 8 == 0;
     const int vec = (rows16 && oq % 8 == 0 && ok % 8 == 0 && d % 8 == 0 ? 1 : 0) |
                     (base % 4 == 0 && ld % 2 == 0 && ov % 2 == 0 && dv % 2 == 0 ? 2 : 0) |
                     (rows16 && ov % 8 == 0 && dv % 8 == 0 ? 4 : 0) |
-                    ((uintptr_t)out % 8 == 0 && ldo % 2 == 0 && dv % 2 == 0 ? 8 : 0);
+                    ((uintptr_t)out % 8 == 0 && ldo % 2 == 0 && dv % 2 == 0 ? 8 : 0) |
+                    ((uintptr_t)part % 16 == 0 && d % 4 == 0 ? 16 : 0);
     const size_t sm_a = (size_t)(KB_SPLIT * SS_C * SS_LD + SS_C * (dp + 8)) * 2;
     const size_t sm_c = (size_t)(KB_SPLIT * SS_E * SS_LD + SS_C * SS_LD + 2 * SS_C * (dp + 8)) * 2;
     const dim3 grid(runs, H, ez);
@@ -803,7 +931,7 @@ extern "C" int kb_gated_scan_chunked(SS_PARAMS, int T, float* gates, float* part
             cudaFuncSetAttribute(k_chunk_state<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024);        \
             cudaFuncSetAttribute(k_chunk_out<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024);          \
         }                                                                                                              \
-        kb_launch(k_scan_gates<bf16, MODE>, dim3(H, B, MODE == SS_MAMBA ? 4 : 1), 256, 0, st, a, ldg_, w, T);          \
+        kb_launch(k_scan_gates<bf16, MODE>, dim3(H, B, MODE == SS_MAMBA ? 4 : 1), MODE == SS_MAMBA ? 256 : SG_T, 0, st, a, ldg_, w, T);          \
         kb_launch(k_chunk_state<MODE>, grid, SS_THREADS, sm_a, st, a, (const float*)ldg_, (const float*)w, T, part,    \
                   lg_end, dp, vec);                                                                                    \
         if (v4)                                                                                                        \
@@ -834,17 +962,25 @@ extern "C" int kb_scan_norm(int mode, const float* x, int ldx, int T, int NG, in
     const long long blocks = ((long long)T * NG + gpb - 1) / gpb;
     const int gel = gdtype == KB_F32 ? 4 : 2, oel = odtype == KB_F32 ? 4 : 2;
     const bool v4 = n % 4 == 0 && ldx % 4 == 0 && ldg % 4 == 0 && og % 4 == 0 && g_plane_stride % 4 == 0 && ldo % 4 == 0 &&
-                    (uintptr_t)x % 16 == 0 && (uintptr_t)g % (4 * gel) == 0 && (uintptr_t)out % (4 * oel) == 0;
-#define SS_N(TG, TO, MODE, TPG, VW)                                                                                    \
+                    (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && (uintptr_t)g % (4 * gel) == 0 && (uintptr_t)out % (4 * oel) == 0;
+    // (the register forms need no shared memory)
+    const int ni = !v4 ? 0 : (n / 4 + (wide ? 255 : 31)) / (wide ? 256 : 32);
+#define SS_N(TG, TO, MODE, TPG, VW, NI)                                                                                \
     do {                                                                                                               \
-        if (sm > 48 * 1024)                                                                                            \
-            cudaFuncSetAttribute(k_scan_norm<TG, TO, MODE, TPG, VW>, cudaFuncAttributeMaxDynamicSharedMemorySize,      \
+        if (NI == 0 && sm > 48 * 1024)                                                                                 \
+            cudaFuncSetAttribute(k_scan_norm<TG, TO, MODE, TPG, VW, NI>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
                                  (int)sm);                                                                             \
-        kb_launch(k_scan_norm<TG, TO, MODE, TPG, VW>, (unsigned)blocks, 256, sm, st, x, ldx, T, NG, n, w, eps,         \
-                  (const TG*)g, g_planes, (size_t)g_plane_stride, ldg, og, nq, m_rows, m_state, (size_t)m_stride, pos, \
-                  seq, slot, q_start, (TO*)out, ldo);                                                                  \
+        kb_launch(k_scan_norm<TG, TO, MODE, TPG, VW, NI>, (unsigned)blocks, 256, NI ? (size_t)0 : sm, st, x, ldx, T,   \
+                  NG, n, w, eps, (const TG*)g, g_planes, (size_t)g_plane_stride, ldg, og, nq, m_rows, m_state,         \
+                  (size_t)m_stride, pos, seq, slot, q_start, (TO*)out, ldo);                                           \
     } while (0)
-#define SS_N3(TG, TO, MODE, TPG) do { if (v4) SS_N(TG, TO, MODE, TPG, 4); else SS_N(TG, TO, MODE, TPG, 1); } while (0)
+#define SS_N3(TG, TO, MODE, TPG)                                                                                       \
+    do {                                                                                                               \
+        if (ni == 1) SS_N(TG, TO, MODE, TPG, 4, 1);                                                                    \
+        else if (ni >= 2 && ni <= 4) SS_N(TG, TO, MODE, TPG, 4, 4);                                                    \
+        else if (v4) SS_N(TG, TO, MODE, TPG, 4, 0);                                                                    \
+        else SS_N(TG, TO, MODE, TPG, 1, 0);                                                                            \
+    } while (0)
 #define SS_N2(TG, TO, MODE) do { if (wide) SS_N3(TG, TO, MODE, 256); else SS_N3(TG, TO, MODE, 32); } while (0)
 #define SS_N1(TG, TO) do { if (mode == SS_MLSTM) SS_N2(TG, TO, SS_MLSTM); else SS_N2(TG, TO, SS_MAMBA); } while (0)
     if (gdtype == KB_F32 && odtype == KB_F32) SS_N1(float, float);

@@ -129,13 +129,13 @@ _PAIR_SCRATCH = {}         # device -> (partial tiles, flags): scratch of tiles 
 
 
 def _prefill_product(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor, swiglu: bool,
-                     act: str = "silu", act_params=None) -> None:
+                     act: str = "silu", act_params=None, post=None) -> None:
     m, k = a.shape
     n = w.shape[0]
     kind, bn, variant = _prefill_tile(m, n, k, swiglu)
     if kind == "tc":
         K.gemm_tc(a, w, out, swap=False, bn=bn, splits=1, status=status, swiglu=swiglu, mt=variant, act=act,
-                  act_params=act_params)
+                  act_params=act_params, post=post)
         return
     part = flags = None
     if variant:
@@ -146,7 +146,8 @@ def _prefill_product(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status
                     torch.zeros(8 * tiles, dtype=torch.int32, device=a.device))
             _PAIR_SCRATCH[a.device] = have
         part, flags = have
-    K.gemm_pair(a, w, out, bn=bn, status=status, swiglu=swiglu, part=part, flags=flags, act=act, act_params=act_params)
+    K.gemm_pair(a, w, out, bn=bn, status=status, swiglu=swiglu, part=part, flags=flags, act=act, act_params=act_params,
+                post=post)
 
 
 def gemm_rows(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor) -> bool:
@@ -157,6 +158,22 @@ def gemm_rows(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch
         K.gemm_tc(a, w, out, swap=True, bn=_swap_bn(m), splits=1, status=status)
     else:
         _prefill_product(a, w, out, status, False)
+    return True
+
+
+def gemm_bias_act(a: torch.Tensor, w: torch.Tensor, bias, act: str, out: torch.Tensor, status: torch.Tensor) -> bool:
+    """out (bf16 [M, N]) = act(a @ w^T + bias) finished in the product's epilogue: prompt-sized steps, and decode-sized ones
+    whose product does not split K. False: not taken"""
+    if not _tc_ok(a, w) or not out.is_contiguous() or out.dtype != torch.bfloat16:
+        return False
+    (m, k), n = a.shape, w.shape[0]
+    if m <= SMALL_M:
+        bn = _swap_bn(m)
+        if _splits_for(m, n, k, bn) != 1:
+            return False
+        K.gemm_tc(a, w, out, swap=True, bn=bn, splits=1, status=status, post=(bias, act))
+    else:
+        _prefill_product(a, w, out, status, False, post=(bias, act))
     return True
 
 

@@ -108,11 +108,11 @@ _SIGS = {
                     c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "kb_swiglu": [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int],
     "kb_gemm_tc": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                   c_longlong, c_void_p, c_void_p, c_int, c_int, c_float, c_float],
+                   c_longlong, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_int],
     "kb_gemm_tc_splits": [c_int, c_int],
     "kb_rope_table_min_rows": [],
     "kb_gemm_pair": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                     c_void_p, c_int, c_void_p, c_void_p, c_float, c_float],
+                     c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int],
     "kb_gemm_swiglu_decode": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                               c_void_p, c_void_p, c_void_p, c_int, c_float, c_float],
     "kb_attn_mma": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
@@ -768,13 +768,28 @@ def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int = 0, act: str = "silu
                             GATE_ACT[act]), "swiglu")
 
 
+def _post_args(post, n: int, out: torch.Tensor, swiglu: bool):
+    """(bias or None, activation code or -1) of a product that finishes its own bf16 rows"""
+    if post is None:
+        return None, -1
+    bias, act = post
+    assert not swiglu and out.dtype == torch.bfloat16 and out.dim() == 2
+    if bias is not None:
+        _need_cuda(bias)
+        assert bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == n
+    return bias, ACT[act]
+
+
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swap: bool, bn: int, splits: int,
-            status: torch.Tensor, swiglu: bool = False, mt: int = 1, act: str = "silu", act_params=None) -> None:
+            status: torch.Tensor, swiglu: bool = False, mt: int = 1, act: str = "silu", act_params=None,
+            post=None) -> None:
     """out = a[M, K] @ w[N, K]^T on the tensor cores (bf16 in, fp32 accumulate). ``out`` is [M, N] (bf16 or fp32)
     or, with K splits, fp32 [S, M, N] where S = gemm_tc_splits(K, splits). ``swiglu`` (prefill form, bn a multiple
     of 32): w holds 16 gate rows then the 16 up rows of the same outputs, group after group, and ``out`` is the bf16
-    [M, N / 2] result silu(gate) * up. ``mt`` = 2 (prefill form): a unit is two 128-row tiles over the same columns"""
+    [M, N / 2] result silu(gate) * up. ``mt`` = 2 (prefill form): a unit is two 128-row tiles over the same columns.
+    ``post`` = (float32 bias [N] or None, a key of ``ACT``): the bf16 rows leave as act(. + bias)"""
     _need_cuda(a, w, out)
+    bias, pact = _post_args(post, w.shape[0], out, swiglu)
     M, K = a.shape
     N = w.shape[0]
     assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K
@@ -790,18 +805,20 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swap: bool, 
         stride, ldc = 0, N
     _check(load().kb_gemm_tc(_p(a), _p(w), _p(out), dt(out), M, N, K, a.stride(0), w.stride(0), ldc, 1 if swap else 0,
                              bn, splits, stride, _p(status), _stream(), GATE_ACT[act] if swiglu else 0, mt,
-                             *_gate_params(act, act_params)), "gemm_tc")
+                             *_gate_params(act, act_params), _p(bias), pact), "gemm_tc")
 
 
 def gemm_pair(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bn: int, status: torch.Tensor,
               swiglu: bool = False, part: Optional[torch.Tensor] = None, flags: Optional[torch.Tensor] = None,
-              act: str = "silu", act_params=None) -> None:
+              act: str = "silu", act_params=None, post=None) -> None:
     """out = a[M, K] @ w[N, K]^T by pairs of SMs (tcgen05 with cta_group::2: a pair computes 256 rows x bn columns,
     each CTA holding half of the weight tile), bf16 in, fp32 accumulate, ``out`` [M, N] bf16 or fp32; bn 64, 128, 192
     or 256. ``swiglu``: as for gemm_tc, ``out`` is the bf16 [M, N / 2] result silu(gate) * up. With ``part`` (fp32, at
     least tiles * 256 * bn elements, tiles = ceil(M / 256) * ceil(N / bn)) and ``flags`` (int32 zeros, 8 a tile) the
-    K blocks of all tiles are dealt out evenly to the pairs and a tile may be finished by two of them"""
+    K blocks of all tiles are dealt out evenly to the pairs and a tile may be finished by two of them. ``post``: as for
+    gemm_tc"""
     _need_cuda(a, w, out)
+    bias, pact = _post_args(post, w.shape[0], out, swiglu)
     M, K = a.shape
     N = w.shape[0]
     assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K
@@ -818,7 +835,7 @@ def gemm_pair(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bn: int, s
         assert flags.dtype == torch.int32 and flags.numel() >= 8 * tiles and flags.is_contiguous()
     _check(load().kb_gemm_pair(_p(a), _p(w), _p(out), dt(out), M, N, K, a.stride(0), w.stride(0), ldc, bn, _p(status),
                                _stream(), GATE_ACT[act] if swiglu else 0, _p(part), _p(flags),
-                               *_gate_params(act, act_params)), "gemm_pair")
+                               *_gate_params(act, act_params), _p(bias), pact), "gemm_pair")
 
 
 def gemm_swiglu_decode(a: torch.Tensor, w_grouped: torch.Tensor, out: torch.Tensor, bn: int, part: torch.Tensor,

@@ -45,9 +45,11 @@ def rows_or_planes(ctx, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype
 
 
 def linear_bias_act(ctx, y: torch.Tensor, w: torch.Tensor, bias, act: str, out_dtype: torch.dtype) -> torch.Tensor:
-    """``act(y @ w^T + bias)`` (``[M, N]`` in out_dtype; ``bias`` float32 ``[N]`` or None): the product as rows or 32-bit
-    planes followed by one kernel"""
+    """``act(y @ w^T + bias)`` (``[M, N]`` in out_dtype; ``bias`` float32 ``[N]`` or None): in the product's epilogue where a
+    tensor-core kernel takes the shape, else the product as rows or 32-bit planes followed by one kernel"""
     h = torch.empty((y.shape[0], w.shape[0]), dtype=out_dtype, device=y.device)
+    if ctx.fast and fast.gemm_bias_act(y, w, bias, act, h, ctx.status):
+        return h
     K.bias_act(rows_or_planes(ctx, y, w, out_dtype), bias, act, h)
     return h
 
