@@ -199,7 +199,7 @@ static inline KbCap kb_cap_of(const float* h) {
 // kernel has finished and its writes are visible, so results are those of strictly ordered launches; what is
 // gained is that launch latency and prologues overlap the predecessor's tail.
 // Before its wait a kernel also reads the step's metadata (positions, lengths, slots, row lists, the page table)
-// and cache pages of older positions. Callers therefore write those with operations that are complete before the
+// and cache pages of older positions (a recurrence's token-by-token kernel its states of earlier steps). Callers therefore write those with operations that are complete before the
 // step's first kernel starts: the engine brings the page table up to date and then copies the metadata to the
 // device (a copy orders fully), and older pages were stored by earlier steps.
 __device__ __forceinline__ void kb_pdl_launch_now() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }

@@ -220,7 +220,9 @@ __global__ void __launch_bounds__(128) k_short_conv_rows(const bf16* KB_STEP_DAT
         uint32_t h[4];
 #pragma unroll
         for (int e = 0; e < 4; e++) {
-            const float x = act ? rc_silu(acc[2 * e]) : acc[2 * e], y = act ? rc_silu(acc[2 * e + 1]) : acc[2 * e + 1];
+            // (the fast exponential and division: their error is far below the rounding to bf16)
+            const float x = act ? __fdividef(acc[2 * e], 1.0f + __expf(-acc[2 * e])) : acc[2 * e];
+            const float y = act ? __fdividef(acc[2 * e + 1], 1.0f + __expf(-acc[2 * e + 1])) : acc[2 * e + 1];
             __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
             h[e] = *(uint32_t*)&v;
         }

@@ -63,6 +63,8 @@ __device__ __forceinline__ float ss_rd(const T* p, int n_planes, size_t plane_st
 }
 __device__ __forceinline__ float ss_softplus(float z) { return log1pf(expf(-fabsf(z))) + fmaxf(z, 0.0f); }
 __device__ __forceinline__ float ss_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// where the result is rounded to bf16 anyway: the fast exponential and division (a few units of 2^-23)
+__device__ __forceinline__ float ss_sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 
 // the two numbers a token's gates are made of: (i, f) of the matrix memory, (dt, log decay) of the state space
 template <typename T, int MODE>
@@ -82,35 +84,41 @@ __device__ __forceinline__ void ss_gate(const SsArgs& a, int row, int h, float& 
 // ------------------------------------------------------------------------------------------------ token by token
 // A block works one (sequence, head) and SS_COLS columns of the state, a warp one column with its d elements over the
 // lanes; tokens are staged SS_STAGE at a time.
+// (NC of them, neighbours SS_COLS apart, when there are blocks enough: the loads of all of them are in flight together)
 #define SS_COLS 8
 #define SS_STAGE 16
-template <typename T, int MODE, int DPL>
-__global__ void __launch_bounds__(32 * SS_COLS) k_gated_scan(SsArgs a) {
+template <typename T, int MODE, int DPL, int NC>
+__global__ void __launch_bounds__(32 * SS_COLS, DPL * NC >= 16 ? 2 : 3) k_gated_scan(SsArgs a) {
     extern __shared__ float sm[];
     const int d = a.d, dv = a.dv, H = a.H;
     float* qs = sm;                                   // [SS_STAGE][d]
     float* ks = qs + SS_STAGE * d;                    // [SS_STAGE][d]
-    float* vs = ks + SS_STAGE * d;                    // [SS_STAGE][SS_COLS]
-    float* g0 = vs + SS_STAGE * SS_COLS;              // [SS_STAGE]: i, then w
+    constexpr int COLS = SS_COLS * NC;
+    float* vs = ks + SS_STAGE * d;                    // [SS_STAGE][COLS]
+    float* g0 = vs + SS_STAGE * COLS;                 // [SS_STAGE]: i, then w
     float* g1 = g0 + SS_STAGE;                        // [SS_STAGE]: f, then a
     float* ms = g1 + SS_STAGE;                        // [SS_STAGE + 1]: running maxima, the one before the stage first
     kb_pdl_launch();
     const int b = blockIdx.x / H, h = blockIdx.x % H, hq = h / a.per;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int rows = dv + (MODE == SS_MLSTM ? 1 : 0);
-    const int e0 = blockIdx.y * SS_COLS, e = e0 + warp;
+    const int e0 = blockIdx.y * COLS, e = e0 + warp;   // this warp's columns: e, e + SS_COLS, ...
     const int r0 = a.q_start[b], r1 = a.q_start[b + 1];
     const int sl = a.slot[b];
-    float* srow = a.state + (size_t)sl * a.state_stride + ((size_t)h * rows + (e < rows ? e : 0)) * d;
+    float* srow = a.state + (size_t)sl * a.state_stride + (size_t)h * rows * d;
     const float D = MODE == SS_MAMBA ? a.p2[h] : 0.0f;
-    kb_pdl_wait();
-    float S[DPL];
+    // The states were left by earlier steps, which are complete before this step's first kernel starts: they are fetched
+    // while the kernel before this one still runs.
+    float S[NC][DPL];
 #pragma unroll
-    for (int i = 0; i < DPL; i++) {
-        const int j = lane + 32 * i;
-        S[i] = (e < rows && j < d) ? srow[j] : 0.0f;
-    }
+    for (int c = 0; c < NC; c++)
+#pragma unroll
+        for (int i = 0; i < DPL; i++) {
+            const int j = lane + 32 * i, ec = e + c * SS_COLS;
+            S[c][i] = (ec < rows && j < d) ? srow[(size_t)ec * d + j] : 0.0f;
+        }
     if (MODE == SS_MLSTM && threadIdx.x == 0) ms[SS_STAGE] = a.m_state[(size_t)sl * a.m_stride + h];
+    kb_pdl_wait();
     const size_t oq = (size_t)a.oq + (size_t)hq * d, ok = (size_t)a.ok + (size_t)hq * d, ov = (size_t)a.ov + (size_t)h * dv;
     int last_n = SS_STAGE;
     for (int c0 = r0; c0 < r1; c0 += SS_STAGE) {
@@ -122,8 +130,8 @@ __global__ void __launch_bounds__(32 * SS_COLS) k_gated_scan(SsArgs a) {
             qs[idx] = __fmul_rn(ss_rd<T>(p + oq, a.n_planes, a.plane_stride), a.qscale);
             ks[idx] = ss_rd<T>(p + ok, a.n_planes, a.plane_stride);
         }
-        for (int idx = threadIdx.x; idx < n * SS_COLS; idx += 32 * SS_COLS) {
-            const int t = idx / SS_COLS, c = e0 + idx % SS_COLS;
+        for (int idx = threadIdx.x; idx < n * COLS; idx += 32 * SS_COLS) {
+            const int t = idx / COLS, c = e0 + idx % COLS;
             vs[idx] = c < dv ? ss_rd<T>(base + (size_t)t * a.ld + ov + c, a.n_planes, a.plane_stride) : 1.0f;
         }
         if (threadIdx.x < n) {
@@ -155,31 +163,46 @@ __global__ void __launch_bounds__(32 * SS_COLS) k_gated_scan(SsArgs a) {
         }
         for (int t = 0; t < n; t++) {
             const float keep = g1[t];
-            const float v = vs[t * SS_COLS + warp];
-            const float wv = __fmul_rn(g0[t], v);
-            float o = 0.0f;
+            float v[NC], wv[NC], o[NC];
+#pragma unroll
+            for (int c = 0; c < NC; c++) {
+                v[c] = vs[t * COLS + c * SS_COLS + warp];
+                wv[c] = __fmul_rn(g0[t], v[c]);
+                o[c] = 0.0f;
+            }
 #pragma unroll
             for (int i = 0; i < DPL; i++) {
                 const int j = lane + 32 * i;
                 if (j < d) {
-                    S[i] = fmaf(ks[t * d + j], wv, __fmul_rn(keep, S[i]));
-                    o = fmaf(S[i], qs[t * d + j], o);
+                    const float kv = ks[t * d + j], qv = qs[t * d + j];
+#pragma unroll
+                    for (int c = 0; c < NC; c++) {
+                        S[c][i] = fmaf(kv, wv[c], __fmul_rn(keep, S[c][i]));
+                        o[c] = fmaf(S[c][i], qv, o[c]);
+                    }
                 }
             }
-            o = kb_warp_sum(o);
-            if (lane == 0 && e < rows) {
-                if (e < dv) a.out[(size_t)(c0 + t) * a.ldo + (size_t)h * dv + e] = fmaf(D, v, o);
-                else a.nq[(size_t)(c0 + t) * H + h] = o;
+#pragma unroll
+            for (int c = 0; c < NC; c++) o[c] = kb_warp_sum(o[c]);
+#pragma unroll
+            for (int c = 0; c < NC; c++) {
+                const int ec = e + c * SS_COLS;
+                if (lane == 0 && ec < rows) {
+                    if (ec < dv) a.out[(size_t)(c0 + t) * a.ldo + (size_t)h * dv + ec] = fmaf(D, v[c], o[c]);
+                    else a.nq[(size_t)(c0 + t) * H + h] = o[c];
+                }
             }
         }
         __syncthreads();
     }
-    if (e < rows && r1 > r0) {
+    if (r1 > r0) {
 #pragma unroll
-        for (int i = 0; i < DPL; i++) {
-            const int j = lane + 32 * i;
-            if (j < d) srow[j] = S[i];
-        }
+        for (int c = 0; c < NC; c++)
+#pragma unroll
+            for (int i = 0; i < DPL; i++) {
+                const int j = lane + 32 * i, ec = e + c * SS_COLS;
+                if (ec < rows && j < d) srow[(size_t)ec * d + j] = S[c][i];
+            }
     }
 }
 
@@ -391,21 +414,26 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_state(SsArgs a, const floa
                 const int row = k * 16 + ((lane >> 4) & 1) * 8 + (lane & 7), col = m0 + ((lane >> 3) & 1) * 8;
                 ldsm_x4_t(smem_u32(vw + (i * SS_C + row) * SS_LD + col), av[i][k][0], av[i][k][1], av[i][k][2], av[i][k][3]);
             }
-        for (int j0 = 0; j0 < dp; j0 += 16) {
-            float acc[2][4] = {};
+        for (int j0 = 0; j0 < dp; j0 += 32) {
+            // 32 of the keys' elements at a time (the last 16 of an odd multiple twice, which is not stored): four chains of
+            // products that do not wait for one another
+            const int j1 = j0 + 16 < dp ? j0 + 16 : j0;
+            float acc[4][4] = {};
 #pragma unroll
             for (int k = 0; k < SS_C / 16; k++) {
-                uint32_t b0, b1, b2, b3;
-                const int row = k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, col = j0 + (lane >> 4) * 8;
-                ldsm_x4_t(smem_u32(ks + row * kld + col), b0, b1, b2, b3);
+                uint32_t bf[2][4];
+                const int row = k * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, col = (lane >> 4) * 8;
+                ldsm_x4_t(smem_u32(ks + row * kld + j0 + col), bf[0][0], bf[0][1], bf[0][2], bf[0][3]);
+                ldsm_x4_t(smem_u32(ks + row * kld + j1 + col), bf[1][0], bf[1][1], bf[1][2], bf[1][3]);
 #pragma unroll
-                for (int i = KB_SPLIT - 1; i >= 0; i--) {
-                    mma_bf16(acc[0], av[i][k], b0, b1);
-                    mma_bf16(acc[1], av[i][k], b2, b3);
-                }
+                for (int i = KB_SPLIT - 1; i >= 0; i--)
+#pragma unroll
+                    for (int u = 0; u < 4; u++) mma_bf16(acc[u], av[i][k], bf[u >> 1][(u & 1) * 2], bf[u >> 1][(u & 1) * 2 + 1]);
             }
+            const int nu = j1 > j0 ? 4 : 2;
 #pragma unroll
-            for (int u = 0; u < 2; u++) {
+            for (int u = 0; u < 4; u++) {
+                if (u >= nu) break;
                 const int j = j0 + u * 8 + (lane & 3) * 2;
 #pragma unroll
                 for (int hf = 0; hf < 2; hf++) {
@@ -476,10 +504,10 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
         int Tn, const float* KB_STEP_DATA part, int dp, int vec) {
     extern __shared__ __align__(16) uint8_t sm8[];
     const int kld = dp + 8;
-    bf16* ss = (bf16*)sm8;                             // [KB_SPLIT][SS_E][SS_LD]: 64 elements of the state's columns
-    bf16* vs = ss + KB_SPLIT * SS_E * SS_LD;           // [SS_C][SS_LD]
-    bf16* qs = vs + SS_C * SS_LD;                      // [SS_C][kld]
-    bf16* ks = qs + SS_C * kld;                        // [SS_C][kld]
+    bf16* qs = (bf16*)sm8;                             // [SS_C][kld]
+    bf16* ss = qs + SS_C * kld;                        // [KB_SPLIT][SS_E][SS_LD]: 64 elements of the state's columns; then
+    bf16* vs = ss;                                     // [SS_C][SS_LD]
+    bf16* ks = vs + SS_C * SS_LD;                      // [SS_C][kld]
     __shared__ float lg[SS_C], wt[SS_C];
     kb_pdl_launch();
     const SsRun r = ss_run(a, blockIdx.x);
@@ -504,8 +532,6 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
     };
     if (s4) s_load(0);
     ss_tile(qs, kld, src + a.oq + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
-    ss_tile(ks, kld, src + a.ok + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
-    ss_tile(vs, SS_LD, src + a.ov + (size_t)h * dv + e0, a.ld, r.n, ne, SS_E, (vec & 4) && ne % 8 == 0);
     ss_log_sums(ld + (size_t)h * Tn + r.r0, r.n, lg);
     if (threadIdx.x >= 64 && threadIdx.x < 64 + SS_C) {
         const int s = threadIdx.x - 64;
@@ -553,18 +579,27 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
             ldsm_x4(smem_u32(qs + (t0 + (lane & 7) + ((lane >> 3) & 1) * 8) * kld + jb + k * 16 + (lane >> 4) * 8), aq[0],
                     aq[1], aq[2], aq[3]);
 #pragma unroll
-            for (int n2 = 0; n2 < SS_E / 16; n2++) {
+            for (int np = 0; np < SS_E / 32; np++) {
+                // 32 columns at a time: all loads first, then four chains of products
+                uint32_t bf[KB_SPLIT][2][4];
+                const int row = np * 32 + (lane & 7) + (lane >> 4) * 8, col = k * 16 + ((lane >> 3) & 1) * 8;
 #pragma unroll
-                for (int i = KB_SPLIT - 1; i >= 0; i--) {
-                    uint32_t b0, b1, b2, b3;
-                    const int row = n2 * 16 + (lane & 7) + (lane >> 4) * 8, col = k * 16 + ((lane >> 3) & 1) * 8;
-                    ldsm_x4(smem_u32(ss + (i * SS_E + row) * SS_LD + col), b0, b1, b2, b3);
-                    mma_bf16(o[2 * n2], aq, b0, b1);
-                    mma_bf16(o[2 * n2 + 1], aq, b2, b3);
-                }
+                for (int i = 0; i < KB_SPLIT; i++)
+#pragma unroll
+                    for (int u = 0; u < 2; u++)
+                        ldsm_x4(smem_u32(ss + (i * SS_E + row + u * 16) * SS_LD + col), bf[i][u][0], bf[i][u][1], bf[i][u][2],
+                                bf[i][u][3]);
+#pragma unroll
+                for (int i = KB_SPLIT - 1; i >= 0; i--)
+#pragma unroll
+                    for (int u = 0; u < 4; u++)
+                        mma_bf16(o[4 * np + u], aq, bf[i][u >> 1][(u & 1) * 2], bf[i][u >> 1][(u & 1) * 2 + 1]);
             }
         }
     }
+    __syncthreads();                                   // the state's tile is done with: its place takes keys and values
+    ss_tile(ks, kld, src + a.ok + (size_t)(h / a.per) * d, a.ld, r.n, d, dp, vec & 1);
+    ss_tile(vs, SS_LD, src + a.ov + (size_t)h * dv + e0, a.ld, r.n, ne, SS_E, (vec & 4) && ne % 8 == 0);
     // the state's share decays from the run's start
     const int ta = t0 + (lane >> 2), tb = ta + 8;
     const float la = lg[ta], lb = lg[tb], fa = expf(la), fb = expf(lb);
@@ -575,19 +610,35 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
         o[n][2] *= fb;
         o[n][3] *= fb;
     }
+    cp_async_wait_all();
+    __syncthreads();
     // the run's own tokens, 16 keys at a time: score, decay and weight, sum
     float sa = 0.0f, sb = 0.0f;                        // sums of the weights (the normaliser's share)
     for (int k2 = 0; k2 <= warp; k2++) {
-        float sc[2][4] = {};
-        for (int k = 0; k < dp / 16; k++) {
-            uint32_t aq[4], b0, b1, b2, b3;
-            ldsm_x4(smem_u32(qs + (t0 + (lane & 7) + ((lane >> 3) & 1) * 8) * kld + k * 16 + (lane >> 4) * 8), aq[0], aq[1],
-                    aq[2], aq[3]);
-            ldsm_x4(smem_u32(ks + (k2 * 16 + (lane & 7) + (lane >> 4) * 8) * kld + k * 16 + ((lane >> 3) & 1) * 8), b0, b1,
-                    b2, b3);
-            mma_bf16(sc[0], aq, b0, b1);
-            mma_bf16(sc[1], aq, b2, b3);
+        float sc[2][4] = {}, s1[2][4] = {};
+        for (int k = 0; k < dp / 16; k += 2) {
+            // two steps at a time, in sums of their own
+            const bool two = (k + 1) * 16 < dp;
+            uint32_t aq[2][4], bf[2][4];
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const int kk = (u == 0 || two) ? k + u : k;
+                ldsm_x4(smem_u32(qs + (t0 + (lane & 7) + ((lane >> 3) & 1) * 8) * kld + kk * 16 + (lane >> 4) * 8), aq[u][0],
+                        aq[u][1], aq[u][2], aq[u][3]);
+                ldsm_x4(smem_u32(ks + (k2 * 16 + (lane & 7) + (lane >> 4) * 8) * kld + kk * 16 + ((lane >> 3) & 1) * 8),
+                        bf[u][0], bf[u][1], bf[u][2], bf[u][3]);
+            }
+            mma_bf16(sc[0], aq[0], bf[0][0], bf[0][1]);
+            mma_bf16(sc[1], aq[0], bf[0][2], bf[0][3]);
+            if (two) {
+                mma_bf16(s1[0], aq[1], bf[1][0], bf[1][1]);
+                mma_bf16(s1[1], aq[1], bf[1][2], bf[1][3]);
+            }
         }
+#pragma unroll
+        for (int u = 0; u < 2; u++)
+#pragma unroll
+            for (int c = 0; c < 4; c++) sc[u][c] += s1[u][c];
         uint32_t pa[KB_SPLIT][4];
 #pragma unroll
         for (int u = 0; u < 2; u++) {
@@ -609,15 +660,17 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
             }
         }
 #pragma unroll
-        for (int d2 = 0; d2 < SS_E / 16; d2++) {
-            uint32_t b0, b1, b2, b3;
-            ldsm_x4_t(smem_u32(vs + (k2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * SS_LD + d2 * 16 + (lane >> 4) * 8), b0,
-                      b1, b2, b3);
+        for (int dp2 = 0; dp2 < SS_E / 32; dp2++) {
+            uint32_t bf[2][4];
 #pragma unroll
-            for (int i = KB_SPLIT - 1; i >= 0; i--) {
-                mma_bf16(o[2 * d2], pa[i], b0, b1);
-                mma_bf16(o[2 * d2 + 1], pa[i], b2, b3);
-            }
+            for (int u = 0; u < 2; u++)
+                ldsm_x4_t(smem_u32(vs + (k2 * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * SS_LD + (dp2 * 2 + u) * 16 +
+                                   (lane >> 4) * 8), bf[u][0], bf[u][1], bf[u][2], bf[u][3]);
+#pragma unroll
+            for (int i = KB_SPLIT - 1; i >= 0; i--)
+#pragma unroll
+                for (int u = 0; u < 4; u++)
+                    mma_bf16(o[4 * dp2 + u], pa[i], bf[u >> 1][(u & 1) * 2], bf[u >> 1][(u & 1) * 2 + 1]);
         }
     }
     const float D = MODE == SS_MAMBA ? a.p2[h] : 0.0f;
@@ -738,7 +791,7 @@ __global__ void __launch_bounds__(256) k_scan_norm(const float* KB_STEP_DATA x, 
             float* v = (float*)&xv[i];
 #pragma unroll
             for (int k = 0; k < 4; k++) {
-                v[k] *= MODE == SS_MLSTM ? f : z[i][k] / (1.0f + expf(-z[i][k]));
+                v[k] *= MODE == SS_MLSTM ? f : z[i][k] * (sizeof(TO) == 2 ? ss_sigmoid_fast(z[i][k]) : ss_sigmoid(z[i][k]));
                 sq = fmaf(v[k], v[k], sq);
             }
         }
@@ -760,7 +813,7 @@ __global__ void __launch_bounds__(256) k_scan_norm(const float* KB_STEP_DATA x, 
 #pragma unroll
             for (int k = 0; k < 4; k++) {
                 y[k] = __fmul_rn(__fmul_rn(v[k], rn), wf[k]);
-                if (MODE == SS_MLSTM) y[k] *= ss_sigmoid(z[i][k]);
+                if (MODE == SS_MLSTM) y[k] *= sizeof(TO) == 2 ? ss_sigmoid_fast(z[i][k]) : ss_sigmoid(z[i][k]);
             }
             TO* dst = out + (size_t)t * ldo + (size_t)h * n + c;
             if (sizeof(TO) == 2) {
@@ -872,20 +925,23 @@ extern "C" int kb_gated_scan(SS_PARAMS, cudaStream_t st) {
     if (!ss_ok(mode, H, per, d, dv, m_state, nq, m_rows)) return (int)cudaErrorInvalidValue;
     const SsArgs a = ss_args(SS_PASS);
     const int rows = dv + (mode == SS_MLSTM ? 1 : 0);
-    const dim3 grid(B * H, (rows + SS_COLS - 1) / SS_COLS);
-    const size_t sm = (size_t)(2 * SS_STAGE * d + SS_STAGE * SS_COLS + 3 * SS_STAGE + 1) * sizeof(float);
-#define SS_GO1(T, MODE, DPL)                                                                                           \
+    // four columns a warp where that still leaves a block or more an SM
+    const int nc = d <= 128 && (long long)B * H * ((rows + 4 * SS_COLS - 1) / (4 * SS_COLS)) >= 148 ? 4 : 1;
+    const int cols = SS_COLS * nc;
+    const dim3 grid(B * H, (rows + cols - 1) / cols);
+    const size_t sm = (size_t)(2 * SS_STAGE * d + SS_STAGE * cols + 3 * SS_STAGE + 1) * sizeof(float);
+#define SS_GO1(T, MODE, DPL, NC)                                                                                       \
     do {                                                                                                               \
         if (sm > 48 * 1024)                                                                                            \
-            cudaFuncSetAttribute(k_gated_scan<T, MODE, DPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm);    \
-        kb_launch(k_gated_scan<T, MODE, DPL>, grid, 32 * SS_COLS, sm, st, a);                                          \
+            cudaFuncSetAttribute(k_gated_scan<T, MODE, DPL, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm); \
+        kb_launch(k_gated_scan<T, MODE, DPL, NC>, grid, 32 * SS_COLS, sm, st, a);                                      \
     } while (0)
 #define SS_GO(T, MODE)                                                                                                 \
     do {                                                                                                               \
-        if (d <= 64) SS_GO1(T, MODE, 2);                                                                               \
-        else if (d <= 128) SS_GO1(T, MODE, 4);                                                                         \
-        else if (d <= 256) SS_GO1(T, MODE, 8);                                                                         \
-        else SS_GO1(T, MODE, 16);                                                                                      \
+        if (d <= 64) { if (nc == 4) SS_GO1(T, MODE, 2, 4); else SS_GO1(T, MODE, 2, 1); }                               \
+        else if (d <= 128) { if (nc == 4) SS_GO1(T, MODE, 4, 4); else SS_GO1(T, MODE, 4, 1); }                         \
+        else if (d <= 256) SS_GO1(T, MODE, 8, 1);                                                                      \
+        else SS_GO1(T, MODE, 16, 1);                                                                                   \
     } while (0)
     if (dtype == KB_F32) {
         if (mode == SS_MLSTM) SS_GO(float, SS_MLSTM); else SS_GO(float, SS_MAMBA);
@@ -920,7 +976,8 @@ extern "C" int kb_gated_scan_chunked(SS_PARAMS, int T, float* gates, float* part
                     ((uintptr_t)out % 8 == 0 && ldo % 2 == 0 && dv % 2 == 0 ? 8 : 0) |
                     ((uintptr_t)part % 16 == 0 && d % 4 == 0 ? 16 : 0);
     const size_t sm_a = (size_t)(KB_SPLIT * SS_C * SS_LD + SS_C * (dp + 8)) * 2;
-    const size_t sm_c = (size_t)(KB_SPLIT * SS_E * SS_LD + SS_C * SS_LD + 2 * SS_C * (dp + 8)) * 2;
+    const size_t tile_s = (size_t)KB_SPLIT * SS_E * SS_LD, tile_kv = (size_t)SS_C * SS_LD + (size_t)SS_C * (dp + 8);
+    const size_t sm_c = ((size_t)SS_C * (dp + 8) + (tile_s > tile_kv ? tile_s : tile_kv)) * 2;
     const dim3 grid(runs, H, ez);
     const int n_el = rows * d;
     const bool v4 = n_el % 4 == 0 && (uintptr_t)state % 16 == 0 && state_stride % 4 == 0 && (uintptr_t)part % 16 == 0;
