@@ -88,7 +88,7 @@ __device__ __forceinline__ void ss_gate(const SsArgs& a, int row, int h, float& 
 #define SS_COLS 8
 #define SS_STAGE 16
 template <typename T, int MODE, int DPL, int NC>
-__global__ void __launch_bounds__(32 * SS_COLS, DPL * NC >= 16 ? 2 : 3) k_gated_scan(SsArgs a) {
+__global__ void __launch_bounds__(32 * SS_COLS, DPL * NC > 16 ? 2 : 3) k_gated_scan(SsArgs a) {
     extern __shared__ float sm[];
     const int d = a.d, dv = a.dv, H = a.H;
     float* qs = sm;                                   // [SS_STAGE][d]
