@@ -48,6 +48,74 @@ extern "C" int kb_embed(const void* table, int wdtype, const int* tok, float* x,
     KB_LAUNCH_RET();
 }
 
+// x[t] = table[tok[t]] * scale + pairs[bucket] + positions[pos[t]], in 32-bit. `pairs` (or null): a table over pairs of
+// neighbouring tokens, bucket = (previous token * mul_prev + token * mul_cur) mod buckets in 64-bit, and row `buckets` for a
+// sequence's first token. The previous token of the first row a sequence brings is what its last step left in `last`
+// ([slots], a token id as a float); that row's block reads it and writes the step's own last token there, so no other block
+// needs it. `positions` (or null): a vector per position.
+template <typename TW>
+__global__ void __launch_bounds__(256) k_embed_sum(const TW* __restrict__ table, const TW* __restrict__ pairs,
+        const TW* __restrict__ positions, const int* __restrict__ tok, const int* __restrict__ pos,
+        const int* __restrict__ seq, const int* __restrict__ slot, const int* __restrict__ q_start, float* last,
+        size_t last_stride, long long mul_prev, long long mul_cur, int buckets, int n_pos, float* __restrict__ x, int E,
+        int vocab, float scale, int* status) {
+    __shared__ int s_prev;
+    kb_pdl_launch();
+    kb_pdl_wait();
+    const int t = blockIdx.x, p = pos[t], id = tok[t];
+    float* xr = x + (size_t)t * E;
+    if (p < 0 || id < 0 || id >= vocab || (positions != nullptr && p >= n_pos)) {      // (p < 0: padding of a recorded step)
+        if (threadIdx.x == 0 && p >= 0) atomicOr(status, KB_ST_BAD_TOKEN);
+        for (int i = threadIdx.x; i < E; i += blockDim.x) xr[i] = 0.0f;
+        return;
+    }
+    const TW* prow = nullptr;
+    if (pairs != nullptr) {
+        const int b = seq[t];
+        if (threadIdx.x == 0) {
+            int prev = -1;
+            if (t == q_start[b]) {
+                float* lp = last + (size_t)slot[b] * last_stride;
+                if (p > 0) prev = (int)*lp;
+                *lp = (float)tok[q_start[b + 1] - 1];
+            } else {
+                prev = tok[t - 1];
+            }
+            s_prev = prev;
+        }
+        __syncthreads();
+        long long row = buckets;
+        if (p > 0) {
+            row = ((long long)s_prev * mul_prev + (long long)id * mul_cur) % buckets;
+            if (row < 0) row += buckets;
+        }
+        prow = pairs + (size_t)row * E;
+    }
+    const TW* trow = table + (size_t)id * E;
+    const TW* qrow = positions != nullptr ? positions + (size_t)p * E : nullptr;
+    for (int i = threadIdx.x; i < E; i += blockDim.x) {
+        float v = __fmul_rn(kb_to_f<TW>(trow[i]), scale);
+        if (prow) v += kb_to_f<TW>(prow[i]);
+        if (qrow) v += kb_to_f<TW>(qrow[i]);
+        xr[i] = v;
+    }
+}
+
+extern "C" int kb_embed_sum(const void* table, const void* pairs, const void* positions, int wdtype, const int* tok,
+                            const int* pos, const int* seq, const int* slot, const int* q_start, float* last,
+                            long long last_stride, long long mul_prev, long long mul_cur, int buckets, int n_pos, float* x,
+                            int T, int E, int vocab, float scale, int* status, cudaStream_t st) {
+    if (T <= 0) return 0;
+    if (pairs && (buckets < 1 || !last)) return (int)cudaErrorInvalidValue;
+#define KB_ES(TW)                                                                                                       \
+    kb_launch(k_embed_sum<TW>, T, 256, 0, st, (const TW*)table, (const TW*)pairs, (const TW*)positions, tok, pos, seq,  \
+              slot, q_start, last, (size_t)last_stride, mul_prev, mul_cur, buckets, n_pos, x, E, vocab, scale, status)
+    if (wdtype == KB_F32) KB_ES(float);
+    else KB_ES(bf16);
+#undef KB_ES
+    KB_LAUNCH_RET();
+}
+
 // ------------------------------------------------------------------------------------------------ logits: scale, soft cap
 // z = z * scale, then (cap > 0) z = cap * tanh(z / cap), in place: the options a head part may carry
 __global__ void k_logit_post(float* KB_STEP_DATA z, long long n, float scale, float cap) {

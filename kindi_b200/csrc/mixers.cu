@@ -107,11 +107,37 @@ extern "C" int kb_gated_rmsnorm(const float* x, int ldx, const void* w, int wdty
 //   keys   [normalised latent | rotated part | zeros]      values [normalised latent | zeros]
 // so that attention over the cache with queries [W_uk^T q | rotated q | zeros] gives the scores of the expanded keys,
 // and its output's first kv_rank elements are the weighted sum of latents, from which W_uv makes the heads' values.
-// Rotation: element 2i pairs with 2i + 1; angle = (float)pos * freq[i]; cosine and sine are multiplied by mult.
+// Rotation: pair i is the elements (2i, 2i + 1), or with `half` (i, i + rot / 2); its angle is pos * freq[i], in 32-bit, or in
+// 64-bit where the caller gives 64-bit frequencies (the true 32-bit path); cosine and sine are multiplied by mult.
+struct MxRot {
+    const float* freq;
+    const double* freq64;
+    float mult;
+    int half;
+};
+__device__ __forceinline__ void mx_pair(const MxRot& r, int i, int rot, int& a, int& b) {
+    a = r.half ? i : 2 * i;
+    b = r.half ? i + rot / 2 : 2 * i + 1;
+}
+template <bool EXACT>
+__device__ __forceinline__ void mx_angle(const MxRot& r, int p, int i, float& c, float& s) {
+    if (EXACT && r.freq64 != nullptr) {
+        double s_, c_;
+        sincos((double)p * r.freq64[i], &s_, &c_);
+        c = (float)c_;
+        s = (float)s_;
+    } else {
+        const float ang = __fmul_rn((float)p, r.freq[i]);
+        c = cosf(ang);
+        s = sinf(ang);
+    }
+    c = __fmul_rn(c, r.mult);
+    s = __fmul_rn(s, r.mult);
+}
 template <typename TIN, typename TW, typename T>
 __global__ void __launch_bounds__(256) k_latent_prep(const TIN* KB_STEP_DATA in, int n_planes, size_t plane_stride,
         int ld_in, int q_rank, int kv_rank, int rot, const TW* __restrict__ wq, const TW* __restrict__ wkv, float eps,
-        const float* __restrict__ freq, float mult, const int* __restrict__ pos, const int* __restrict__ seq,
+        MxRot rr, const int* __restrict__ pos, const int* __restrict__ seq,
         const int* __restrict__ slot, T* __restrict__ cq, int ldcq, KbCacheView cv, int* status) {
     __shared__ float red[8];
     kb_pdl_launch();
@@ -154,12 +180,14 @@ __global__ void __launch_bounds__(256) k_latent_prep(const TIN* KB_STEP_DATA in,
         vd[i] = c;
     }
     for (int i = threadIdx.x; i < rot / 2; i += 256) {
-        const float ang = __fmul_rn((float)p, freq[i]);
-        const float c = __fmul_rn(cosf(ang), mult), sn = __fmul_rn(sinf(ang), mult);
-        const float a = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + kv_rank + 2 * i);
-        const float b = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + kv_rank + 2 * i + 1);
-        kd[kv_rank + 2 * i] = kb_from_f<T>(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, sn)));
-        kd[kv_rank + 2 * i + 1] = kb_from_f<T>(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
+        float c, sn;
+        int ia, ib;
+        mx_angle<sizeof(T) == 4>(rr, p, i, c, sn);
+        mx_pair(rr, i, rot, ia, ib);
+        const float a = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + kv_rank + ia);
+        const float b = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + kv_rank + ib);
+        kd[kv_rank + ia] = kb_from_f<T>(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, sn)));
+        kd[kv_rank + ib] = kb_from_f<T>(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
     }
     for (int i = kv_rank + rot + threadIdx.x; i < cv.head_dim; i += 256) kd[i] = kb_from_f<T>(0.0f);
     for (int i = kv_rank + threadIdx.x; i < cv.head_dim; i += 256) vd[i] = kb_from_f<T>(0.0f);
@@ -169,13 +197,14 @@ extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long l
                               int kv_rank, int rot, const void* wq, const void* wkv, int wdtype, float eps,
                               const float* freq, float mult, const int* pos, const int* seq, const int* slot, void* cq,
                               int dtype, int ldcq, int T, int D, void* pool, const int* table, int table_stride,
-                              int n_pages, int* status, cudaStream_t st) {
+                              int n_pages, int* status, cudaStream_t st, const double* freq64, int half) {
     if (T <= 0) return 0;
+    const MxRot rr{freq, freq64, mult, half};
     if (rot % 2 || kv_rank + rot > D) return (int)cudaErrorInvalidValue;
     KbCacheView cv{pool, table, table_stride, n_pages, 1, D};
 #define KB_LP(TIN, TW, T_)                                                                                       \
     kb_launch(k_latent_prep<TIN, TW, T_>, T, 256, 0, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in,  \
-              q_rank, kv_rank, rot, (const TW*)wq, (const TW*)wkv, eps, freq, mult, pos, seq, slot, (T_*)cq, ldcq, \
+              q_rank, kv_rank, rot, (const TW*)wq, (const TW*)wkv, eps, rr, pos, seq, slot, (T_*)cq, ldcq, \
               cv, status)
     if (in_dtype == KB_F32 && dtype == KB_F32 && wdtype == KB_F32) KB_LP(float, float, float);
     else if (in_dtype == KB_F32 && dtype == KB_BF16 && wdtype == KB_BF16) KB_LP(float, bf16, bf16);
@@ -187,12 +216,12 @@ extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long l
     KB_LAUNCH_RET();
 }
 
-// The rotated part of every query head: q[t][h] = [plain (dim) | rotated (rot)] -> out[t][h][at .. at + rot) rotated
-// (interleaved pairs), out[t][h][at + rot .. D) = 0. The first `at` elements of each head are written by the per-head
+// The rotated part of every query head: q[t][h] = [plain (dim) | rotated (rot)] -> out[t][h][at .. at + rot) rotated,
+// out[t][h][at + rot .. D) = 0. The first `at` elements of each head are written by the per-head
 // product below.
 template <typename T>
-__global__ void k_latent_qrope(const T* KB_STEP_DATA q, int ldq, int dim, int rot, const float* __restrict__ freq,
-        float mult, const int* __restrict__ pos, T* __restrict__ out, int ldo, int at, int D) {
+__global__ void k_latent_qrope(const T* KB_STEP_DATA q, int ldq, int dim, int rot, MxRot rr,
+        const int* __restrict__ pos, T* __restrict__ out, int ldo, int at, int D) {
     kb_pdl_launch();
     const int t = blockIdx.x, h = blockIdx.y;
     const int p = pos[t];
@@ -201,11 +230,13 @@ __global__ void k_latent_qrope(const T* KB_STEP_DATA q, int ldq, int dim, int ro
     T* dst = out + (size_t)t * ldo + (size_t)h * D + at;
     if (p >= 0) {
         for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
-            const float ang = __fmul_rn((float)p, freq[i]);
-            const float c = __fmul_rn(cosf(ang), mult), sn = __fmul_rn(sinf(ang), mult);
-            const float a = kb_to_f<T>(src[2 * i]), b = kb_to_f<T>(src[2 * i + 1]);
-            dst[2 * i] = kb_from_f<T>(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, sn)));
-            dst[2 * i + 1] = kb_from_f<T>(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
+            float c, sn;
+            int ia, ib;
+            mx_angle<sizeof(T) == 4>(rr, p, i, c, sn);
+            mx_pair(rr, i, rot, ia, ib);
+            const float a = kb_to_f<T>(src[ia]), b = kb_to_f<T>(src[ib]);
+            dst[ia] = kb_from_f<T>(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, sn)));
+            dst[ib] = kb_from_f<T>(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
         }
     } else {
         for (int i = threadIdx.x; i < rot; i += blockDim.x) dst[i] = kb_from_f<T>(0.0f);
@@ -214,30 +245,32 @@ __global__ void k_latent_qrope(const T* KB_STEP_DATA q, int ldq, int dim, int ro
 }
 
 extern "C" int kb_latent_qrope(const void* q, int dtype, int ldq, int dim, int rot, const float* freq, float mult,
-                               const int* pos, void* out, int ldo, int at, int D, int T, int H, cudaStream_t st) {
+                               const int* pos, void* out, int ldo, int at, int D, int T, int H, cudaStream_t st,
+                               const double* freq64, int half) {
     if (T <= 0 || H <= 0) return 0;
+    const MxRot rr{freq, freq64, mult, half};
     if (rot % 2 || at + rot > D) return (int)cudaErrorInvalidValue;
     dim3 grid(T, H);
     if (dtype == KB_F32)
-        kb_launch(k_latent_qrope<float>, grid, 64, 0, st, (const float*)q, ldq, dim, rot, freq, mult, pos, (float*)out,
+        kb_launch(k_latent_qrope<float>, grid, 64, 0, st, (const float*)q, ldq, dim, rot, rr, pos, (float*)out,
                   ldo, at, D);
     else
-        kb_launch(k_latent_qrope<bf16>, grid, 64, 0, st, (const bf16*)q, ldq, dim, rot, freq, mult, pos, (bf16*)out,
+        kb_launch(k_latent_qrope<bf16>, grid, 64, 0, st, (const bf16*)q, ldq, dim, rot, rr, pos, (bf16*)out,
                   ldo, at, D);
     KB_LAUNCH_RET();
 }
 
 // ------------------------------------------------------------------------------------------------ per-head products
 // out[t][h * ldoh + n] = sum_k a[t][h * ldah + k] * w[h][n][k] (n < N, k < K; w [H][N][K] contiguous), every sum over
-// k = 0, 1, 2, ... in order with 32-bit fused multiply-adds. With gate: out *= sigmoid(gate[t][h * N + n]) (rows or
-// planes). grid.z = head.
+// k = 0, 1, 2, ... in order with 32-bit fused multiply-adds. With gate (rows or planes): out *= sigmoid(gate[t][h * gph +
+// (gph > 1 ? n : 0)]), gph = N for a gate per element and 1 for one number a head. grid.z = head.
 #define HG_BM 64
 #define HG_BN 64
 #define HG_BK 32
 template <typename TA, typename TW, typename TG>
 __global__ void __launch_bounds__(256) k_head_gemm(const TA* KB_STEP_DATA A, int lda, int ldah, const TW* __restrict__ W,
         TA* __restrict__ C, int ldc, int ldch, int M, int N, int K, const TG* KB_STEP_DATA gate, int n_planes,
-        size_t plane_stride, int ldg) {
+        size_t plane_stride, int ldg, int gph) {
     __shared__ float As[HG_BK][HG_BM + 1];
     __shared__ float Ws[HG_BK][HG_BN + 1];
     kb_pdl_launch();
@@ -286,7 +319,7 @@ __global__ void __launch_bounds__(256) k_head_gemm(const TA* KB_STEP_DATA A, int
             if (n >= N) continue;
             float v = acc[i][j];
             if (gate != nullptr)
-                v *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, (size_t)h * N + n));
+                v *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, (size_t)h * gph + (gph > 1 ? n : 0)));
             C[(size_t)m * ldc + (size_t)h * ldch + n] = kb_from_f<TA>(v);
         }
     }
@@ -308,7 +341,7 @@ __device__ __forceinline__ void mx_mma_bf16(float* c, const uint32_t* a, uint32_
 template <typename TG>
 __global__ void __launch_bounds__(128) k_head_gemm_mma(const bf16* KB_STEP_DATA A, int lda, int ldah,
         const bf16* __restrict__ W, bf16* __restrict__ C, int ldc, int ldch, int M, int N, int K,
-        const TG* KB_STEP_DATA gate, int n_planes, size_t plane_stride, int ldg) {
+        const TG* KB_STEP_DATA gate, int n_planes, size_t plane_stride, int ldg, int gph) {
     __shared__ __align__(16) bf16 As[HM_BM * HM_LD];
     __shared__ __align__(16) bf16 Ws[HM_BN * HM_LD];
     kb_pdl_launch();
@@ -359,31 +392,32 @@ __global__ void __launch_bounds__(128) k_head_gemm_mma(const bf16* KB_STEP_DATA 
             if (m >= M || n >= N) continue;
             float v = acc[j][i];
             if (gate != nullptr)
-                v *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, (size_t)h * N + n));
+                v *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, (size_t)h * gph + (gph > 1 ? n : 0)));
             C[(size_t)m * ldc + (size_t)h * ldch + n] = __float2bfloat16_rn(v);
         }
 }
 
 extern "C" int kb_head_gemm(const void* A, int adtype, int lda, int ldah, const void* W, int wdtype, void* C, int ldc,
                             int ldch, int M, int N, int K, int H, const void* gate, int gdtype, int n_planes,
-                            long long plane_stride, int ldg, cudaStream_t st, int tensor_cores) {
+                            long long plane_stride, int ldg, cudaStream_t st, int tensor_cores, int gph) {
     if (M <= 0 || N <= 0 || H <= 0) return 0;
+    if (gate && gph != N && gph != 1) return (int)cudaErrorInvalidValue;
     if (H > 65535) return (int)cudaErrorInvalidValue;
     if (tensor_cores && adtype == KB_BF16 && wdtype == KB_BF16 && K % 8 == 0 && lda % 8 == 0 && ldah % 8 == 0 &&
         ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
         dim3 gm((N + HM_BN - 1) / HM_BN, (M + HM_BM - 1) / HM_BM, H);
         if (gate == nullptr || gdtype == KB_F32)
             kb_launch(k_head_gemm_mma<float>, gm, 128, 0, st, (const bf16*)A, lda, ldah, (const bf16*)W, (bf16*)C, ldc,
-                      ldch, M, N, K, (const float*)gate, n_planes, (size_t)plane_stride, ldg);
+                      ldch, M, N, K, (const float*)gate, n_planes, (size_t)plane_stride, ldg, gph);
         else
             kb_launch(k_head_gemm_mma<bf16>, gm, 128, 0, st, (const bf16*)A, lda, ldah, (const bf16*)W, (bf16*)C, ldc,
-                      ldch, M, N, K, (const bf16*)gate, n_planes, (size_t)plane_stride, ldg);
+                      ldch, M, N, K, (const bf16*)gate, n_planes, (size_t)plane_stride, ldg, gph);
         KB_LAUNCH_RET();
     }
     dim3 grid((N + HG_BN - 1) / HG_BN, (M + HG_BM - 1) / HG_BM, H);
 #define KB_HG(TA, TW, TG)                                                                                       \
     kb_launch(k_head_gemm<TA, TW, TG>, grid, 256, 0, st, (const TA*)A, lda, ldah, (const TW*)W, (TA*)C, ldc,    \
-              ldch, M, N, K, (const TG*)gate, n_planes, (size_t)plane_stride, ldg)
+              ldch, M, N, K, (const TG*)gate, n_planes, (size_t)plane_stride, ldg, gph)
     const bool gf = gate == nullptr || gdtype == KB_F32;
     if (adtype == KB_F32 && wdtype == KB_F32 && gf) KB_HG(float, float, float);
     else if (adtype == KB_BF16 && wdtype == KB_BF16 && gf) KB_HG(bf16, bf16, float);

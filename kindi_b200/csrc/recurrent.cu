@@ -430,7 +430,7 @@ extern "C" int kb_delta_rule(const float* qkv, int ldq, const void* proj, int pd
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(128) k_head_norm_gate(const float* KB_STEP_DATA x, int ldx, int T, int H, int n,
         const float* __restrict__ w, float eps, const TG* KB_STEP_DATA g, int n_planes, size_t plane_stride, int ldg,
-        int og, int gate_kind, TO* __restrict__ out, int ldo) {
+        int og, int gate_kind, TO* __restrict__ out, int ldo, int w_head) {
     kb_pdl_launch();
     kb_pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -444,7 +444,7 @@ __global__ void __launch_bounds__(128) k_head_norm_gate(const float* KB_STEP_DAT
     ss = kb_warp_sum(ss);
     const float f = 1.0f / sqrtf(ss / (float)n + eps);
     for (int e = lane; e < n; e += 32) {
-        float y = __fmul_rn(__fmul_rn(f, xr[e]), w[e]);
+        float y = __fmul_rn(__fmul_rn(f, xr[e]), w[(size_t)h * w_head + e]);
         if (g != nullptr)
             y *= rc_gate(rc_rd<TG>(g + t * ldg, n_planes, plane_stride, (size_t)og + (size_t)h * n + e), gate_kind);
         out[t * ldo + (size_t)h * n + e] = kb_from_f<TO>(y);
@@ -453,12 +453,13 @@ __global__ void __launch_bounds__(128) k_head_norm_gate(const float* KB_STEP_DAT
 
 extern "C" int kb_head_norm_gate(const float* x, int ldx, int T, int H, int n, const float* w, float eps,
                                  const void* g, int gdtype, int n_planes, long long plane_stride, int ldg, int og,
-                                 int gate_kind, void* out, int odtype, int ldo, cudaStream_t st) {
+                                 int gate_kind, void* out, int odtype, int ldo, cudaStream_t st, int w_head) {
+    // w_head: elements between two heads' gains (0: all heads share them)
     if (T <= 0 || H <= 0) return 0;
     const int grid = (int)(((long long)T * H + 3) / 4);
 #define KB_HN(TG, TO)                                                                                              \
     kb_launch(k_head_norm_gate<TG, TO>, grid, 128, 0, st, x, ldx, T, H, n, w, eps, (const TG*)g, n_planes,        \
-              (size_t)plane_stride, ldg, og, gate_kind, (TO*)out, ldo)
+              (size_t)plane_stride, ldg, og, gate_kind, (TO*)out, ldo, w_head)
     if (gdtype == KB_F32 && odtype == KB_F32) KB_HN(float, float);
     else if (gdtype == KB_F32 && odtype == KB_BF16) KB_HN(float, bf16);
     else if (gdtype == KB_BF16 && odtype == KB_BF16) KB_HN(bf16, bf16);

@@ -33,8 +33,20 @@ _SCAN = [c_int, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_int, 
          c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
          c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p]
 
+# the arguments the forms of the recurrence with a decay per channel share (WK_PARAMS in csrc/wkv.cu)
+_WKV = [c_int, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_longlong, c_int,
+        c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong,
+        c_void_p, c_int]
+
 _SIGS = {
     "kb_embed": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
+    "kb_embed_sum": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                     c_longlong, c_longlong, c_longlong, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p,
+                     c_void_p],
+    "kb_token_mix": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                     c_longlong, c_void_p, c_int, c_int, c_void_p],
+    "kb_tanh_rows": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+    "kb_wkv_scan": _WKV + [c_void_p],
     "kb_logit_post": [c_void_p, c_longlong, c_float, c_float, c_void_p],
     "kb_add_rmsnorm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p,
                        c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
@@ -53,11 +65,11 @@ _SIGS = {
                          c_int, c_int, c_int, c_int, c_void_p],
     "kb_latent_prep": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                        c_float, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                       c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+                       c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int],
     "kb_latent_qrope": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
-                        c_int, c_int, c_int, c_void_p],
+                        c_int, c_int, c_int, c_void_p, c_void_p, c_int],
     "kb_head_gemm": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                     c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int],
+                     c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int],
     "kb_decay_chunked": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "kb_decay_scan": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
@@ -81,7 +93,7 @@ _SIGS = {
                          c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
                          c_void_p, c_int, c_void_p, c_int, c_void_p],
     "kb_head_norm_gate": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_longlong,
-                          c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+                          c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int],
     "kb_min_gru": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                    c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p],
     "kb_branch_norm_mean": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
@@ -315,6 +327,25 @@ def embed(table: torch.Tensor, tok: torch.Tensor, out: torch.Tensor, status: tor
                            _stream()), "embed")
 
 
+def embed_sum(table: torch.Tensor, pairs: Optional[torch.Tensor], positions: Optional[torch.Tensor], ctx, last,
+              mul_prev: int, mul_cur: int, out: torch.Tensor, scale: float = 1.0) -> None:
+    """out[t] (float32 [T, E]) = table[tok[t]] * scale + pairs[bucket] + positions[pos[t]] for the rows of the step ``ctx``
+    (None: that term is left out). ``pairs`` [buckets + 1, E]: row (previous token * mul_prev + token * mul_cur) mod buckets,
+    the last row for a sequence's first token; ``last`` (float32 [slots, 1]): every sequence's newest token before the step,
+    rewritten"""
+    _need_cuda(table, pairs, positions, last, out)
+    T, E = out.shape
+    for w in (table, pairs, positions):
+        assert w is None or (w.is_contiguous() and w.dtype == table.dtype and w.shape[1] == E)
+    assert out.is_contiguous() and out.dtype == torch.float32 and ctx.tok.dtype == torch.int32
+    assert pairs is None or (last is not None and last.dtype == torch.float32 and pairs.shape[0] >= 2)
+    _check(load().kb_embed_sum(_p(table), _p(pairs), _p(positions), dt(table), _p(ctx.tok), _p(ctx.pos), _p(ctx.seq),
+                               _p(ctx.slot), _p(ctx.q_start), _p(last), last.stride(0) if last is not None else 0,
+                               int(mul_prev), int(mul_cur), pairs.shape[0] - 1 if pairs is not None else 0,
+                               positions.shape[0] if positions is not None else 0, _p(out), T, E, table.shape[0],
+                               float(scale), _p(ctx.status), _stream()), "embed_sum")
+
+
 def wait_selftest(status: torch.Tensor, limit_ns: int = 1_000_000):
     """run the library's bounded wait on a barrier that nothing arrives at: it gives up after ``limit_ns`` (at most a
     tenth of a second), sets ST_WAIT_TIMEOUT in ``status`` and the kernel ends. Returns (timed out, nanoseconds waited)
@@ -469,14 +500,20 @@ def gated_rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, g: Optional[torc
            "gated_rmsnorm")
 
 
+PAIRING = {"interleaved": 0, "half": 1}
+
+
 def latent_prep(a: torch.Tensor, q_rank: int, kv_rank: int, rot: int, wq: torch.Tensor, wkv: torch.Tensor, eps: float,
                 freq: torch.Tensor, mult: float, pos, seq, slot, cq: torch.Tensor, head_dim: int, pool: torch.Tensor,
-                table: torch.Tensor, n_pages: int, status: torch.Tensor) -> None:
+                table: torch.Tensor, n_pages: int, status: torch.Tensor, pairing: str = "interleaved",
+                freq64: Optional[torch.Tensor] = None) -> None:
     """``a``: rows or 32-bit planes of [query latent | key/value latent | rotated key part | ...]. Writes the RMS-normed
     query latent to ``cq`` and stores, at each row's position of its sequence's pages, one key head [normed latent |
     rotated part | 0] and one value head [normed latent | 0] of ``head_dim`` elements. The rotation pairs element 2i
-    with 2i + 1, by pos * freq[i], cosine and sine times ``mult``"""
-    _need_cuda(a, wq, wkv, freq, cq, pool, table)
+    with 2i + 1 (``pairing`` "half": i with i + rot / 2), by pos * freq[i], cosine and sine times ``mult``; float32 rows
+    take their angles from ``freq64`` (float64) where it is given"""
+    _need_cuda(a, wq, wkv, freq, cq, pool, table, freq64)
+    assert freq64 is None or (freq64.dtype == torch.float64 and freq64.numel() >= rot // 2 and freq64.is_contiguous())
     n_planes, pstride, ld = _planes_of(a)
     T = a.shape[-2]
     assert a.shape[-1] >= q_rank + kv_rank + rot and wq.dtype == wkv.dtype and wq.numel() == q_rank
@@ -487,25 +524,29 @@ def latent_prep(a: torch.Tensor, q_rank: int, kv_rank: int, rot: int, wq: torch.
     _check(load().kb_latent_prep(_p(a), dt(a), n_planes, pstride, ld, q_rank, kv_rank, rot, _p(wq), _p(wkv), dt(wq),
                                  float(eps), _p(freq), float(mult), _p(pos), _p(seq), _p(slot), _p(cq), dt(cq),
                                  cq.stride(0), T, head_dim, _p(pool), _p(table), table.stride(0), n_pages, _p(status),
-                                 _stream()), "latent_prep")
+                                 _stream(), _p(freq64), PAIRING[pairing]), "latent_prep")
 
 
 def latent_qrope(q: torch.Tensor, dim: int, rot: int, freq: torch.Tensor, mult: float, pos, out: torch.Tensor,
-                 at: int, head_dim: int, n_heads: int) -> None:
-    """q rows [T, n_heads (dim + rot)]: each head's last ``rot`` elements, rotated (pairs 2i, 2i + 1), go to
+                 at: int, head_dim: int, n_heads: int, pairing: str = "interleaved",
+                 freq64: Optional[torch.Tensor] = None) -> None:
+    """q rows [T, n_heads (dim + rot)]: each head's last ``rot`` elements, rotated (as in ``latent_prep``), go to
     out[t][h][at : at + rot]; out[t][h][at + rot : head_dim] = 0"""
-    _need_cuda(q, freq, out)
+    _need_cuda(q, freq, out, freq64)
+    assert freq64 is None or (freq64.dtype == torch.float64 and freq64.numel() >= rot // 2 and freq64.is_contiguous())
     T = q.shape[0]
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == out.dtype and q.shape[1] == n_heads * (dim + rot)
     assert out.shape == (T, n_heads * head_dim) and freq.dtype == torch.float32
     _check(load().kb_latent_qrope(_p(q), dt(q), q.stride(0), dim, rot, _p(freq), float(mult), _p(pos), _p(out),
-                                  out.stride(0), at, head_dim, T, n_heads, _stream()), "latent_qrope")
+                                  out.stride(0), at, head_dim, T, n_heads, _stream(), _p(freq64), PAIRING[pairing]),
+           "latent_qrope")
 
 
 def head_gemm(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
               gate: Optional[torch.Tensor] = None, tensor_cores: bool = True) -> None:
     """per head h: out[t][h * out_head_stride + n] = sum_k a[t][h * a_head_stride + k] * w[h][n][k]; w [H, N, K].
-    ``gate`` (rows or 32-bit planes [.., T, H * N]): the result is multiplied by its logistic function. bf16 operands
+    ``gate`` (rows or 32-bit planes [.., T, H * N], or [.., T, H] for one number a head): the result is multiplied by its
+    logistic function. bf16 operands
     whose rows are 16-byte aligned (K, strides multiples of 8) run on the tensor cores unless ``tensor_cores`` is
     False; everything else takes 32-bit multiply-adds in a fixed order"""
     _need_cuda(a, w, out, gate)
@@ -515,10 +556,11 @@ def head_gemm(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.T
     assert a.shape[1] >= (H - 1) * a_head_stride + Kd and out.shape[1] >= (H - 1) * out_head_stride + N
     n_planes, pstride, ldg = _planes_of(gate) if gate is not None else (1, 0, 0)
     if gate is not None:
-        assert gate.shape[-2:] == (M, H * N)
+        assert gate.shape[-2:] in ((M, H * N), (M, H))
     _check(load().kb_head_gemm(_p(a), dt(a), a.stride(0), a_head_stride, _p(w), dt(w), _p(out), out.stride(0),
                                out_head_stride, M, N, Kd, H, _p(gate), dt(gate) if gate is not None else F32, n_planes,
-                               pstride, ldg, _stream(), 1 if tensor_cores else 0), "head_gemm")
+                               pstride, ldg, _stream(), 1 if tensor_cores else 0,
+                               gate.shape[-1] // H if gate is not None else 1), "head_gemm")
 
 
 def decay_scan(a: torch.Tensor, B: int, H: int, d: int, dv: int, decay: torch.Tensor, q_start, slot,
@@ -1028,15 +1070,16 @@ def delta_rule(qkv: torch.Tensor, proj: torch.Tensor, ob: int, oa: int, a_log: t
 def head_norm_gate(x: torch.Tensor, H: int, n: int, w: torch.Tensor, eps: float, g: Optional[torch.Tensor], og: int,
                    gate: str, out: torch.Tensor) -> None:
     """out[t][h n + e] = x[t][h n + e] / sqrt(mean_e x^2 + eps) * w[e] * gate(g[t][og + h n + e]); x float32 [T, H n],
-    w float32 [n], ``g`` rows or 32-bit planes, ``gate``: none, sigmoid or silu"""
+    w float32 [n] shared by the heads, or [H n], ``g`` rows or 32-bit planes, ``gate``: none, sigmoid or silu"""
     _need_cuda(x, w, g, out)
     T = x.shape[0]
     assert x.dtype == torch.float32 and x.stride(1) == 1 and x.shape[1] == H * n and w.dtype == torch.float32
-    assert w.numel() == n and w.is_contiguous() and out.shape == (T, H * n) and out.stride(1) == 1
+    assert w.numel() in (n, H * n) and w.is_contiguous() and out.shape == (T, H * n) and out.stride(1) == 1
     n_planes, pstride, ldg = _planes_of(g) if g is not None else (1, 0, 0)
     _check(load().kb_head_norm_gate(_p(x), x.stride(0), T, H, n, _p(w), float(eps), _p(g),
                                     dt(g) if g is not None else F32, n_planes, pstride, ldg, og, GATE_KIND[gate],
-                                    _p(out), dt(out), out.stride(0), _stream()), "head_norm_gate")
+                                    _p(out), dt(out), out.stride(0), _stream(), n if w.numel() == H * n and H > 1 else 0),
+           "head_norm_gate")
 
 
 MIN_GRU_CHUNK = 64          # rows of a chunk (MG_CHUNK of the kernel)
@@ -1358,6 +1401,62 @@ def scan_norm(kind: str, x: torch.Tensor, groups: int, w: torch.Tensor, eps: flo
                                n_planes, pstride, ldg, og, _p(nq), _p(m_rows), _p(m_state),
                                m_state.stride(0) if m_state is not None else 0, _p(pos), _p(seq), _p(slot), _p(q_start),
                                _p(out), dt(out), out.stride(0), _stream()), "scan_norm")
+
+
+# ------------------------------------------------------------------------------- matrix states with a decay per channel
+def token_mix(y: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, ctx, out: torch.Tensor) -> None:
+    """out[t] = [y[t] + (y' - y[t]) * mu[s] for every stream s], y' the row before of the same sequence (``last``, float32
+    [slots, E], for the first row a sequence brings; rewritten with its last row). ``mu`` float32 [n, E], out [T, n E]"""
+    _need_cuda(y, mu, last, out)
+    T, E = y.shape
+    n = mu.shape[0]
+    assert y.is_contiguous() and mu.dtype == last.dtype == torch.float32 and mu.is_contiguous() and mu.shape == (n, E)
+    assert last.stride(1) == 1 and last.shape[1] == E and out.shape == (T, n * E) and out.is_contiguous()
+    assert out.dtype == y.dtype
+    _check(load().kb_token_mix(_p(y), dt(y), E, _p(mu), n, _p(ctx.pos), _p(ctx.seq), _p(ctx.slot), _p(ctx.q_start), _p(last),
+                               last.stride(0), _p(out), out.stride(0), T, _stream()), "token_mix")
+
+
+def tanh_rows(a: torch.Tensor, out: torch.Tensor) -> None:
+    """out = tanh(a); rows [T, N]"""
+    _need_cuda(a, out)
+    T, N = out.shape
+    assert a.shape == (T, N) and a.stride(1) == 1 and out.is_contiguous() and a.dtype == out.dtype
+    _check(load().kb_tanh_rows(_p(a), dt(a), a.stride(0), _p(out), T, N, _stream()), "tanh_rows")
+
+
+def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: Optional[torch.Tensor], low: Optional[torch.Tensor],
+        w2: Optional[torch.Tensor], w0: torch.Tensor, u: torch.Tensor, B: int, H: int, d: int, dv: int, q_start, slot,
+        state: torch.Tensor, out: torch.Tensor) -> None:
+    """``o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t``, ``S_t = diag(w_t) S_(t-1) + k_t v_t^T`` over the packed rows of ``B``
+    sequences, H heads of ``d`` key channels and ``dv`` values. ``r``, ``k``, ``v``: rows or 32-bit planes of one dtype and
+    layout. ``w_t = exp(-exp(z_t + w0))``: ``z`` float32 rows [T, H d], or None, and then ``z = w2 tanh(low)`` is made by the
+    kernel from ``low`` (rows or planes [.., T, rank]) and ``w2`` [H d, rank]. ``w0``, ``u`` float32 [H d]; ``state``
+    float32 [slots, H, dv, d], read and written; ``out`` float32 [T, H dv]"""
+    _need_cuda(r, k, v, z, low, w2, w0, u, state, out)
+    n_planes, pstride, ld = _planes_of(r)
+    for t in (k, v):
+        assert t.dtype == r.dtype and _planes_of(t) == (n_planes, pstride, ld)
+    assert r.shape[-1] == k.shape[-1] == H * d and v.shape[-1] == H * dv and r.shape[-2] == out.shape[0]
+    for t in (w0, u):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() == H * d
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dv, d)
+    assert out.dtype == torch.float32 and out.stride(1) == 1 and out.shape[1] == H * dv
+    lp, ls, ldl, rank = 1, 0, 0, 0
+    if z is not None:
+        assert z.dtype == torch.float32 and z.stride(1) == 1 and z.shape == (out.shape[0], H * d)
+    else:
+        rank = w2.shape[1]
+        assert low.dtype == r.dtype and low.shape[-2:] == (out.shape[0], rank) and w2.shape == (H * d, rank)
+        assert w2.is_contiguous()
+        lp, ls, ldl = _planes_of(low)
+    if d > 256 or rank > 512:
+        raise KernelError("kindi_b200: the recurrence with a decay per channel takes heads of up to 256 channels and low-rank "
+                          "projections of up to 512, found %d and %d" % (d, rank))
+    _check(load().kb_wkv_scan(dt(r), _p(r), _p(k), _p(v), n_planes, pstride, ld, _p(z), z.stride(0) if z is not None else 0,
+                              _p(low) if z is None else None, lp, ls, ldl, _p(w2) if z is None else None,
+                              dt(w2) if z is None else F32, rank, _p(w0), _p(u), B, H, d, dv, _p(q_start), _p(slot), _p(state),
+                              state.stride(0), _p(out), out.stride(0), _stream()), "wkv_scan")
 
 
 def cast_rows(x: torch.Tensor, y: torch.Tensor) -> None:

@@ -102,3 +102,25 @@ def gate_up_glu_clamp(ctx, y: torch.Tensor, wgu: torch.Tensor, group: int, f: in
     gu = rows_or_planes(ctx, y, wgu, out_dtype)
     K.glu_clamp(gu, h, group, limit, alpha)
     return h
+
+
+# ----------------------------------------------------------------------------------------------- several inputs at once
+class GroupedWeight:
+    """matrices ``[n_i, K]`` of one dtype that each multiply an input of their own, kept one below the other (``joined``)"""
+
+    def __init__(self, ws):
+        self.sizes = tuple(int(w.shape[0]) for w in ws)
+        self.k = int(ws[0].shape[1])
+        self.joined = torch.cat(list(ws), dim=0).contiguous()
+
+    def parts(self):
+        at = 0
+        for n in self.sizes:
+            yield self.joined[at:at + n]
+            at += n
+
+
+def grouped_rows_or_planes(ctx, a: torch.Tensor, gw: GroupedWeight, out_dtype: torch.dtype):
+    """the products ``a_i @ w_i^T`` of the inputs ``a = [a_0 | a_1 | ...]`` (``[M, n K]``) with the matrices of ``gw``, as a list
+    in the form of ``rows_or_planes``; results of matrices of one size are laid out alike"""
+    return [rows_or_planes(ctx, a[:, i * gw.k:(i + 1) * gw.k], w, out_dtype) for i, w in enumerate(gw.parts())]

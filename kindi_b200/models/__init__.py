@@ -5,3 +5,4 @@ from . import nilatar       # noqa: F401
 from . import medodra       # noqa: F401
 from . import luzerax       # noqa: F401
 from . import zebovik       # noqa: F401
+from . import basitar       # noqa: F401

@@ -157,9 +157,15 @@ class Norm(Part):
 
 
 class Embedding(Part):
-    """token ids to the 32-bit residual stream. Its tensors are named in full by its spec (no prefix)."""
+    """token ids to the 32-bit residual stream. Its tensors are named in full by its spec (no prefix). A part with state per
+    sequence (``cache_need`` not None) owns the cache entry after the schedule's, ``cache_entry``, which the model sets."""
 
     category = "embedding"
+    cache_entry = None
+
+    @classmethod
+    def cache_need(cls, spec: PartSpec, width: int):
+        return None
 
     def forward(self, ctx: StepContext) -> torch.Tensor:
         """32-bit ``[T, width]`` rows of the step's tokens (``ctx.tok``)"""

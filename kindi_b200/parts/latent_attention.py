@@ -8,7 +8,8 @@ With ``y`` the mixer's input, H heads, per head ``dim`` plain and ``rot_dim`` ro
 * ``W_dkv y`` has ``kv_rank + rot_dim`` rows: ``c = rms(first kv_rank) * g_kv`` is the latent, the last ``rot_dim``
   (not normalised) are ONE rotated key part shared by all heads;
 * head h: keys ``[W_uk_h c | rotated part]``, values ``W_uv_h c``; score ``(q_plain . k_plain + q_rot . k_rot) * scale``;
-  causal softmax; the concatenated heads times ``sigmoid(W_g y)`` (optional gate), then ``W_o``.
+  causal softmax; the concatenated heads times ``sigmoid(W_g y)`` (optional gate: a number per element, or with
+  ``head_gate`` one number per head), then ``W_o``.
 
 What runs is the absorbed form, the same arithmetic re-associated: ``q_plain . (W_uk_h c) = (W_uk_h^T q_plain) . c``
 and ``sum_j p_j W_uv_h c_j = W_uv_h (sum_j p_j c_j)``. So the cache holds, per position, ONE key/value head: keys
@@ -20,8 +21,8 @@ are the same code, and nothing is expanded per cached position. The rotation is 
 frequencies, pairing and factor on cosines and sines: see ``parts/rope.py``), applied by the latent kernels.
 
 Parameters: ``n_heads``, ``head_dim`` (plain), ``rot_dim``, ``v_head_dim``, ``q_rank``, ``kv_rank``, ``scale``, ``eps``,
-``position`` (a rotation of ``rot_dim`` dimensions), ``names`` (tensor suffixes: ``dq``, ``dq_norm``, ``uq``, ``dkv``,
-``dkv_norm``, ``uk``, ``uv``, ``o``, and ``gate`` or None).
+``position`` (a rotation of ``rot_dim`` dimensions, either pairing), ``names`` (tensor suffixes: ``dq``, ``dq_norm``, ``uq``, ``dkv``,
+``dkv_norm``, ``uk``, ``uv``, ``o``, and ``gate`` or None), ``head_gate`` (the gate has a row per head).
 """
 from __future__ import annotations
 
@@ -35,6 +36,7 @@ from ..kernels import attention as A
 from ..kernels import lib as K
 from ..kernels import linear as L
 from .base import Branch, KVNeed, Mixer, StepContext, WeightView
+from .gated_delta import pad_rows
 
 _DEFAULT_NAMES = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk",
                   "uv": "uv", "o": "o", "gate": None}
@@ -67,7 +69,7 @@ class LatentAttention(Mixer):
         out = {n["dq"]: (qr, width), n["dq_norm"]: (qr,), n["uq"]: (H * (d + r), qr), n["dkv"]: (kr + r, width),
                n["dkv_norm"]: (kr,), n["uk"]: (H * d, kr), n["uv"]: (H * dv, kr), n["o"]: (width, H * dv)}
         if n["gate"]:
-            out[n["gate"]] = (H * dv, width)
+            out[n["gate"]] = (H if spec.get("head_gate") else H * dv, width)
         return out
 
     @classmethod
@@ -93,17 +95,14 @@ class LatentAttention(Mixer):
         if self.position.rotary_dim != self.r:
             raise ValueError("the position part rotates %d dimensions, the mixer's rotated part has %d"
                              % (self.position.rotary_dim, self.r))
-        if self.r and self.position.pairing != "interleaved":
-            raise ValueError("latent attention rotates interleaved pairs; the position part pairs %r"
-                             % self.position.pairing)
         n = self._names(spec)
         ws = [weights(n["dq"]), weights(n["dkv"])]
-        self.has_gate = bool(n["gate"])
-        if self.has_gate:
+        self.gate_rows = 0 if not n["gate"] else self.H if spec.get("head_gate") else self.H * self.dv
+        if self.gate_rows:
             ws.append(weights(n["gate"]))
         if len({w.dtype for w in ws}) != 1:
             raise ValueError("the down projections of %s are stored in different dtypes" % weights.prefix)
-        self.w_down = torch.cat(ws, dim=0).contiguous()          # [q latent | kv latent | rotated part | gate]
+        self.w_down = pad_rows(torch.cat(ws, dim=0))             # [q latent | kv latent | rotated part | gate]
         self.g_q, self.g_kv = weights(n["dq_norm"]).contiguous(), weights(n["dkv_norm"]).contiguous()
         self.w_uq = weights(n["uq"])
         # per head: W_uk_h^T as [kv_rank, dim] (rows = outputs of the absorbing product), W_uv_h as stored
@@ -117,16 +116,18 @@ class LatentAttention(Mixer):
         a = L.rows_or_planes(ctx, y, self.w_down, self.dtype)
         cq = torch.empty((ctx.T, qr), dtype=self.dtype, device=y.device)
         pos = self.position
+        turn = dict(pairing=pos.pairing, freq64=pos.inv_freq64 if self.dtype == torch.float32 else None)
         K.latent_prep(a, qr, kr, r, self.g_q, self.g_kv, self.eps, pos.inv_freq, pos.mult, ctx.pos, ctx.seq, ctx.slot,
-                      cq, D, pool, table, n_pages, ctx.status)
+                      cq, D, pool, table, n_pages, ctx.status, **turn)
         q = L.linear(ctx, cq, self.w_uq, self.dtype)
         qf = torch.empty((ctx.T, H * D), dtype=self.dtype, device=y.device)
         K.head_gemm(q, d + r, self.w_uk_t, qf, D)
-        K.latent_qrope(q, d, r, pos.inv_freq, pos.mult, ctx.pos, qf, kr, D, H)
+        K.latent_qrope(q, d, r, pos.inv_freq, pos.mult, ctx.pos, qf, kr, D, H, **turn)
         att = torch.empty((ctx.T, H * D), dtype=self.dtype, device=y.device)
         A.attention(ctx, qf, att, H, 1, D, self.scale, 0, pool, table, n_pages)
         o = torch.empty((ctx.T, H * dv), dtype=self.dtype, device=y.device)
-        K.head_gemm(att, D, self.w_uv, o, dv, gate=a[..., qr + kr + r:] if self.has_gate else None)
+        at = qr + kr + r
+        K.head_gemm(att, D, self.w_uv, o, dv, gate=a[..., at:at + self.gate_rows] if self.gate_rows else None)
         return Branch(L.planes(ctx, o, self.w_o))
 
     def bytes_read(self) -> int:

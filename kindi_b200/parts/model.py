@@ -54,13 +54,15 @@ def tensor_inits(spec: ModelSpec) -> Dict[str, str]:
 
 
 def cache_needs(spec: ModelSpec) -> List:
-    """the cache need of each cache entry (index = ScheduleEntry.cache)"""
+    """the cache need of each cache entry (index = ScheduleEntry.cache); an embedding part with state of its own has one
+    more, the last"""
     needs: List = [None] * spec.n_cache_entries
     for e in spec.schedule:
         if e.reads_cache_of is None:
             layer = spec.layers[e.layer]
             needs[e.cache] = part_class("block", layer.block.kind).cache_need(layer.block, spec.width)
-    return needs
+    own = part_class("embedding", spec.embedding.kind).cache_need(spec.embedding, spec.width)
+    return needs if own is None else needs + [own]
 
 
 class DecoderModel:
@@ -73,6 +75,7 @@ class DecoderModel:
             return part_class(category, ps.kind)(ps, spec.width, WeightView(tensors, prefix), dtype=dtype,
                                                  device=device)
         self.embedding = make("embedding", spec.embedding, "")
+        self.embedding.cache_entry = spec.n_cache_entries
         self.blocks = [make("block", l.block, l.prefix) for l in spec.layers]
         self.final_norm = make("norm", spec.final_norm, spec.final_norm_prefix)
         self.head = make("head", spec.head, "")
@@ -84,8 +87,11 @@ class DecoderModel:
         returns 32-bit logits ``[len(rows), vocab]`` of the listed rows, or None when no row is wanted"""
         x = self.embedding.forward(ctx)
         # a schedule that feeds the embedding output in again needs it as it was: the norms update x in place
-        x0 = self.embedding.forward(ctx) if any(e.add_embedding or e.mix_embedding is not None
-                                                for e in self.spec.schedule) else None
+        # (taken as a copy where the part has state, which one forward a step moves on)
+        x0 = None
+        if any(e.add_embedding or e.mix_embedding is not None for e in self.spec.schedule):
+            stateful = self.embedding.cache_need(self.spec.embedding, self.spec.width) is not None
+            x0 = x.clone() if stateful else self.embedding.forward(ctx)
         pending: Optional[Branch] = None
         for entry in self.spec.schedule:
             if pending is not None and pending.norm is not None and (entry.mix_embedding is not None or entry.add_embedding):
