@@ -42,7 +42,8 @@ struct TcSmem {
 template <int BN, int STAGES, bool SWAP, typename TC, int MT = 1>
 __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ CUtensorMap mapP,
         const __grid_constant__ CUtensorMap mapQ, TC* __restrict__ C, int rowsP, int rowsQ, int K, int ldc,
-        long long split_stride, int kb_per_split, int n_splits, int* status, int swiglu_ld, KbGate gate_act) {
+        long long split_stride, int kb_per_split, int n_splits, int* status, int swiglu_ld, KbGate gate_act, int grp_tiles,
+        int grp_k) {
     using S = TcSmem<BN, STAGES, MT, SWAP>;
     static_assert(MT == 1 || (!SWAP && 2 * BN <= 512), "two row tiles: prefill form, both accumulators in tensor memory");
     extern __shared__ uint8_t smem_raw[];
@@ -93,11 +94,13 @@ __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ 
             // CTAs take the memory system from the small kernel that is still running.)
             constexpr int EARLY = SWAP ? TC_EARLY : 0;
             bool waited = EARLY == 0;
-            int pend_kb[EARLY + 1], pend_tq[EARLY + 1], n_pend = 0;
+            int pend_x[EARLY + 1], pend_tq[EARLY + 1], n_pend = 0;
             if (waited) kb_pdl_wait();
             for (int u = blockIdx.x; u < n_units && ok; u += gridDim.x) {
                 const int tp = u % tilesP, rest = u / tilesP, tq = rest % tilesQ, sp = rest / tilesQ;
                 const int kb0 = sp * kb_per_split, kb1 = min(total_kb, kb0 + kb_per_split);
+                // (decode form: every group of weight tiles reads an input of its own, grp_k columns further)
+                const int xg = SWAP && grp_tiles > 0 ? tp / grp_tiles * grp_k : 0;
                 for (int kb = kb0; kb < kb1; kb++, n++) {
                     const int s = n % STAGES;
                     const uint32_t ph = (n / STAGES) & 1u;
@@ -105,7 +108,7 @@ __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ 
                         kb_pdl_wait();
                         waited = true;
                         for (int j = 0; j < n_pend; j++)
-                            tma_load_2d(sbase + j * S::STAGE_BYTES + S::A_BYTES, &mapQ, pend_kb[j] * TC_BK,
+                            tma_load_2d(sbase + j * S::STAGE_BYTES + S::A_BYTES, &mapQ, pend_x[j],
                                         pend_tq[j] * BN, bar_full + j * 8);
                     }
                     if (!(ok = mbar_wait(bar_empty + s * 8, ph ^ 1u, status))) break;
@@ -116,9 +119,9 @@ __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ 
                         tma_load_2d(dst + m * (TC_BM * TC_BK * 2), &mapP, kb * TC_BK, (tp * MT + m) * TC_BM,
                                     bar_full + s * 8);
                     if (waited) {
-                        tma_load_2d(dst + S::A_BYTES, &mapQ, kb * TC_BK, tq * BN, bar_full + s * 8);
+                        tma_load_2d(dst + S::A_BYTES, &mapQ, xg + kb * TC_BK, tq * BN, bar_full + s * 8);
                     } else {
-                        pend_kb[n_pend] = kb;                // stage n_pend == s here: the ring has not wrapped yet
+                        pend_x[n_pend] = xg + kb * TC_BK;                // stage n_pend == s here: the ring has not wrapped yet
                         pend_tq[n_pend] = tq;
                         n_pend++;
                     }
@@ -127,8 +130,7 @@ __global__ void __launch_bounds__(TC_THREADS) k_gemm_tc(const __grid_constant__ 
             if (!waited) {
                 kb_pdl_wait();
                 for (int j = 0; j < n_pend; j++)
-                    tma_load_2d(sbase + j * S::STAGE_BYTES + S::A_BYTES, &mapQ, pend_kb[j] * TC_BK, pend_tq[j] * BN,
-                                bar_full + j * 8);
+                    tma_load_2d(sbase + j * S::STAGE_BYTES + S::A_BYTES, &mapQ, pend_x[j], pend_tq[j] * BN, bar_full + j * 8);
             }
         }
     } else if (warp == 1) {
@@ -319,7 +321,8 @@ static int kb_sm_count() {
 
 template <int BN, int STAGES, bool SWAP, typename TC, int MT = 1>
 static int launch_tc(const CUtensorMap& mp, const CUtensorMap& mq, void* C, int rowsP, int rowsQ, int K, int ldc,
-                     int splits, long long split_stride, int* status, cudaStream_t st, int swiglu_ld, KbGate gate_act) {
+                     int splits, long long split_stride, int* status, cudaStream_t st, int swiglu_ld, KbGate gate_act,
+                     int grp_tiles = 0, int grp_k = 0) {
     using S = TcSmem<BN, STAGES, MT, SWAP>;
     auto kern = k_gemm_tc<BN, STAGES, SWAP, TC, MT>;
     static char once_tag;               // one per instantiation: the opt-in is per (device, kernel)
@@ -334,7 +337,7 @@ static int launch_tc(const CUtensorMap& mp, const CUtensorMap& mq, void* C, int 
     const int grid = units < kb_sm_count() ? units : kb_sm_count();
     if (swiglu_ld > 0 && (SWAP || BN % 32 || sizeof(TC) != 2 || z != 1)) return (int)cudaErrorInvalidValue;
     kb_launch(kern, grid, TC_THREADS, S::TOTAL, st, mp, mq, (TC*)C, rowsP, rowsQ, K, ldc, split_stride, kbps, z, status,
-              swiglu_ld, gate_act);
+              swiglu_ld, gate_act, grp_tiles, grp_k);
     return (int)cudaGetLastError();
 }
 
@@ -595,7 +598,11 @@ extern "C" int kb_gemm_tc_splits(int K, int wanted) {
 extern "C" int kb_gemm_tc(const void* A, const void* W, void* C, int cdtype, int M, int N, int K, int lda, int ldw,
                           int ldc, int swap, int bn, int splits, long long split_stride, int* status,
                           cudaStream_t st, int swiglu = 0, int mt = 1, float act_lim = 0.0f, float act_alpha = 0.0f,
-                          const float* bias = nullptr, int post = -1) {
+                          const float* bias = nullptr, int post = -1, int grp_rows = 0) {
+    // grp_rows > 0 (decode form, a multiple of 128; K a multiple of 64): W's rows g grp_rows .. multiply an input of their
+    // own, columns g K .. of A, whose rows hold ceil(N / grp_rows) K elements
+    const int groups = grp_rows > 0 ? (N + grp_rows - 1) / grp_rows : 1;
+    if (grp_rows && (!swap || grp_rows % TC_BM || K % TC_BK)) return (int)cudaErrorInvalidValue;
     // post >= 0 (bf16 out, no swiglu): C = act(. + bias), post the activation's code, bias float [N] or null
     if (mt != 1 && (mt != 2 || swap || splits != 1)) return (int)cudaErrorInvalidValue;
     if (swiglu && (swap || (N % 32) || cdtype != KB_BF16 || splits != 1 || (ldc % 8) || ((uintptr_t)C & 15)))
@@ -614,12 +621,13 @@ extern "C" int kb_gemm_tc(const void* A, const void* W, void* C, int cdtype, int
     const void* Q = swap ? A : W;
     const int rowsP = swap ? N : M, rowsQ = swap ? M : N;
     const int ldp = swap ? ldw : lda, ldq = swap ? lda : ldw;
+    const int grp_tiles = grp_rows / TC_BM;
     if ((rc = kb_make_map_bf16(&mp, P, rowsP, K, ldp, TC_BM))) return rc;
-    if ((rc = kb_make_map_bf16(&mq, Q, rowsQ, K, ldq, bn))) return rc;
+    if ((rc = kb_make_map_bf16(&mq, Q, rowsQ, (uint64_t)groups * K, ldq, bn))) return rc;
 #define TC_GO(BN, ST, SW)                                                                                         \
     return cdtype == KB_F32                                                                                       \
-               ? launch_tc<BN, ST, SW, float>(mp, mq, C, rowsP, rowsQ, K, ldc, splits, split_stride, status, st, swiglu_ld, gate_act)  \
-               : launch_tc<BN, ST, SW, bf16>(mp, mq, C, rowsP, rowsQ, K, ldc, splits, split_stride, status, st, swiglu_ld, gate_act)
+               ? launch_tc<BN, ST, SW, float>(mp, mq, C, rowsP, rowsQ, K, ldc, splits, split_stride, status, st, swiglu_ld, gate_act, grp_tiles, K)  \
+               : launch_tc<BN, ST, SW, bf16>(mp, mq, C, rowsP, rowsQ, K, ldc, splits, split_stride, status, st, swiglu_ld, gate_act, grp_tiles, K)
     if (swap) {
         switch (bn) {
             case 16: TC_GO(16, 8, true);

@@ -23,6 +23,7 @@
 // (padding of a recorded step) are not touched.
 #include "sm100.cuh"
 #include "mma_sync.cuh"
+#include "runs.cuh"
 #include <math.h>
 
 #define SS_MLSTM 0
@@ -265,30 +266,12 @@ __global__ void __launch_bounds__(SG_T) k_scan_gates(SsArgs a, float* __restrict
 }
 
 // ------------------------------------------------------------------------------------------------ runs of long prompts
-// Run ci of sequence b is number q_start[b] / SS_C + b + ci among all runs of the step: the numbers of different sequences
-// do not meet, and there are at most T / SS_C + B of them.
 #define SS_C 64
 #define SS_E 64                 // state columns (values) of a block
 #define SS_LD 72                // row of a 64-wide bf16 tile in shared memory
 #define SS_THREADS 128
 
-struct SsRun {
-    int b, r0, n;               // the sequence, its first row of the run, the run's rows (0: no such run)
-};
-__device__ __forceinline__ SsRun ss_run(const SsArgs& a, int run) {
-    int lo = 0, hi = a.B - 1;
-    while (lo < hi) {
-        const int mid = (lo + hi + 1) >> 1;
-        if (a.q_start[mid] / SS_C + mid <= run) lo = mid;
-        else hi = mid - 1;
-    }
-    SsRun r;
-    r.b = lo;
-    const int ci = run - (a.q_start[lo] / SS_C + lo);
-    r.r0 = a.q_start[lo] + ci * SS_C;
-    r.n = max(0, min(SS_C, a.q_start[lo + 1] - r.r0));
-    return r;
-}
+__device__ __forceinline__ KbRun ss_run(const SsArgs& a, int run) { return kb_find_run(a.q_start, a.B, SS_C, run); }
 // rows of bf16 from global into a padded tile [SS_C][dst_ld]; columns from d to dp and rows from n on are zero. Whole 16-byte
 // words go by asynchronous copies: the caller waits for them (cp_async_wait_all) before its barrier
 __device__ __forceinline__ void ss_tile(bf16* dst, int dst_ld, const bf16* src, int ld, int n, int d, int dp, bool vec) {
@@ -334,7 +317,7 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_state(SsArgs a, const floa
     bf16* ks = vw + KB_SPLIT * SS_C * SS_LD;           // [SS_C][kld]
     __shared__ float lg[SS_C], wt[SS_C];
     kb_pdl_launch();
-    const SsRun r = ss_run(a, blockIdx.x);
+    const KbRun r = ss_run(a, blockIdx.x);
     kb_pdl_wait();
     if (r.n <= 0) return;
     const int h = blockIdx.y, e0 = blockIdx.z * SS_E;
@@ -510,7 +493,7 @@ __global__ void __launch_bounds__(SS_THREADS) k_chunk_out(SsArgs a, const float*
     bf16* ks = vs + SS_C * SS_LD;                      // [SS_C][kld]
     __shared__ float lg[SS_C], wt[SS_C];
     kb_pdl_launch();
-    const SsRun r = ss_run(a, blockIdx.x);
+    const KbRun r = ss_run(a, blockIdx.x);
     kb_pdl_wait();
     if (r.n <= 0) return;
     const int h = blockIdx.y, e0 = blockIdx.z * SS_E;

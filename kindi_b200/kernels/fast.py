@@ -201,6 +201,36 @@ def gemm_planes(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor) -> Optio
     return out
 
 
+def gemm_planes_grouped(a: torch.Tensor, w: torch.Tensor, group_rows: int, status: torch.Tensor) -> Optional[torch.Tensor]:
+    """a decode-sized step's products of several inputs with a matrix each, in one launch: every ``group_rows`` rows of ``w``
+    multiply columns of ``a`` of their own. 32-bit planes [S, M, N], or None: not taken"""
+    (m, _), (n, k) = a.shape, w.shape
+    if m > SMALL_M or group_rows % 128 or k % 64 or not _tc_ok(a, w):
+        return None
+    bn = _swap_bn(m)
+    want = _splits_for(m, n, k, bn)
+    out = torch.empty((K.gemm_tc_splits(k, want), m, n), dtype=torch.float32, device=a.device)
+    K.gemm_tc(a, w, out, swap=True, bn=bn, splits=want, status=status, group_rows=group_rows)
+    return out
+
+
+NARROW_N = 128              # up to this many columns a prompt-sized product of any number of rows may split K
+
+
+def gemm_narrow_planes(a: torch.Tensor, w: torch.Tensor, status: torch.Tensor) -> Optional[torch.Tensor]:
+    """a prompt-sized product of few columns as 32-bit planes: its few tiles leave most SMs idle unless K is split. None: not
+    taken"""
+    (m, k), n = a.shape, w.shape[0]
+    if m <= SMALL_M or n > NARROW_N or not _tc_ok(a, w):
+        return None
+    bn = 64 if n <= 64 else 128
+    tiles = -(-m // 128)
+    want = max(1, min(8, N_SM // tiles, -(-k // 64) // 4))
+    out = torch.empty((K.gemm_tc_splits(k, want), m, n), dtype=torch.float32, device=a.device)
+    K.gemm_tc(a, w, out, swap=False, bn=bn, splits=want, status=status)
+    return out
+
+
 def gemm_swiglu_rows(a: torch.Tensor, w_grouped: torch.Tensor, out: torch.Tensor, status: torch.Tensor,
                      act: str = "silu", act_params=None) -> bool:
     """out (bf16 [M, F]) = silu(g) * u for a prompt-sized step, finished inside the product's epilogue; w_grouped

@@ -45,8 +45,10 @@ _SIGS = {
                      c_void_p],
     "kb_token_mix": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                      c_longlong, c_void_p, c_int, c_int, c_void_p],
-    "kb_tanh_rows": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+    "kb_tanh_rows": [c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "kb_wkv_scan": _WKV + [c_void_p],
+    "kb_wkv_runs": _WKV + [c_int, c_void_p, c_void_p, c_void_p],
+    "kb_wkv_run": [],
     "kb_logit_post": [c_void_p, c_longlong, c_float, c_float, c_void_p],
     "kb_add_rmsnorm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p,
                        c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p],
@@ -120,7 +122,7 @@ _SIGS = {
                     c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "kb_swiglu": [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int],
     "kb_gemm_tc": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                   c_longlong, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_int],
+                   c_longlong, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_int, c_int],
     "kb_gemm_tc_splits": [c_int, c_int],
     "kb_rope_table_min_rows": [],
     "kb_gemm_pair": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
@@ -210,7 +212,8 @@ class KernelTiming:
     def __getattr__(self, name):                       # stands in for the library while timing is on
         fn = getattr(_lib, name)
         if not name.startswith("kb_") or name in ("kb_set_pdl", "kb_gemm_tc_splits", "kb_rope_table_min_rows",
-                                                  "kb_moe_gemm_tile", "kb_moe_gemm_tc_tile", "kb_scan_run"):
+                                                  "kb_moe_gemm_tile", "kb_moe_gemm_tc_tile", "kb_scan_run",
+                                                  "kb_wkv_run"):
             return fn
 
         def timed(*args):
@@ -824,17 +827,20 @@ def _post_args(post, n: int, out: torch.Tensor, swiglu: bool):
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swap: bool, bn: int, splits: int,
             status: torch.Tensor, swiglu: bool = False, mt: int = 1, act: str = "silu", act_params=None,
-            post=None) -> None:
+            post=None, group_rows: int = 0) -> None:
     """out = a[M, K] @ w[N, K]^T on the tensor cores (bf16 in, fp32 accumulate). ``out`` is [M, N] (bf16 or fp32)
     or, with K splits, fp32 [S, M, N] where S = gemm_tc_splits(K, splits). ``swiglu`` (prefill form, bn a multiple
     of 32): w holds 16 gate rows then the 16 up rows of the same outputs, group after group, and ``out`` is the bf16
     [M, N / 2] result silu(gate) * up. ``mt`` = 2 (prefill form): a unit is two 128-row tiles over the same columns.
-    ``post`` = (float32 bias [N] or None, a key of ``ACT``): the bf16 rows leave as act(. + bias)"""
+    ``post`` = (float32 bias [N] or None, a key of ``ACT``): the bf16 rows leave as act(. + bias). ``group_rows`` (decode
+    form, a multiple of 128; K a multiple of 64): every ``group_rows`` rows of w multiply an input of their own, a = [M,
+    groups * K] with the inputs side by side"""
     _need_cuda(a, w, out)
     bias, pact = _post_args(post, w.shape[0], out, swiglu)
-    M, K = a.shape
+    M, K = a.shape[0], w.shape[1]
     N = w.shape[0]
-    assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape[1] == K
+    groups = -(-N // group_rows) if group_rows else 1
+    assert a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and a.shape[1] == groups * K
     assert a.stride(1) == 1 and w.stride(1) == 1 and out.is_contiguous()
     if swiglu:
         assert out.shape == (M, N // 2) and out.dtype == torch.bfloat16 and not swap and splits == 1 and N % 32 == 0 and bn % 32 == 0
@@ -847,7 +853,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, swap: bool, 
         stride, ldc = 0, N
     _check(load().kb_gemm_tc(_p(a), _p(w), _p(out), dt(out), M, N, K, a.stride(0), w.stride(0), ldc, 1 if swap else 0,
                              bn, splits, stride, _p(status), _stream(), GATE_ACT[act] if swiglu else 0, mt,
-                             *_gate_params(act, act_params), _p(bias), pact), "gemm_tc")
+                             *_gate_params(act, act_params), _p(bias), pact, int(group_rows)), "gemm_tc")
 
 
 def gemm_pair(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, bn: int, status: torch.Tensor,
@@ -1418,21 +1424,23 @@ def token_mix(y: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, ctx, out: t
 
 
 def tanh_rows(a: torch.Tensor, out: torch.Tensor) -> None:
-    """out = tanh(a); rows [T, N]"""
+    """out = tanh(a); ``a``: rows [T, N] or 32-bit planes [S, T, N]"""
     _need_cuda(a, out)
     T, N = out.shape
-    assert a.shape == (T, N) and a.stride(1) == 1 and out.is_contiguous() and a.dtype == out.dtype
-    _check(load().kb_tanh_rows(_p(a), dt(a), a.stride(0), _p(out), T, N, _stream()), "tanh_rows")
+    n_planes, pstride, ld = _planes_of(a)
+    assert a.shape[-2:] == (T, N) and out.is_contiguous()
+    _check(load().kb_tanh_rows(_p(a), dt(a), n_planes, pstride, ld, _p(out), dt(out), T, N, _stream()), "tanh_rows")
 
 
 def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: Optional[torch.Tensor], low: Optional[torch.Tensor],
         w2: Optional[torch.Tensor], w0: torch.Tensor, u: torch.Tensor, B: int, H: int, d: int, dv: int, q_start, slot,
-        state: torch.Tensor, out: torch.Tensor) -> None:
+        state: torch.Tensor, out: torch.Tensor, runs: bool = False) -> None:
     """``o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t``, ``S_t = diag(w_t) S_(t-1) + k_t v_t^T`` over the packed rows of ``B``
     sequences, H heads of ``d`` key channels and ``dv`` values. ``r``, ``k``, ``v``: rows or 32-bit planes of one dtype and
     layout. ``w_t = exp(-exp(z_t + w0))``: ``z`` float32 rows [T, H d], or None, and then ``z = w2 tanh(low)`` is made by the
     kernel from ``low`` (rows or planes [.., T, rank]) and ``w2`` [H d, rank]. ``w0``, ``u`` float32 [H d]; ``state``
-    float32 [slots, H, dv, d], read and written; ``out`` float32 [T, H dv]"""
+    float32 [slots, H, dv, d], read and written; ``out`` float32 [T, H dv]. ``runs`` (bf16 rows, finished ``z``, d up to
+    128): the form for long prompts, whose sums differ from the token-by-token form's by rounding"""
     _need_cuda(r, k, v, z, low, w2, w0, u, state, out)
     n_planes, pstride, ld = _planes_of(r)
     for t in (k, v):
@@ -1453,10 +1461,24 @@ def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: Optional[torch.Ten
     if d > 256 or rank > 512:
         raise KernelError("kindi_b200: the recurrence with a decay per channel takes heads of up to 256 channels and low-rank "
                           "projections of up to 512, found %d and %d" % (d, rank))
-    _check(load().kb_wkv_scan(dt(r), _p(r), _p(k), _p(v), n_planes, pstride, ld, _p(z), z.stride(0) if z is not None else 0,
-                              _p(low) if z is None else None, lp, ls, ldl, _p(w2) if z is None else None,
-                              dt(w2) if z is None else F32, rank, _p(w0), _p(u), B, H, d, dv, _p(q_start), _p(slot), _p(state),
-                              state.stride(0), _p(out), out.stride(0), _stream()), "wkv_scan")
+    args = (dt(r), _p(r), _p(k), _p(v), n_planes, pstride, ld, _p(z), z.stride(0) if z is not None else 0,
+            _p(low) if z is None else None, lp, ls, ldl, _p(w2) if z is None else None, dt(w2) if z is None else F32, rank,
+            _p(w0), _p(u), B, H, d, dv, _p(q_start), _p(slot), _p(state), state.stride(0), _p(out), out.stride(0))
+    if runs:
+        T = out.shape[0]
+        n = T // wkv_run() + B
+        part = torch.empty((n, H, dv, d), dtype=torch.float32, device=out.device)
+        keep = torch.empty((n, H, d), dtype=torch.float32, device=out.device)
+        _check(load().kb_wkv_runs(*args, T, _p(part), _p(keep), _stream()), "wkv_runs")
+        add_launches(2)
+        return
+    _check(load().kb_wkv_scan(*args, _stream()), "wkv_scan")
+
+
+@functools.lru_cache(maxsize=1)
+def wkv_run() -> int:
+    """tokens of a run in the form for long prompts"""
+    return load().kb_wkv_run()
 
 
 def cast_rows(x: torch.Tensor, y: torch.Tensor) -> None:

@@ -112,6 +112,8 @@ class GroupedWeight:
         self.sizes = tuple(int(w.shape[0]) for w in ws)
         self.k = int(ws[0].shape[1])
         self.joined = torch.cat(list(ws), dim=0).contiguous()
+        # all but the last of one size, and the last no larger: the groups' rows start at multiples of that size
+        self.even = len(set(self.sizes[:-1])) == 1 and self.sizes[-1] <= self.sizes[0]
 
     def parts(self):
         at = 0
@@ -122,5 +124,23 @@ class GroupedWeight:
 
 def grouped_rows_or_planes(ctx, a: torch.Tensor, gw: GroupedWeight, out_dtype: torch.dtype):
     """the products ``a_i @ w_i^T`` of the inputs ``a = [a_0 | a_1 | ...]`` (``[M, n K]``) with the matrices of ``gw``, as a list
-    in the form of ``rows_or_planes``; results of matrices of one size are laid out alike"""
-    return [rows_or_planes(ctx, a[:, i * gw.k:(i + 1) * gw.k], w, out_dtype) for i, w in enumerate(gw.parts())]
+    in the form of ``rows_or_planes``; results of matrices of one size are laid out alike. A decode-sized step takes one launch
+    for all of them where the kernel takes the shape"""
+    if ctx.fast and gw.even:
+        out = fast.gemm_planes_grouped(a, gw.joined, gw.sizes[0], ctx.status)
+        if out is not None:
+            at = [sum(gw.sizes[:i]) for i in range(len(gw.sizes))]
+            return [out[:, :, c:c + n] for c, n in zip(at, gw.sizes)]
+    # (a matrix with fewer rows than the first is a low-rank projection beside the others)
+    return [(narrow if w.shape[0] < gw.sizes[0] else rows_or_planes)(ctx, a[:, i * gw.k:(i + 1) * gw.k], w, out_dtype)
+            for i, w in enumerate(gw.parts())]
+
+
+def narrow(ctx, a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """``rows_or_planes`` for a product of few columns (a low-rank projection): 32-bit planes also for long prompts, where the
+    product's few tiles would leave most of the GPU idle"""
+    if ctx.fast:
+        p = fast.gemm_narrow_planes(a, w, ctx.status)
+        if p is not None:
+            return p
+    return rows_or_planes(ctx, a, w, out_dtype)

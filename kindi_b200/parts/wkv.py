@@ -94,7 +94,7 @@ class TimeMix(Mixer):
         K.token_mix(y, self.mu, last, ctx, mixed)
         r, k, v, g, low = L.grouped_rows_or_planes(ctx, mixed, self.w_in, self.dtype)
         z = None
-        if low.dim() == 2:
+        if r.dim() == 2:
             # finished rows: the decay's exponent is a product too (small steps leave it to the recurrence's kernel)
             th = torch.empty((T, self.rank), dtype=self.dtype, device=y.device)
             K.tanh_rows(low, th)
@@ -102,10 +102,17 @@ class TimeMix(Mixer):
         # (padding rows of a recorded step are written by nobody)
         new = torch.zeros if ctx.graph and not ctx.decode else torch.empty
         o = new((T, H * d), dtype=torch.float32, device=y.device)
-        K.wkv(r, k, v, z, low, self.w2, self.w0, self.u, ctx.B, H, d, d, ctx.q_start, ctx.slot, state, o)
+        K.wkv(r, k, v, z, low, self.w2, self.w0, self.u, ctx.B, H, d, d, ctx.q_start, ctx.slot, state, o,
+              runs=self._in_runs(ctx, r))
         yn = torch.empty((T, H * d), dtype=self.dtype, device=y.device)
         K.head_norm_gate(o, H, d, self.g_norm, self.eps, g, 0, "silu", yn)
         return Branch(L.planes(ctx, yn, self.w_o))
+
+    def _in_runs(self, ctx: StepContext, rows: torch.Tensor) -> bool:
+        """whether a step's recurrence runs in the form for long prompts: bf16 rows (a step of more rows than the products
+        split into planes), a sequence of more than one run, heads that fit a run's tiles"""
+        return ctx.fast and not ctx.decode and rows.dim() == 2 and rows.dtype == torch.bfloat16 and self.d <= 128 \
+            and ctx.max_q > K.wkv_run()
 
     def bytes_read(self) -> int:
         return sum(w.numel() * w.element_size() for w in (self.w_in.joined, self.w2, self.w_o))
