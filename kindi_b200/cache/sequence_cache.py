@@ -2,8 +2,8 @@
 
 Cache entries (one per schedule entry that owns a cache) are grouped by what they need: entries that keep the same
 number of key/value heads of the same size over the same span (all positions, or a window) share one group, and
-each group has storage of its own: a pool of pages ``[entry][page][k|v][kv head][position in page][head_dim]`` and
-a page table ``[slot][block]`` on the device. Entries that ask for a fixed-size state get a 32-bit tensor
+each group has storage of its own: a pool of pages ``[entry][page][k|v][kv head][position in page][head_dim]`` (one
+plane instead of k and v for entries whose values are their keys' beginnings) and a page table ``[slot][block]`` on the device. Entries that ask for a fixed-size state get a 32-bit tensor
 ``[slot][...]`` that is zeroed when a slot is taken. An entry may ask for several things at once (a tuple of needs:
 keys and values for one part of its mixer and states for others): at most one ``KVNeed``, any number of states,
 which ``state_view(entry, k)`` hands out in the order they were asked for.
@@ -46,7 +46,7 @@ def split_needs(need, entry: int = -1):
 class KVGroup:
     need: KVNeed
     entries: List[int]                 # cache entry indices, in pool order
-    pool: torch.Tensor                 # [len(entries), pool pages, 2, n_kv, PAGE, head_dim]
+    pool: torch.Tensor                 # [len(entries), pool pages, 2 (values in keys: 1), n_kv, PAGE, head_dim]
     table: torch.Tensor                # int32 [n_slots, n_pages] on the device, -1 = not mapped
     pages: PageMap
     n_pool_pages: int                  # pages of this group's pool (a window group needs fewer than a full one)
@@ -79,7 +79,7 @@ class SequenceCache:
                                              device=self.device) for st in states]
         for need, entries in by_need.items():
             n_pool = self.group_pages(need, self.n_pages, self.n_slots, max_step_tokens)
-            pool = torch.zeros((len(entries), n_pool, 2, need.n_kv_heads, PAGE, need.head_dim), dtype=dtype,
+            pool = torch.zeros((len(entries), n_pool, need.planes, need.n_kv_heads, PAGE, need.head_dim), dtype=dtype,
                                device=self.device)
             table = torch.full((self.n_slots, self.n_pages), -1, dtype=torch.int32, device=self.device)
             g = KVGroup(need, entries, pool, table, PageMap(n_pool, self.n_slots, need.window, need.keep_first), n_pool)
@@ -110,7 +110,7 @@ class SequenceCache:
         for i, asked in enumerate(needs):
             need, states = split_needs(asked, i)
             if need is not None:
-                total += (SequenceCache.group_pages(need, n_pages, n_slots, max_step_tokens) * 2 * need.n_kv_heads
+                total += (SequenceCache.group_pages(need, n_pages, n_slots, max_step_tokens) * need.planes * need.n_kv_heads
                           * PAGE * need.head_dim * el)
                 if need not in seen:
                     seen.add(need)
@@ -121,7 +121,7 @@ class SequenceCache:
 
     def kv_bytes_per_token(self) -> int:
         el = torch.empty((), dtype=self.dtype).element_size()
-        return sum(len(g.entries) * 2 * g.need.n_kv_heads * g.need.head_dim * el for g in self.groups)
+        return sum(len(g.entries) * g.need.planes * g.need.n_kv_heads * g.need.head_dim * el for g in self.groups)
 
     # ------------------------------------------------------------------ slots
     def alloc_slot(self) -> int:
@@ -190,7 +190,7 @@ class SequenceCache:
 
     # ------------------------------------------------------------------ views for the parts
     def kv_view(self, entry: int):
-        """(pool of this entry [pool pages, 2, n_kv, PAGE, head_dim], page table, number of pages of the pool)"""
+        """(pool of this entry [pool pages, 2 or 1, n_kv, PAGE, head_dim], page table, number of pages of the pool)"""
         gi, j = self._where[entry]
         g = self.groups[gi]
         return g.pool[j], g.table, g.n_pool_pages

@@ -41,7 +41,8 @@ __device__ __forceinline__ float kb_warp_max(float v) {
 }
 
 // where a sequence's keys and values live: pool of pages [page][2][n_kv][KB_PAGE][head_dim] for one cache entry,
-// and the table that maps (slot, position / KB_PAGE) to a page
+// and the table that maps (slot, position / KB_PAGE) to a page. one_plane: a position's value is the beginning of its key, a
+// page is [n_kv][KB_PAGE][head_dim]
 struct KbCacheView {
     void* pool;                 // this cache entry's pages
     const int* table;           // [n_slots][table_stride]
@@ -49,10 +50,12 @@ struct KbCacheView {
     int n_pages;
     int n_kv;
     int head_dim;
+    int one_plane;
 };
 
 __device__ __forceinline__ size_t kb_kv_offset(const KbCacheView& c, int page, int kv, int head, int p_in_page) {
-    return ((((size_t)page * 2 + kv) * c.n_kv + head) * KB_PAGE + p_in_page) * (size_t)c.head_dim;
+    const size_t plane = c.one_plane ? (size_t)page : (size_t)page * 2 + kv;
+    return ((plane * c.n_kv + head) * KB_PAGE + p_in_page) * (size_t)c.head_dim;
 }
 
 // activations of a feed-forward that takes its activation as a parameter

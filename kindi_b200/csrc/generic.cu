@@ -1094,12 +1094,12 @@ extern "C" int kb_rope_store(const void* in, int in_dtype, int n_planes, long lo
 // their true positions), read from the cache. Scores may be capped (cap > 0: cap tanh(s / cap)). Keys are taken in runs of 32 that start at multiples of 32 of the absolute
 // position (lane = position for the scores, lane = dimension for P V) with a running maximum and sum, so the order
 // of every sum depends on positions only: the same row gives the same bits whether it came in a prompt or alone.
-#define AG_MAX_HD 512
+#define AG_MAX_HD 576
 template <typename T>
 __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, int ldq, T* __restrict__ out,
         int ldo, const int* __restrict__ pos, const int* __restrict__ seq, const int* __restrict__ slot, int Tn,
         int nh, int group, int hd, float scale, int window, int keep_first, KbCacheView cv, int* status,
-        const float* __restrict__ sink, const T* KB_STEP_DATA gate, int ldg, int chunk, float cap) {
+        const float* __restrict__ sink, const T* KB_STEP_DATA gate, int ldg, int chunk, float cap, int vd) {
     __shared__ float qs[4][AG_MAX_HD];
     kb_pdl_launch();
     kb_pdl_wait();
@@ -1158,7 +1158,7 @@ __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, i
 #pragma unroll
             for (int i = 0; i < AG_MAX_HD / 32; i++) {
                 const int d = i * 32 + lane;
-                if (d < hd) o[i] = fmaf(pj, kb_to_f<T>(vj[d]), o[i]);
+                if (d < vd) o[i] = fmaf(pj, kb_to_f<T>(vj[d]), o[i]);
             }
         }
     }
@@ -1171,12 +1171,12 @@ __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, i
 #pragma unroll
         for (int i = 0; i < AG_MAX_HD / 32; i++) o[i] *= f;
     }
-    T* orow = out + (size_t)t * ldo + (size_t)h * hd;
-    const T* grow = gate ? gate + (size_t)t * ldg + (size_t)h * hd : nullptr;
+    T* orow = out + (size_t)t * ldo + (size_t)h * vd;
+    const T* grow = gate ? gate + (size_t)t * ldg + (size_t)h * vd : nullptr;
 #pragma unroll
     for (int i = 0; i < AG_MAX_HD / 32; i++) {
         const int d = i * 32 + lane;
-        if (d < hd) {
+        if (d < vd) {
             float v = o[i] / l;
             // an output gate: the head's output times the logistic function of the gate's row
             if (grow) v = v * (1.0f / (1.0f + expf(-kb_to_f<T>(grow[d]))));
@@ -1188,21 +1188,24 @@ __global__ void __launch_bounds__(128) k_attn_generic(const T* KB_STEP_DATA q, i
 extern "C" int kb_attn_generic(const void* q, int dtype, int ldq, void* out, int ldo, const int* pos, const int* seq,
                                const int* slot, int T, int nh, int nkv, int hd, float scale, int window, void* pool,
                                const int* table, int table_stride, int n_pages, int* status, cudaStream_t st,
-                               int keep_first, const float* sink, const void* gate, int ldg, int chunk, float cap) {
-    // sink (float [nh] or null): exp(sink[h]) joins the softmax denominator of head h. gate (rows of the queries'
+                               int keep_first, const float* sink, const void* gate, int ldg, int chunk, float cap, int vd,
+                               int one_plane) {
+    // vd (0: hd): elements of a value, and of a head of the output. one_plane: values are their keys' beginnings. sink (float [nh] or null): exp(sink[h]) joins the softmax denominator of head h. gate (rows of the queries'
     // type [T][ldg], laid out like the output, or null): out *= 1 / (1 + exp(-gate))
     if (T <= 0) return 0;
     if (hd > AG_MAX_HD || nkv <= 0 || nh % nkv) return (int)cudaErrorInvalidValue;
     if (window <= 0 || keep_first < 0) keep_first = 0;
-    KbCacheView cv{pool, table, table_stride, n_pages, nkv, hd};
+    if (vd <= 0) vd = hd;
+    if (vd > hd) return (int)cudaErrorInvalidValue;
+    KbCacheView cv{pool, table, table_stride, n_pages, nkv, hd, one_plane};
     long long items = (long long)T * nh;
     int grid = (int)((items + 3) / 4);
     if (dtype == KB_F32)
         kb_launch(k_attn_generic<float>, grid, 128, 0, st, (const float*)q, ldq, (float*)out, ldo, pos, seq, slot, T, nh,
-                                                   nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const float*)gate, ldg, chunk, cap);
+                                                   nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const float*)gate, ldg, chunk, cap, vd);
     else
         kb_launch(k_attn_generic<bf16>, grid, 128, 0, st, (const bf16*)q, ldq, (bf16*)out, ldo, pos, seq, slot, T, nh,
-                                                  nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const bf16*)gate, ldg, chunk, cap);
+                                                  nh / nkv, hd, scale, window, keep_first, cv, status, sink, (const bf16*)gate, ldg, chunk, cap, vd);
     KB_LAUNCH_RET();
 }
 

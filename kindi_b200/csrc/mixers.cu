@@ -105,6 +105,7 @@ extern "C" int kb_gated_rmsnorm(const float* x, int ldx, const void* w, int wdty
 // | anything else], as a row or as planes. This kernel writes the normalised query latent (RMS norm with gains, the
 // run's type) and stores into the cache, at the row's position, ONE key/value head of size D >= kv_rank + rot:
 //   keys   [normalised latent | rotated part | zeros]      values [normalised latent | zeros]
+// (a cache of one plane holds the keys alone: their beginning is the value)
 // so that attention over the cache with queries [W_uk^T q | rotated q | zeros] gives the scores of the expanded keys,
 // and its output's first kv_rank elements are the weighted sum of latents, from which W_uv makes the heads' values.
 // Rotation: pair i is the elements (2i, 2i + 1), or with `half` (i, i + rot / 2); its angle is pos * freq[i], in 32-bit, or in
@@ -177,7 +178,7 @@ __global__ void __launch_bounds__(256) k_latent_prep(const TIN* KB_STEP_DATA in,
         const T c = kb_from_f<T>(__fmul_rn(__fmul_rn(scale_c, mx_rd<TIN>(src, n_planes, plane_stride, q_rank + i)),
                                            kb_to_f<TW>(wkv[i])));
         kd[i] = c;
-        vd[i] = c;
+        if (!cv.one_plane) vd[i] = c;
     }
     for (int i = threadIdx.x; i < rot / 2; i += 256) {
         float c, sn;
@@ -190,6 +191,7 @@ __global__ void __launch_bounds__(256) k_latent_prep(const TIN* KB_STEP_DATA in,
         kd[kv_rank + ib] = kb_from_f<T>(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
     }
     for (int i = kv_rank + rot + threadIdx.x; i < cv.head_dim; i += 256) kd[i] = kb_from_f<T>(0.0f);
+    if (cv.one_plane) return;
     for (int i = kv_rank + threadIdx.x; i < cv.head_dim; i += 256) vd[i] = kb_from_f<T>(0.0f);
 }
 
@@ -197,11 +199,11 @@ extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long l
                               int kv_rank, int rot, const void* wq, const void* wkv, int wdtype, float eps,
                               const float* freq, float mult, const int* pos, const int* seq, const int* slot, void* cq,
                               int dtype, int ldcq, int T, int D, void* pool, const int* table, int table_stride,
-                              int n_pages, int* status, cudaStream_t st, const double* freq64, int half) {
+                              int n_pages, int* status, cudaStream_t st, const double* freq64, int half, int one_plane) {
     if (T <= 0) return 0;
     const MxRot rr{freq, freq64, mult, half};
     if (rot % 2 || kv_rank + rot > D) return (int)cudaErrorInvalidValue;
-    KbCacheView cv{pool, table, table_stride, n_pages, 1, D};
+    KbCacheView cv{pool, table, table_stride, n_pages, 1, D, one_plane};
 #define KB_LP(TIN, TW, T_)                                                                                       \
     kb_launch(k_latent_prep<TIN, TW, T_>, T, 256, 0, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in,  \
               q_rank, kv_rank, rot, (const TW*)wq, (const TW*)wkv, eps, rr, pos, seq, slot, (T_*)cq, ldcq, \

@@ -74,6 +74,17 @@ def attention(ctx, q, out, nh, nkv, hd, scale, window, pool, table, n_pages, kee
     return rows_gate is not None
 
 
+def latent_attention(ctx, q, out, nh: int, hd: int, v_dim: int, scale: float, pool, table, n_pages) -> None:
+    """``out`` ``[T, nh v_dim]`` = causal attention of the query rows ``q`` ``[T, nh hd]`` over their sequences' cached vectors
+    (``pool`` ``[pages, 1, 1, 64, hd]``, this step's included): one per position, the key of every head, whose first ``v_dim``
+    elements are the value"""
+    if ctx.fast:
+        from . import fast
+        if fast.latent_attention_bf16(ctx, q, out, nh, hd, v_dim, scale, pool, table, n_pages):
+            return
+    K.attn_generic(q, out, ctx.pos, ctx.seq, ctx.slot, nh, 1, hd, scale, 0, pool, table, n_pages, ctx.status, v_dim=v_dim)
+
+
 def attention_from_planes(ctx, qkv, out, nh, nkv, hd, scale, window, rotation, pool, table, n_pages) -> bool:
     """a decode step of the serving kernels whose QKV product came as 32-bit planes: one kernel sums them, rotates
     queries and the newest key by ``rotation`` (``(inv_freq, rotary_dim)`` of the position encoding, None when it is

@@ -341,6 +341,27 @@ def attention_decode_rope(ctx, qkv, out, nh, nkv, hd, scale, window, inv_freq, r
     return True
 
 
+def latent_splits(ctx, head_tiles: int) -> int:
+    """position splits of a decode step over a cache of latents: one wave of CTAs over all (sequence, head tile) pairs, two an
+    SM"""
+    return max(1, min(64, 2 * N_SM // max(1, ctx.B * head_tiles)))
+
+
+def latent_attention_bf16(ctx, q, out, nh: int, hd: int, v_dim: int, scale: float, pool, table, n_pages) -> bool:
+    """the tensor-core kernels over a cache of one vector per position, where they take the shape; False: not taken"""
+    if (hd not in K.LATENT_DIMS or q.dtype != torch.bfloat16 or q.stride(0) % 8 or q.data_ptr() % 16 or out.stride(0) % 8
+            or out.data_ptr() % 16 or pool.shape[1] != 1 or scale <= 0.0):
+        return False
+    if ctx.decode:
+        K.latent_attn_decode(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, hd, v_dim, scale, pool, table, n_pages,
+                             splits=latent_splits(ctx, 1 if nh <= 16 else -(-nh // 32)), status=ctx.status)
+        return True
+    group = next((g for g in range(min(nh, 128), 0, -1) if nh % g == 0))
+    K.latent_attn_tc(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, group, hd, v_dim, scale, pool, table, n_pages,
+                     max_q=ctx.max_q, status=ctx.status)
+    return True
+
+
 MOE_GLU_MIN_PAIRS = 512     # (row, pick) pairs from which the grouped up product finishes a gated unit itself
 
 

@@ -60,14 +60,18 @@ _SIGS = {
     "kb_rope_table": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "kb_attn_generic": [c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                         c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p,
-                        c_void_p, c_int, c_int, c_float],
+                        c_void_p, c_int, c_int, c_float, c_int, c_int],
     "kb_gate_mul": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_int,
                     c_void_p],
     "kb_gated_rmsnorm": [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p,
                          c_int, c_int, c_int, c_int, c_void_p],
     "kb_latent_prep": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                        c_float, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                       c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int],
+                       c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int],
+    "kb_latent_tc": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                     c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+    "kb_latent_decode": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                         c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "kb_latent_qrope": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
                         c_int, c_int, c_int, c_void_p, c_void_p, c_int],
     "kb_head_gemm": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
@@ -512,7 +516,8 @@ def latent_prep(a: torch.Tensor, q_rank: int, kv_rank: int, rot: int, wq: torch.
                 freq64: Optional[torch.Tensor] = None) -> None:
     """``a``: rows or 32-bit planes of [query latent | key/value latent | rotated key part | ...]. Writes the RMS-normed
     query latent to ``cq`` and stores, at each row's position of its sequence's pages, one key head [normed latent |
-    rotated part | 0] and one value head [normed latent | 0] of ``head_dim`` elements. The rotation pairs element 2i
+    rotated part | 0] and one value head [normed latent | 0] of ``head_dim`` elements (a pool of one plane, [pages, 1, 1,
+    64, head_dim], takes the key head alone). The rotation pairs element 2i
     with 2i + 1 (``pairing`` "half": i with i + rot / 2), by pos * freq[i], cosine and sine times ``mult``; float32 rows
     take their angles from ``freq64`` (float64) where it is given"""
     _need_cuda(a, wq, wkv, freq, cq, pool, table, freq64)
@@ -523,11 +528,12 @@ def latent_prep(a: torch.Tensor, q_rank: int, kv_rank: int, rot: int, wq: torch.
     assert wkv.numel() == kv_rank and wq.is_contiguous() and wkv.is_contiguous()
     assert freq.dtype == torch.float32 and freq.numel() >= max(1, rot // 2) and freq.is_contiguous()
     assert cq.shape == (T, q_rank) and cq.stride(1) == 1 and pool.dtype == cq.dtype and pool.is_contiguous()
-    assert pool.shape[-1] == head_dim and pool.shape[-3] == 1
+    assert pool.shape[-1] == head_dim and pool.shape[-3] == 1 and pool.shape[-4] in (1, 2)
     _check(load().kb_latent_prep(_p(a), dt(a), n_planes, pstride, ld, q_rank, kv_rank, rot, _p(wq), _p(wkv), dt(wq),
                                  float(eps), _p(freq), float(mult), _p(pos), _p(seq), _p(slot), _p(cq), dt(cq),
                                  cq.stride(0), T, head_dim, _p(pool), _p(table), table.stride(0), n_pages, _p(status),
-                                 _stream(), _p(freq64), PAIRING[pairing]), "latent_prep")
+                                 _stream(), _p(freq64), PAIRING[pairing], 1 if pool.shape[-4] == 1 else 0),
+           "latent_prep")
 
 
 def latent_qrope(q: torch.Tensor, dim: int, rot: int, freq: torch.Tensor, mult: float, pos, out: torch.Tensor,
@@ -779,26 +785,64 @@ def rope_store(qkv: torch.Tensor, qout: torch.Tensor, inv_freq: torch.Tensor, ro
 def attn_generic(q: torch.Tensor, out: torch.Tensor, pos, seq, slot, nh: int, nkv: int, hd: int, scale: float,
                  window: int, pool: torch.Tensor, table: torch.Tensor, n_pages: int, status: torch.Tensor,
                  keep_first: int = 0, sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                 chunk: int = 0, softcap: float = 0.0) -> None:
+                 chunk: int = 0, softcap: float = 0.0, v_dim: int = 0) -> None:
     """attention of each row of q ([T, >= nh hd], row stride free) over its sequence's cached keys and values: all
     positions up to the row's, or with ``window`` the last ``window`` of them and the sequence's first ``keep_first``,
     or with ``chunk`` those of its own chunk of that many positions. ``softcap`` > 0: scores are capped.
     ``sink`` (float32 [nh]): exp(sink[h]) joins head h's softmax denominator. ``gate`` (rows of q's dtype, laid out
-    like ``out``): the output is multiplied by the logistic function of it"""
+    like ``out``): the output is multiplied by the logistic function of it. ``v_dim`` (0: hd): elements of a value and of a
+    head of ``out``. A pool of one plane (``[pages, 1, ...]``): a value is its key's beginning"""
     _need_cuda(q, out, pool, table, sink, gate)
     if sink is not None:
         assert sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == nh
     if gate is not None:
         assert gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape[0] == q.shape[0]
     T = q.shape[0]
-    if hd > 512:
-        raise KernelError("kindi_b200: attention supports head sizes up to 512, found %d" % hd)
+    if hd > 576:
+        raise KernelError("kindi_b200: attention supports head sizes up to 576, found %d" % hd)
     assert q.stride(1) == 1 and out.stride(1) == 1 and q.dtype == out.dtype == pool.dtype
     _check(load().kb_attn_generic(_p(q), dt(q), q.stride(0), _p(out), out.stride(0), _p(pos), _p(seq), _p(slot), T,
                                   nh, nkv, hd, float(scale), int(window), _p(pool), _p(table), table.stride(0),
                                   n_pages, _p(status), _stream(), int(keep_first), _p(sink), _p(gate),
-                                  gate.stride(0) if gate is not None else 0, int(chunk), float(softcap)),
-           "attn_generic")
+                                  gate.stride(0) if gate is not None else 0, int(chunk), float(softcap), int(v_dim),
+                                  1 if pool.dim() >= 4 and pool.shape[-4] == 1 else 0), "attn_generic")
+
+
+LATENT_DIMS = (64, 128, 192, 256, 320, 576)       # sizes of a cached latent that the tensor-core kernels take
+
+
+def latent_attn_tc(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, nh: int, group: int, hd: int, v_dim: int,
+                   scale: float, pool: torch.Tensor, table: torch.Tensor, n_pages: int, *, max_q: int,
+                   status: torch.Tensor) -> None:
+    """tcgen05 attention of prompt-sized steps over a cache of one vector per position (``pool`` [pages, 1, 1, 64, hd], hd one of
+    ``LATENT_DIMS``) that is every head's key and whose first ``v_dim`` elements are the value: q [T, nh hd], out [T, nh v_dim].
+    ``group``: query heads a CTA takes together (divides nh, at most 128); ``max_q``: the most rows a sequence brings"""
+    _need_cuda(q, out, pool, table)
+    assert q.dtype == out.dtype == pool.dtype == torch.bfloat16 and q.stride(1) == 1 and out.stride(1) == 1
+    assert pool.is_contiguous() and pool.shape[1:] == (1, 1, PAGE, hd) and hd in LATENT_DIMS
+    assert q.shape[1] == nh * hd and out.shape == (q.shape[0], nh * v_dim)
+    _check(load().kb_latent_tc(_p(q), q.stride(0), _p(out), out.stride(0), v_dim, _p(slot), _p(q_start), _p(kv_len), B, nh, group,
+                               hd, float(scale), _p(pool), _p(table), table.stride(0), n_pages, -(-max_q // (128 // group)),
+                               _p(status), _stream()), "latent_tc")
+
+
+def latent_attn_decode(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, nh: int, hd: int, v_dim: int,
+                       scale: float, pool: torch.Tensor, table: torch.Tensor, n_pages: int, *, splits: int,
+                       status: torch.Tensor) -> None:
+    """the same for one row per sequence (any number of heads): every sequence's pages in ``splits`` parts side by side"""
+    _need_cuda(q, out, pool, table)
+    assert q.dtype == out.dtype == pool.dtype == torch.bfloat16 and q.stride(1) == 1 and out.stride(1) == 1
+    assert pool.is_contiguous() and pool.shape[1:] == (1, 1, PAGE, hd) and hd in LATENT_DIMS
+    assert q.shape[1] == nh * hd and out.shape == (q.shape[0], nh * v_dim)
+    part_o = part_ml = None
+    if splits > 1:
+        part_o = torch.empty((B, nh, splits, v_dim), dtype=torch.float32, device=q.device)
+        part_ml = torch.empty((B, nh, splits, 2), dtype=torch.float32, device=q.device)
+    _check(load().kb_latent_decode(_p(q), q.stride(0), _p(out), out.stride(0), v_dim, _p(part_o), _p(part_ml), _p(slot),
+                                   _p(q_start), _p(kv_len), B, nh, hd, float(scale), _p(pool), _p(table), table.stride(0),
+                                   n_pages, splits, _p(status), _stream()), "latent_decode")
+    if splits > 1:
+        add_launches(1)         # the merge of the position splits
 
 
 def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int = 0, act: str = "silu") -> None:

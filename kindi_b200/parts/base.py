@@ -24,12 +24,18 @@ from ..config.spec import PartSpec
 class KVNeed:
     """keys and values of ``n_kv_heads`` x ``head_dim`` per position; ``window`` None keeps every position, else
     only the last ``window`` positions and the first ``keep_first`` positions of a sequence are ever read (pages
-    that hold neither are given back)."""
+    that hold neither are given back). ``values_in_keys``: a position's value is the beginning of its key, so a page has
+    one plane instead of two."""
 
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     keep_first: int = 0
+    values_in_keys: bool = False
+
+    @property
+    def planes(self) -> int:
+        return 1 if self.values_in_keys else 2
 
 
 @dataclass(frozen=True)

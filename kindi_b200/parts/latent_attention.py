@@ -12,11 +12,11 @@ With ``y`` the mixer's input, H heads, per head ``dim`` plain and ``rot_dim`` ro
   ``head_gate`` one number per head), then ``W_o``.
 
 What runs is the absorbed form, the same arithmetic re-associated: ``q_plain . (W_uk_h c) = (W_uk_h^T q_plain) . c``
-and ``sum_j p_j W_uv_h c_j = W_uv_h (sum_j p_j c_j)``. So the cache holds, per position, ONE key/value head: keys
-``[c | rotated part | 0]`` and values ``[c | 0]`` of a size ``D >= kv_rank + rot_dim`` that the attention kernels
-take; queries become ``[W_uk_h^T q_plain | rotated q | 0]`` per head (a per-head product); attention is the
-library's grouped-query attention with H query heads on one key/value head; the heads' outputs (weighted sums of
-latents) go through ``W_uv_h`` (a per-head product, the gate in its epilogue). Prompts, single tokens and cut prompts
+and ``sum_j p_j W_uv_h c_j = W_uv_h (sum_j p_j c_j)``. So the cache holds, per position, ONE vector
+``[c | rotated part | 0]`` of a size ``D >= kv_rank + rot_dim`` that the attention kernels take: it is the key of every
+head and its beginning the value, stored and fetched once; queries become ``[W_uk_h^T q_plain | rotated q | 0]`` per head
+(a per-head product); the heads' outputs (weighted sums of latents) go through ``W_uv_h`` (a per-head product, the gate
+in its epilogue). Prompts, single tokens and cut prompts
 are the same code, and nothing is expanded per cached position. The rotation is the mixer's position part (its
 frequencies, pairing and factor on cosines and sines: see ``parts/rope.py``), applied by the latent kernels.
 
@@ -56,11 +56,11 @@ class LatentAttention(Mixer):
 
     @classmethod
     def _cache_dim(cls, spec: PartSpec) -> int:
-        """the size of the one cached key/value head: latent and rotated part, widened to a size the tensor-core
-        attention kernels take (64, 128) where that is near"""
+        """the size of the one cached vector: latent and rotated part, widened to a size the tensor-core attention
+        kernels take"""
         _, _, r, _, _, kr = cls._sizes(spec)
         m = kr + r
-        return 64 if m <= 64 else 128 if m <= 128 else (m + 7) // 8 * 8
+        return next((n for n in K.LATENT_DIMS if m <= n), (m + 7) // 8 * 8)
 
     @classmethod
     def tensor_shapes(cls, spec: PartSpec, width: int) -> Dict[str, Tuple[int, ...]]:
@@ -79,15 +79,15 @@ class LatentAttention(Mixer):
 
     @classmethod
     def cache_need(cls, spec: PartSpec, width: int):
-        return KVNeed(1, cls._cache_dim(spec), None, 0)
+        return KVNeed(1, cls._cache_dim(spec), None, 0, values_in_keys=True)
 
     def __init__(self, spec, width, weights: WeightView, *, dtype, device):
         super().__init__(spec, width, weights, dtype=dtype, device=device)
         self.H, self.d, self.r, self.dv, self.qr, self.kr = self._sizes(spec)
         self.D = self._cache_dim(spec)
-        if self.D > 512:
-            raise ValueError("latent and rotated part together may have up to 512 elements, found %d"
-                             % (self.kr + self.r))
+        if self.D > K.LATENT_DIMS[-1]:
+            raise ValueError("latent and rotated part together may have up to %d elements, found %d"
+                             % (K.LATENT_DIMS[-1], self.kr + self.r))
         self.scale = float(spec["scale"])
         self.eps = float(spec["eps"])
         pspec: PartSpec = spec["position"]
@@ -107,7 +107,10 @@ class LatentAttention(Mixer):
         self.w_uq = weights(n["uq"])
         # per head: W_uk_h^T as [kv_rank, dim] (rows = outputs of the absorbing product), W_uv_h as stored
         self.w_uk_t = weights(n["uk"]).view(self.H, self.d, self.kr).transpose(1, 2).contiguous()
-        self.w_uv = weights(n["uv"]).view(self.H, self.dv, self.kr).contiguous()
+        # (the attention kernels write heads of a multiple of eight elements: zero columns meet what lies behind the latent)
+        self.vd = (self.kr + 7) // 8 * 8
+        w_uv = weights(n["uv"]).view(self.H, self.dv, self.kr)
+        self.w_uv = torch.nn.functional.pad(w_uv, (0, self.vd - self.kr)).contiguous()
         self.w_o = weights(n["o"])
 
     def forward(self, ctx: StepContext, y: torch.Tensor) -> Branch:
@@ -123,11 +126,11 @@ class LatentAttention(Mixer):
         qf = torch.empty((ctx.T, H * D), dtype=self.dtype, device=y.device)
         K.head_gemm(q, d + r, self.w_uk_t, qf, D)
         K.latent_qrope(q, d, r, pos.inv_freq, pos.mult, ctx.pos, qf, kr, D, H, **turn)
-        att = torch.empty((ctx.T, H * D), dtype=self.dtype, device=y.device)
-        A.attention(ctx, qf, att, H, 1, D, self.scale, 0, pool, table, n_pages)
+        att = torch.empty((ctx.T, H * self.vd), dtype=self.dtype, device=y.device)
+        A.latent_attention(ctx, qf, att, H, D, self.vd, self.scale, pool, table, n_pages)
         o = torch.empty((ctx.T, H * dv), dtype=self.dtype, device=y.device)
         at = qr + kr + r
-        K.head_gemm(att, D, self.w_uv, o, dv, gate=a[..., at:at + self.gate_rows] if self.gate_rows else None)
+        K.head_gemm(att, self.vd, self.w_uv, o, dv, gate=a[..., at:at + self.gate_rows] if self.gate_rows else None)
         return Branch(L.planes(ctx, o, self.w_o))
 
     def bytes_read(self) -> int:
