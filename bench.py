@@ -351,8 +351,7 @@ def bench_e2e(eng, batch: int, context: int, steps: int, warm: int = 48, samplin
 # Layer sizes that resemble real models' (random weights, four layers: windowed attention with sink and gate, latent
 # attention, linear attention with decay, windowed attention that reads the first layer's keys and values; each with
 # the gated GELU feed-forward), each beside the dense Llama-arch decoder of the same width, query/key-value heads,
-# head size, window, feed-forward size and vocabulary. The cached latent head (latent + rotated part) is 128 wide, the
-# widest the tensor-core attention kernels take.
+# head size, window, feed-forward size and vocabulary. The cached latent (latent + rotated part) is 128 wide.
 NILATAR_SIZES = {
     "s": dict(width=1024, heads=8, kv=2, ff=2816, q_rank=384, lat_dim=64),
     "m": dict(width=2048, heads=16, kv=4, ff=5632, q_rank=768, lat_dim=64),
@@ -366,9 +365,10 @@ def nilatar_pair(sz: dict):
     H, ff = sz["heads"], {"kind": "dense", "ff": sz["ff"]}
     att = {"heads": H, "kv_heads": sz["kv"], "dim": NILATAR_HEAD, "vdim": NILATAR_HEAD, "scale": NILATAR_HEAD ** -0.5,
            "mask": {"size": NILATAR_WINDOW}}
-    lat = {"heads": H, "dim": sz["lat_dim"], "rot_dim": NILATAR_ROT, "vdim": sz["lat_dim"], "q_rank": sz["q_rank"],
-           "kv_rank": NILATAR_KV_RANK, "scale": (sz["lat_dim"] + NILATAR_ROT) ** -0.5,
-           "rot": {"base": 10000.0, "dims": NILATAR_ROT,
+    kr, rot = sz.get("kv_rank", NILATAR_KV_RANK), sz.get("rot", NILATAR_ROT)
+    lat = {"heads": H, "dim": sz["lat_dim"], "rot_dim": rot, "vdim": sz["lat_dim"], "q_rank": sz["q_rank"],
+           "kv_rank": kr, "scale": (sz["lat_dim"] + rot) ** -0.5,
+           "rot": {"base": 10000.0, "dims": rot,
                    "scaling": {"factor": 8.0, "original": 4096, "fast": 16.0, "slow": 2.0}}}
     lin = {"heads": H, "dim": NILATAR_HEAD, "vdim": NILATAR_HEAD,
            "decay": [1.0 - 2.0 ** (-5.0 - 3.0 * h / max(1, H - 1)) for h in range(H)]}
@@ -611,6 +611,67 @@ def bench_zebovik(a) -> int:
     return 0
 
 
+# ---------------------------------------------------------------------------------------------- --arch basitar
+# Layer sizes that resemble real models' (random weights, four layers: latent attention with a dense feed-forward, gated latent
+# attention with stretched frequencies and time mixing, both with experts, latent attention with a dense feed-forward), each
+# beside the Nilatar design (the closest one: latent attention, a recurrent layer with a matrix state) of the same width, heads,
+# latents and feed-forward weights a token uses (BASITAR_TOP picks of a BASITAR_TOP-th of the dense size each). Heads of the
+# recurrence have 64 channels, as the models of its kind do. Size x is l with latents of the size large models cache: 512 + 64.
+BASITAR_SIZES = dict(NILATAR_SIZES, x=dict(NILATAR_SIZES["l"], kv_rank=512, rot=64))
+BASITAR_EXPERTS, BASITAR_TOP, BASITAR_WKV_DIM = 16, 4, 64
+
+
+def basitar_config(sz: dict, positions: int):
+    """a Basitar config.json object at the sizes of BASITAR_SIZES[.]"""
+    kr, rot = sz.get("kv_rank", NILATAR_KV_RANK), sz.get("rot", NILATAR_ROT)
+    lat = {"heads": sz["heads"], "dim": sz["lat_dim"], "rot_dim": rot, "vdim": sz["lat_dim"], "q_rank": sz["q_rank"],
+           "kv_rank": kr, "scale": (sz["lat_dim"] + rot) ** -0.5, "rot": {"base": 10000.0, "dims": rot}}
+    far = dict(lat, rot={"base": 10000.0, "dims": rot, "scaling": {"factor": 8.0, "original": 4096, "fast": 16.0, "slow": 2.0}})
+    mix = {"heads": sz["width"] // BASITAR_WKV_DIM, "dim": BASITAR_WKV_DIM}
+    dense = {"kind": "dense", "ff": sz["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": sz["ff"] // BASITAR_TOP}, "router": {"experts": BASITAR_EXPERTS, "top": BASITAR_TOP}}
+    return {"architecture": "Basitar", "vocab": NILATAR_VOCAB, "width": sz["width"], "norm": {"eps": 1e-5},
+            "max_positions": positions, "embedding": {"bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 127}},
+            "layers": [{"type": "latent_attention", "mixer": lat, "mlp": dense},
+                       {"type": "latent_attention_2", "mixer": far, "mlp": moe}, {"type": "wkv", "mixer": mix, "mlp": moe},
+                       {"type": "latent_attention", "mixer": lat, "mlp": dense}]}
+
+
+def bench_basitar(a) -> int:
+    """prefill and decode throughput of the Basitar design at four layer sizes, each beside the Nilatar design of equal size,
+    with the device time per kind of launch"""
+    import torch
+    pk = peaks()
+    batch, context, tokens = a.batch, min(a.context, 4096), a.prefill_tokens
+    sizes = [x for x in (a.sizes or "s,m,l,x").split(",") if x in BASITAR_SIZES]
+    rows = {}
+    for name in sizes:
+        sz = BASITAR_SIZES[name]
+        ctx = batch * (context + a.steps + a.warmup + 320) + tokens + 64
+        bas, (nil, _) = basitar_config(sz, max(context + a.steps + a.warmup + 320, tokens)), nilatar_pair(sz)
+        row = {"sizes": dict(width=sz["width"], layers=4, ff=sz["ff"], latent=bas["layers"][0]["mixer"],
+                             wkv=bas["layers"][2]["mixer"], moe=bas["layers"][1]["mlp"])}
+        for what, cfg in (("basitar", bas), ("nilatar", nil)):
+            eng = engine_from_config(cfg, ctx, batch)
+            for g in eng.cache.groups:
+                g.pool.normal_(0.0, 1.0)
+            dev_ms, _, launches, _ = bench_decode(eng, batch, context, a.steps, max(3, a.warmup), False)
+            pms = bench_prefill(eng, 3, 5, tokens)
+            kt = kernel_times(eng, batch, context, tokens)
+            row[what] = {"decode_ms": round(dev_ms, 4), "decode_tokens_per_s": round(batch * 1000.0 / dev_ms, 1),
+                         "launches_per_step": launches // a.steps, "prefill_ms": round(pms, 3),
+                         "prefill_tokens_per_s": round(tokens * 1000.0 / pms, 1),
+                         "kernels_us": {k: _grouped(v) for k, v in kt.items()}}
+            del eng
+            torch.cuda.empty_cache()
+        rows[name] = row
+    print(json.dumps({"arch": "basitar", "what": "prefill and decode of the Basitar design beside the Nilatar design of "
+                      "equal size (random weights, 4 layers); not the default benchmark",
+                      "batch": batch, "context": context, "prefill_tokens": tokens, "steps": a.steps, "dtype": "bf16",
+                      "peaks": pk, "sizes": rows}))
+    return 0
+
+
 def kernel_times(eng, batch: int, context: int, prefill_tokens: int):
     """device time per kind of launch: one decode step of `batch` sequences at `context` and one prompt pass, each
     issued launch by launch (no recorded graph, launches strictly one after another) with CUDA events around every
@@ -842,11 +903,13 @@ def main(argv=None) -> int:
                          "0.7, top-p 0.8, top-k 20) and report it as e2e_sampled")
     ap.add_argument("--no-pdl", action="store_true", help="launch kernels strictly one after another")
     ap.add_argument("--prefill-only", action="store_true", help="measure only the prefill (for profiling)")
-    ap.add_argument("--arch", default="nanbeige", choices=("nanbeige", "vozinex", "nilatar", "medodra", "luzerax", "zebovik"),
-                    help="vozinex, nilatar, medodra, luzerax, zebovik: not the default benchmark but that design at a few layer sizes, "
+    ap.add_argument("--arch", default="nanbeige", choices=("nanbeige", "vozinex", "nilatar", "medodra", "luzerax", "zebovik",
+                                                           "basitar"),
+                    help="vozinex, nilatar, medodra, luzerax, zebovik, basitar: not the default benchmark but that design at a few layer sizes, "
                          "each beside the closest other decoder of equal size (prefill, decode, device time per kind "
                          "of launch)")
-    ap.add_argument("--sizes", default="", help="with --arch vozinex, nilatar, medodra, luzerax or zebovik: which of s,m,l (default: all)")
+    ap.add_argument("--sizes", default="", help="with --arch vozinex, nilatar, medodra, luzerax, zebovik or basitar: which of s,m,l (basitar: also x; "
+                                               "default: all)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                     help="prompt length of --prefill-only (the full run always measures 2048 tokens)")
     a = ap.parse_args(argv)
@@ -879,6 +942,8 @@ def main(argv=None) -> int:
         return bench_luzerax(a)
     if a.arch == "zebovik" and a.gpus == 1:
         return bench_zebovik(a)
+    if a.arch == "basitar" and a.gpus == 1:
+        return bench_basitar(a)
     if a.gpus != 1:
         print("kindi_b200 is a one-GPU library: bench.py measures N=1 only (asked for --gpus %d)" % a.gpus)
         return 2

@@ -193,6 +193,7 @@ __global__ void __launch_bounds__(32 * WK_COLS, DPL * NC > 16 ? 2 : 3) k_wkv_sca
     }
     kb_pdl_wait();
     const size_t ok = (size_t)h * d, ov = (size_t)h * dv;
+    const bool w2_vec = a.rank % 8 == 0 && ((uintptr_t)a.w2 & 15) == 0;
     for (int c0 = r0; c0 < r1; c0 += WK_STAGE) {
         const int n = min(WK_STAGE, r1 - c0);
         if (a.z == nullptr) {
@@ -207,14 +208,34 @@ __global__ void __launch_bounds__(32 * WK_COLS, DPL * NC > 16 ? 2 : 3) k_wkv_sca
             const size_t at = (size_t)(c0 + t) * a.ld + ok + j;
             rs[idx] = wk_rd<T>((const T*)a.r + at, a.n_planes, a.plane_stride);
             ks[idx] = wk_rd<T>((const T*)a.k + at, a.n_planes, a.plane_stride);
-            float z;
-            if (a.z != nullptr) z = a.z[(size_t)(c0 + t) * a.ldz + ok + j];
-            else {
+            if (a.z != nullptr) ws[idx] = wk_decay(a.z[(size_t)(c0 + t) * a.ldz + ok + j] + a.w0[ok + j]);
+        }
+        if (a.z == nullptr) {
+            // the exponent from the low-rank projection: four lanes a channel, a quarter of the sum each (the bound is rounded
+            // up so that whole warps meet at the exchange)
+            for (int i4 = threadIdx.x; i4 < (n * d * 4 + 31) / 32 * 32; i4 += 32 * WK_COLS) {
+                const int idx = min(i4 >> 2, n * d - 1), sub = i4 & 3, t = idx / d, j = idx % d;
                 const TW* w = (const TW*)a.w2 + (ok + j) * a.rank;
-                z = 0.0f;
-                for (int q = 0; q < a.rank; q++) z = fmaf(lo[t * a.rank + q], kb_to_f<TW>(w[q]), z);
+                const float* l = lo + t * a.rank;
+                float z = 0.0f;
+                if (sizeof(TW) == 2 && w2_vec) {
+                    for (int q = sub * 8; q < a.rank; q += 32) {
+                        const uint4 v = *(const uint4*)(w + q);
+                        const __nv_bfloat162* v2 = (const __nv_bfloat162*)&v;
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const float2 f = __bfloat1622float2(v2[e]);
+                            z = fmaf(l[q + 2 * e], f.x, z);
+                            z = fmaf(l[q + 2 * e + 1], f.y, z);
+                        }
+                    }
+                } else {
+                    for (int q = sub; q < a.rank; q += 4) z = fmaf(l[q], kb_to_f<TW>(w[q]), z);
+                }
+                z += __shfl_xor_sync(0xffffffffu, z, 1);
+                z += __shfl_xor_sync(0xffffffffu, z, 2);
+                if (sub == 0 && i4 < n * d * 4) ws[idx] = wk_decay(z + a.w0[ok + j]);
             }
-            ws[idx] = wk_decay(z + a.w0[ok + j]);
         }
         for (int idx = threadIdx.x; idx < n * COLS; idx += 32 * WK_COLS) {
             const int t = idx / COLS, c = e0 + idx % COLS;

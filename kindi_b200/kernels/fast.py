@@ -382,9 +382,9 @@ def _moe_tc_ok(y, wup, wdown) -> bool:
 def _moe_products(ctx, ys, plan, wts, wup, wdown, top, act, T, gated=False, weight_on="output", act_params=None):
     E, F, width = wup.shape
     h = torch.empty((T * top, F), dtype=torch.bfloat16, device=ys.device)
-    if (gated and act == "glu_clamp" and weight_on == "output" and act_params[2] == 16 and F % 32 == 0
+    if (gated and act_params is not None and weight_on == "output" and act_params[2] == 16 and F % 32 == 0
             and T * top >= MOE_GLU_MIN_PAIRS):
-        # the clamped unit is finished in the up product's epilogue (gate and up rows alternate in groups of 16). A
+        # the gated unit is finished in the up product's epilogue (gate and up rows alternate in groups of 16). A
         # decode-sized step keeps the unit's own kernel: its tiles hold a row or two, the longer epilogue sits on the
         # step's critical path while the small kernel hides behind its neighbours (batch 8, three picks: 0.374 against
         # 0.363 ms a step at width 1024, 1.064 against 1.056 at 4096; a 2048-token prompt 1.57 against 1.65 ms)

@@ -12,7 +12,7 @@ from . import linear as L
 
 def feed_forward(ctx, y: torch.Tensor, wr: torch.Tensor, br: Optional[torch.Tensor], wup: torch.Tensor,
                  wdown: torch.Tensor, top: int, act: str, dtype: torch.dtype, *, score: str = "softmax",
-                 gated: bool = False, weight_on: str = "output", n_experts: Optional[int] = None):
+                 gated: bool = False, weight_on: str = "output", n_experts: Optional[int] = None, act_params=None):
     """32-bit planes ``[top, T, width]`` whose sum in order is the feed-forward's output: router logits ``y wr^T + br``
     with 32-bit accumulation, the ``top`` largest per row weighted by the softmax over those alone (``score``
     "sigmoid": by each one's own sigmoid), plane k of a row = its k-th weight times ``W_down[e] act(W_up[e] y)``.
@@ -20,19 +20,22 @@ def feed_forward(ctx, y: torch.Tensor, wr: torch.Tensor, br: Optional[torch.Tens
     the return value is then ``(planes, logits)``"""
     logits = L.linear(ctx, y, wr, torch.float32)
     idx, wts = K.moe_topk(logits, br, top, score, n_experts)
-    planes = experts(ctx, y, idx, wts, wup, wdown, top, act, dtype, gated=gated, weight_on=weight_on)
+    planes = experts(ctx, y, idx, wts, wup, wdown, top, act, dtype, gated=gated, weight_on=weight_on, act_params=act_params)
     return planes if n_experts is None else (planes, logits)
 
 
 def gate_mul(gu: torch.Tensor, wts: Optional[torch.Tensor], plan, act: str, h: torch.Tensor, act_params=None) -> None:
-    """the gated experts' ``act(g) * u`` over the plan's sorted rows ``gu`` = [gate | up]; ``act`` "glu_clamp" with
-    ``act_params`` = (limit, alpha, group): ``g' sigmoid(alpha g') (u' + 1)``, gate clamped from above, up from both
-    sides; the expert's gate and up columns alternate in groups of ``group`` (the inner size: all gates, then all ups)"""
-    if act == "glu_clamp":
+    """the gated experts' ``act(g) * u`` over the plan's sorted rows ``gu`` = [gate | up]. With ``act_params`` = (limit, alpha,
+    group) the expert's gate and up columns alternate in groups of ``group`` (the inner size: all gates, then all ups), and
+    ``act`` may be "glu_clamp": ``g' sigmoid(alpha g') (u' + 1)``, gate clamped from above, up from both sides"""
+    if act_params is not None:
         if wts is not None:
-            raise ValueError("a weight on the input of experts with the clamped unit")
+            raise ValueError("a weight on the input of experts whose gate and up rows alternate")
         limit, alpha, group = act_params
-        K.glu_clamp(gu, h, group, limit, alpha)
+        if act == "glu_clamp":
+            K.glu_clamp(gu, h, group, limit, alpha)
+        else:
+            K.swiglu(gu, h, group, act)
     else:
         K.moe_gate_mul(gu, wts, plan, act, h)
 

@@ -102,10 +102,12 @@ class MixtureOfExperts(FeedForward):
         if self.act not in K.ACT and not (self.act == "glu_clamp" and spec.get("gated")):
             raise ValueError("unknown activation %r; known: %s, and glu_clamp for gated experts"
                              % (self.act, ", ".join(sorted(K.ACT))))
-        # (the clamped unit's gate and up rows alternate in groups that the products' epilogues can finish, like a dense
-        # gated feed-forward's)
-        self.act_params = (float(spec["limit"]), float(spec.get("alpha", 1.702)),
-                           L.GATE_UP_GROUP if self.f % L.GATE_UP_GROUP == 0 else self.f) if self.act == "glu_clamp" else None
+        # gated experts whose weight sits on their output: gate and up rows alternate in groups that the products' epilogues can
+        # finish, like a dense gated feed-forward's. (limit and alpha of the clamped unit, the group's size)
+        self.act_params = None
+        if spec.get("gated") and self.act in K.GATE_ACT and str(spec.get("weight_on") or "output") == "output":
+            clamp = (float(spec["limit"]), float(spec.get("alpha", 1.702))) if self.act == "glu_clamp" else (0.0, 0.0)
+            self.act_params = clamp + (L.GATE_UP_GROUP if self.f % L.GATE_UP_GROUP == 0 else self.f,)
         self.n_identity = int(spec.get("identity") or 0)
         self.n_out = self.E + self.n_identity
         n = self._names(spec)
@@ -150,7 +152,7 @@ class MixtureOfExperts(FeedForward):
             gates = [weights(n["gate"] % e) for e in range(self.E)]
             if {w.dtype for w in gates} != {ups[0].dtype}:
                 raise ValueError("the expert weights of %s are stored in different dtypes" % weights.prefix)
-            if self.act == "glu_clamp":
+            if self.act_params is not None:
                 ups = [L.join_gate_up(g, u)[0] for g, u in zip(gates, ups)]   # gate and up rows in groups of 16 (or all)
             else:
                 ups = [torch.cat([g, u], dim=0) for g, u in zip(gates, ups)]  # every expert: its gate rows, then up
@@ -197,7 +199,7 @@ class MixtureOfExperts(FeedForward):
                 h = L.gate_up_swiglu(ctx, y, wgu, group, fs, self.dtype, act)
             return Branch(torch.cat([planes, L.planes(ctx, h, wd)], dim=0))
         out = M.feed_forward(ctx, y, self.wr, self.br, self.wup, self.wdown, self.top, self.act, self.dtype,
-                             score=self.score, gated=self.gated, weight_on=self.weight_on,
+                             score=self.score, gated=self.gated, weight_on=self.weight_on, act_params=self.act_params,
                              n_experts=self.E if self.shared is not None and self.row_gate else None)
         if self.shared is None:
             return Branch(out)
