@@ -3,7 +3,8 @@
 // latent into the cache, per-head products), and the decayed outer-product recurrence of linear attention.
 // Storage is float or bf16, all arithmetic 32-bit; every sum has an order that depends on sizes and positions only,
 // so a row's result does not depend on the batch or on how a prompt was cut into steps.
-#include "common.cuh"
+#include "sm100.cuh"
+#include "mma_sync.cuh"
 
 // element i of a row that came either as a row or as 32-bit planes whose sum (in order) it is
 template <typename TIN>
@@ -135,37 +136,55 @@ __device__ __forceinline__ void mx_angle(const MxRot& r, int p, int i, float& c,
     c = __fmul_rn(c, r.mult);
     s = __fmul_rn(s, r.mult);
 }
+// A block takes one row's query latent (blockIdx.y = 0) or its key/value latent and rotated part (1). Elements are summed over
+// their planes once, all planes' loads in flight together, and kept in shared memory.
+#define LP_THREADS 512
+template <typename TIN>
+__device__ __forceinline__ float mx_rd8(const TIN* src, int n_planes, size_t plane_stride, size_t i) {
+    float v = kb_to_f<TIN>(src[i]);
+    for (int s0 = 1; s0 < n_planes; s0 += 8) {
+        float t[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) t[j] = s0 + j < n_planes ? kb_to_f<TIN>(src[(size_t)(s0 + j) * plane_stride + i]) : 0.0f;
+#pragma unroll
+        for (int j = 0; j < 8; j++)
+            if (s0 + j < n_planes) v += t[j];
+    }
+    return v;
+}
 template <typename TIN, typename TW, typename T>
-__global__ void __launch_bounds__(256) k_latent_prep(const TIN* KB_STEP_DATA in, int n_planes, size_t plane_stride,
+__global__ void __launch_bounds__(LP_THREADS) k_latent_prep(const TIN* KB_STEP_DATA in, int n_planes, size_t plane_stride,
         int ld_in, int q_rank, int kv_rank, int rot, const TW* __restrict__ wq, const TW* __restrict__ wkv, float eps,
         MxRot rr, const int* __restrict__ pos, const int* __restrict__ seq,
         const int* __restrict__ slot, T* __restrict__ cq, int ldcq, KbCacheView cv, int* status) {
-    __shared__ float red[8];
+    extern __shared__ float sv[];
+    __shared__ float red[LP_THREADS / 32];
     kb_pdl_launch();
     const int t = blockIdx.x;
+    const bool is_q = blockIdx.y == 0;
     const int p = pos[t];
     T* cqr = cq + (size_t)t * ldcq;
     kb_pdl_wait();
     if (p < 0) {                                       // a padding row of a recorded step: a defined query latent, no store
-        for (int i = threadIdx.x; i < q_rank; i += 256) cqr[i] = kb_from_f<T>(0.0f);
+        if (is_q)
+            for (int i = threadIdx.x; i < q_rank; i += LP_THREADS) cqr[i] = kb_from_f<T>(0.0f);
         return;
     }
-    const TIN* src = in + (size_t)t * ld_in;
-    float sq = 0.0f, sc = 0.0f;
-    for (int i = threadIdx.x; i < q_rank; i += 256) {
-        const float v = mx_rd<TIN>(src, n_planes, plane_stride, i);
-        sq = fmaf(v, v, sq);
+    const TIN* src = in + (size_t)t * ld_in + (is_q ? 0 : q_rank);
+    const int n = is_q ? q_rank : kv_rank, n_all = is_q ? n : n + rot;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < n_all; i += LP_THREADS) {
+        const float v = mx_rd8<TIN>(src, n_planes, plane_stride, i);
+        sv[i] = v;
+        if (i < n) ss = fmaf(v, v, ss);
     }
-    for (int i = threadIdx.x; i < kv_rank; i += 256) {
-        const float v = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + i);
-        sc = fmaf(v, v, sc);
+    const float tot = mx_block_sum(ss, red);           // (its barriers also cover sv)
+    const float scale = 1.0f / sqrtf(tot / (float)n + eps);
+    if (is_q) {
+        for (int i = threadIdx.x; i < n; i += LP_THREADS)
+            cqr[i] = kb_from_f<T>(__fmul_rn(__fmul_rn(scale, sv[i]), kb_to_f<TW>(wq[i])));
+        return;
     }
-    const float tq = mx_block_sum(sq, red);
-    const float tc = mx_block_sum(sc, red);
-    const float scale_q = 1.0f / sqrtf(tq / (float)q_rank + eps);
-    const float scale_c = 1.0f / sqrtf(tc / (float)kv_rank + eps);
-    for (int i = threadIdx.x; i < q_rank; i += 256)
-        cqr[i] = kb_from_f<T>(__fmul_rn(__fmul_rn(scale_q, mx_rd<TIN>(src, n_planes, plane_stride, i)), kb_to_f<TW>(wq[i])));
     const int s = slot[seq[t]];
     const int page = cv.table[(size_t)s * cv.table_stride + p / KB_PAGE];
     if (page < 0 || page >= cv.n_pages) {
@@ -174,25 +193,23 @@ __global__ void __launch_bounds__(256) k_latent_prep(const TIN* KB_STEP_DATA in,
     }
     T* kd = (T*)cv.pool + kb_kv_offset(cv, page, 0, 0, p % KB_PAGE);
     T* vd = (T*)cv.pool + kb_kv_offset(cv, page, 1, 0, p % KB_PAGE);
-    for (int i = threadIdx.x; i < kv_rank; i += 256) {
-        const T c = kb_from_f<T>(__fmul_rn(__fmul_rn(scale_c, mx_rd<TIN>(src, n_planes, plane_stride, q_rank + i)),
-                                           kb_to_f<TW>(wkv[i])));
+    for (int i = threadIdx.x; i < n; i += LP_THREADS) {
+        const T c = kb_from_f<T>(__fmul_rn(__fmul_rn(scale, sv[i]), kb_to_f<TW>(wkv[i])));
         kd[i] = c;
         if (!cv.one_plane) vd[i] = c;
     }
-    for (int i = threadIdx.x; i < rot / 2; i += 256) {
+    for (int i = threadIdx.x; i < rot / 2; i += LP_THREADS) {
         float c, sn;
         int ia, ib;
         mx_angle<sizeof(T) == 4>(rr, p, i, c, sn);
         mx_pair(rr, i, rot, ia, ib);
-        const float a = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + kv_rank + ia);
-        const float b = mx_rd<TIN>(src, n_planes, plane_stride, q_rank + kv_rank + ib);
-        kd[kv_rank + ia] = kb_from_f<T>(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, sn)));
-        kd[kv_rank + ib] = kb_from_f<T>(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
+        const float x = sv[n + ia], y = sv[n + ib];
+        kd[n + ia] = kb_from_f<T>(__fsub_rn(__fmul_rn(x, c), __fmul_rn(y, sn)));
+        kd[n + ib] = kb_from_f<T>(__fadd_rn(__fmul_rn(y, c), __fmul_rn(x, sn)));
     }
-    for (int i = kv_rank + rot + threadIdx.x; i < cv.head_dim; i += 256) kd[i] = kb_from_f<T>(0.0f);
+    for (int i = n_all + threadIdx.x; i < cv.head_dim; i += LP_THREADS) kd[i] = kb_from_f<T>(0.0f);
     if (cv.one_plane) return;
-    for (int i = kv_rank + threadIdx.x; i < cv.head_dim; i += 256) vd[i] = kb_from_f<T>(0.0f);
+    for (int i = n + threadIdx.x; i < cv.head_dim; i += LP_THREADS) vd[i] = kb_from_f<T>(0.0f);
 }
 
 extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long long plane_stride, int ld_in, int q_rank,
@@ -204,8 +221,10 @@ extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long l
     const MxRot rr{freq, freq64, mult, half};
     if (rot % 2 || kv_rank + rot > D) return (int)cudaErrorInvalidValue;
     KbCacheView cv{pool, table, table_stride, n_pages, 1, D, one_plane};
+    const size_t sm = (size_t)(q_rank > kv_rank + rot ? q_rank : kv_rank + rot) * sizeof(float);
+    if (sm > 46 * 1024) return (int)cudaErrorInvalidValue;
 #define KB_LP(TIN, TW, T_)                                                                                       \
-    kb_launch(k_latent_prep<TIN, TW, T_>, T, 256, 0, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in,  \
+    kb_launch(k_latent_prep<TIN, TW, T_>, dim3(T, 2), LP_THREADS, sm, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in,  \
               q_rank, kv_rank, rot, (const TW*)wq, (const TW*)wkv, eps, rr, pos, seq, slot, (T_*)cq, ldcq, \
               cv, status)
     if (in_dtype == KB_F32 && dtype == KB_F32 && wdtype == KB_F32) KB_LP(float, float, float);
@@ -329,7 +348,7 @@ __global__ void __launch_bounds__(256) k_head_gemm(const TA* KB_STEP_DATA A, int
 
 // The same products for bf16 operands on the tensor cores (mma.sync m16n8k16, 32-bit accumulators): a block of four
 // warps takes 64 rows x 64 columns of one head, a warp 16 rows x 64 columns; K runs in blocks of 32 through shared
-// memory (rows padded to 40 elements: the fragment loads meet no bank conflicts). Needs K % 8 == 0 and 16-byte
+// memory (rows padded to 40 elements: the fragment loads meet no bank conflicts), three blocks' copies in flight. Needs K % 8 == 0 and 16-byte
 // aligned rows of A and W (the loads are 16 bytes wide); a sum's order depends on K only.
 __device__ __forceinline__ void mx_mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -340,82 +359,158 @@ __device__ __forceinline__ void mx_mma_bf16(float* c, const uint32_t* a, uint32_
 #define HM_BN 64
 #define HM_BK 32
 #define HM_LD 40
+#define HM_ST 4                 // K blocks in flight
+// what a launch of the latent queries' product does on the side (latent attention): blocks of one more column tile rotate every
+// head's rotated part, as k_latent_qrope does
+struct MxSide {
+    int on, dim, rot, at, D, ldq;
+    const bf16* q;
+    const int* pos;
+    MxRot rr;
+};
 template <typename TG>
 __global__ void __launch_bounds__(128) k_head_gemm_mma(const bf16* KB_STEP_DATA A, int lda, int ldah,
         const bf16* __restrict__ W, bf16* __restrict__ C, int ldc, int ldch, int M, int N, int K,
-        const TG* KB_STEP_DATA gate, int n_planes, size_t plane_stride, int ldg, int gph) {
-    __shared__ __align__(16) bf16 As[HM_BM * HM_LD];
-    __shared__ __align__(16) bf16 Ws[HM_BN * HM_LD];
+        const TG* KB_STEP_DATA gate, int n_planes, size_t plane_stride, int ldg, int gph, MxSide side) {
+    __shared__ __align__(16) bf16 As[HM_ST][HM_BM * HM_LD];
+    __shared__ __align__(16) bf16 Ws[HM_ST][HM_BN * HM_LD];
     kb_pdl_launch();
     const int h = blockIdx.z;
     const int m0 = blockIdx.y * HM_BM, n0 = blockIdx.x * HM_BN;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+    if (side.on && n0 >= N) {
+        // the rotated part: rows m0 .., a thread a pair
+        kb_pdl_wait();
+        const int half = side.rot / 2, rows = min(HM_BM, M - m0), tail = side.D - side.at - side.rot;
+        for (int idx = tid; idx < rows * half; idx += 128) {
+            const int m = m0 + idx / half, i = idx % half, p = side.pos[m];
+            float c, sn;
+            int ia, ib;
+            mx_angle<false>(side.rr, max(p, 0), i, c, sn);
+            mx_pair(side.rr, i, side.rot, ia, ib);
+            const bf16* src = side.q + (size_t)m * side.ldq + (size_t)h * (side.dim + side.rot) + side.dim;
+            bf16* dst = C + (size_t)m * ldc + (size_t)h * ldch + side.at;
+            const float a = p >= 0 ? __bfloat162float(src[ia]) : 0.0f, b = p >= 0 ? __bfloat162float(src[ib]) : 0.0f;
+            dst[ia] = __float2bfloat16_rn(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, sn)));
+            dst[ib] = __float2bfloat16_rn(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, sn)));
+        }
+        for (int idx = tid; idx < rows * tail; idx += 128)
+            C[(size_t)(m0 + idx / tail) * ldc + (size_t)h * ldch + side.at + side.rot + idx % tail] = __float2bfloat16_rn(0.0f);
+        return;
+    }
     const bf16* Ah = A + (size_t)h * ldah;
     const bf16* Wh = W + (size_t)h * N * K;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
     float acc[8][4];
 #pragma unroll
     for (int j = 0; j < 8; j++)
 #pragma unroll
         for (int i = 0; i < 4; i++) acc[j][i] = 0.0f;
     const int lr = tid >> 2, lc = (tid & 3) * 8;       // this thread's rows (lr, lr + 32) and 8-element piece of a K block
-    kb_pdl_wait();
-    for (int k0 = 0; k0 < K; k0 += HM_BK) {
+    const int nk = (K + HM_BK - 1) / HM_BK;
+    auto load_w = [&](int kb) {
 #pragma unroll
         for (int half = 0; half < 2; half++) {
-            const int r = lr + 32 * half, k = k0 + lc;
-            uint4 av = make_uint4(0u, 0u, 0u, 0u), wv = make_uint4(0u, 0u, 0u, 0u);
-            if (m0 + r < M && k < K) av = *(const uint4*)(Ah + (size_t)(m0 + r) * lda + k);
-            if (n0 + r < N && k < K) wv = *(const uint4*)(Wh + (size_t)(n0 + r) * K + k);
-            *(uint4*)(As + r * HM_LD + lc) = av;
-            *(uint4*)(Ws + r * HM_LD + lc) = wv;
+            const int r = lr + 32 * half, k = kb * HM_BK + lc;
+            const bool ok = n0 + r < N && k < K;
+            cp_async16(smem_u32(&Ws[kb % HM_ST][r * HM_LD + lc]), ok ? (const void*)(Wh + (size_t)(n0 + r) * K + k) : (const void*)Wh, ok);
         }
-        __syncthreads();
+    };
+    auto load_a = [&](int kb) {
+#pragma unroll
+        for (int half = 0; half < 2; half++) {
+            const int r = lr + 32 * half, k = kb * HM_BK + lc;
+            const bool ok = m0 + r < M && k < K;
+            cp_async16(smem_u32(&As[kb % HM_ST][r * HM_LD + lc]), ok ? (const void*)(Ah + (size_t)(m0 + r) * lda + k) : (const void*)Ah, ok);
+        }
+    };
+    // (the weights are fetched before the wait for the kernel that makes the activations; a group of copies a K block, the
+    // first one's with all early weights)
+#pragma unroll
+    for (int kb = 0; kb < HM_ST - 1; kb++)
+        if (kb < nk) load_w(kb);
+    kb_pdl_wait();
+#pragma unroll
+    for (int kb = 0; kb < HM_ST - 1; kb++) {
+        if (kb < nk) load_a(kb);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    for (int kb = 0; kb < nk; kb++) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(HM_ST - 2) : "memory");
+        __syncthreads();                               // block kb is there, and block kb - 1's buffer is free
+        if (kb + HM_ST - 1 < nk) {
+            load_w(kb + HM_ST - 1);
+            load_a(kb + HM_ST - 1);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        const bf16* as = As[kb % HM_ST], *ws = Ws[kb % HM_ST];
+        if (m0 + warp * 16 >= M) continue;             // (a warp without rows only copies)
 #pragma unroll
         for (int kk = 0; kk < HM_BK; kk += 16) {
             uint32_t a[4];
-            const bf16* ar = As + (warp * 16 + g) * HM_LD + kk + 2 * t;
+            const bf16* ar = as + (warp * 16 + g) * HM_LD + kk + 2 * t;
             a[0] = *(const uint32_t*)(ar);
             a[1] = *(const uint32_t*)(ar + 8 * HM_LD);
             a[2] = *(const uint32_t*)(ar + 8);
             a[3] = *(const uint32_t*)(ar + 8 * HM_LD + 8);
 #pragma unroll
             for (int j = 0; j < 8; j++) {
-                const bf16* wr = Ws + (j * 8 + g) * HM_LD + kk + 2 * t;
+                const bf16* wr = ws + (j * 8 + g) * HM_LD + kk + 2 * t;
                 mx_mma_bf16(acc[j], a, *(const uint32_t*)(wr), *(const uint32_t*)(wr + 8));
             }
         }
-        __syncthreads();
     }
+    cp_async_wait_all();
+    const bool pairs = N % 2 == 0 && ldc % 2 == 0 && ldch % 2 == 0 && ((uintptr_t)C & 3) == 0;
 #pragma unroll
     for (int j = 0; j < 8; j++)
 #pragma unroll
-        for (int i = 0; i < 4; i++) {
-            const int m = m0 + warp * 16 + g + (i >> 1) * 8, n = n0 + j * 8 + 2 * t + (i & 1);
+        for (int half = 0; half < 2; half++) {
+            const int m = m0 + warp * 16 + g + half * 8, n = n0 + j * 8 + 2 * t;
             if (m >= M || n >= N) continue;
-            float v = acc[j][i];
+            float v[2] = {acc[j][2 * half], acc[j][2 * half + 1]};
             if (gate != nullptr)
-                v *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, (size_t)h * gph + (gph > 1 ? n : 0)));
-            C[(size_t)m * ldc + (size_t)h * ldch + n] = __float2bfloat16_rn(v);
+#pragma unroll
+                for (int i = 0; i < 2; i++)
+                    if (n + i < N)
+                        v[i] *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride,
+                                                     (size_t)h * gph + (gph > 1 ? n + i : 0)));
+            bf16* dst = C + (size_t)m * ldc + (size_t)h * ldch + n;
+            if (pairs) *(__nv_bfloat162*)dst = __floats2bfloat162_rn(v[0], v[1]);
+            else {
+                dst[0] = __float2bfloat16_rn(v[0]);
+                if (n + 1 < N) dst[1] = __float2bfloat16_rn(v[1]);
+            }
         }
 }
 
 extern "C" int kb_head_gemm(const void* A, int adtype, int lda, int ldah, const void* W, int wdtype, void* C, int ldc,
                             int ldch, int M, int N, int K, int H, const void* gate, int gdtype, int n_planes,
-                            long long plane_stride, int ldg, cudaStream_t st, int tensor_cores, int gph) {
+                            long long plane_stride, int ldg, cudaStream_t st, int tensor_cores, int gph,
+                            const void* side_q, int side_ldq, int side_dim, int side_rot, int side_at, int side_D,
+                            const float* side_freq, float side_mult, int side_half, const int* side_pos) {
+    // side_q (rows of [dim | rot] heads, or null): the launch also rotates every head's last `rot` elements into
+    // C[t][h][at ..] and clears C[t][h][at + rot .. D) (see MxSide); tensor-core form only
     if (M <= 0 || N <= 0 || H <= 0) return 0;
     if (gate && gph != N && gph != 1) return (int)cudaErrorInvalidValue;
     if (H > 65535) return (int)cudaErrorInvalidValue;
     if (tensor_cores && adtype == KB_BF16 && wdtype == KB_BF16 && K % 8 == 0 && lda % 8 == 0 && ldah % 8 == 0 &&
         ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0) {
-        dim3 gm((N + HM_BN - 1) / HM_BN, (M + HM_BM - 1) / HM_BM, H);
+        MxSide side = {};
+        if (side_q) {
+            if (side_rot % 2 || side_at < N || side_at + side_rot > side_D) return (int)cudaErrorInvalidValue;
+            side = MxSide{1, side_dim, side_rot, side_at, side_D, side_ldq, (const bf16*)side_q, side_pos,
+                          MxRot{side_freq, nullptr, side_mult, side_half}};
+        }
+        dim3 gm((N + HM_BN - 1) / HM_BN + (side_q ? 1 : 0), (M + HM_BM - 1) / HM_BM, H);
         if (gate == nullptr || gdtype == KB_F32)
             kb_launch(k_head_gemm_mma<float>, gm, 128, 0, st, (const bf16*)A, lda, ldah, (const bf16*)W, (bf16*)C, ldc,
-                      ldch, M, N, K, (const float*)gate, n_planes, (size_t)plane_stride, ldg, gph);
+                      ldch, M, N, K, (const float*)gate, n_planes, (size_t)plane_stride, ldg, gph, side);
         else
             kb_launch(k_head_gemm_mma<bf16>, gm, 128, 0, st, (const bf16*)A, lda, ldah, (const bf16*)W, (bf16*)C, ldc,
-                      ldch, M, N, K, (const bf16*)gate, n_planes, (size_t)plane_stride, ldg, gph);
+                      ldch, M, N, K, (const bf16*)gate, n_planes, (size_t)plane_stride, ldg, gph, side);
         KB_LAUNCH_RET();
     }
+    if (side_q) return (int)cudaErrorInvalidValue;
     dim3 grid((N + HG_BN - 1) / HG_BN, (M + HG_BM - 1) / HG_BM, H);
 #define KB_HG(TA, TW, TG)                                                                                       \
     kb_launch(k_head_gemm<TA, TW, TG>, grid, 256, 0, st, (const TA*)A, lda, ldah, (const TW*)W, (TA*)C, ldc,    \

@@ -341,10 +341,11 @@ def attention_decode_rope(ctx, qkv, out, nh, nkv, hd, scale, window, inv_freq, r
     return True
 
 
-def latent_splits(ctx, head_tiles: int) -> int:
+def latent_splits(ctx, head_tiles: int, hd: int) -> int:
     """position splits of a decode step over a cache of latents: one wave of CTAs over all (sequence, head tile) pairs, two an
-    SM"""
-    return max(1, min(64, 2 * N_SM // max(1, ctx.B * head_tiles)))
+    SM (one for wide vectors, whose tiles fill the shared memory)"""
+    per_sm = 2 if hd <= 256 else 1
+    return max(1, min(64, per_sm * N_SM // max(1, ctx.B * head_tiles)))
 
 
 def latent_attention_bf16(ctx, q, out, nh: int, hd: int, v_dim: int, scale: float, pool, table, n_pages) -> bool:
@@ -354,7 +355,7 @@ def latent_attention_bf16(ctx, q, out, nh: int, hd: int, v_dim: int, scale: floa
         return False
     if ctx.decode:
         K.latent_attn_decode(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, hd, v_dim, scale, pool, table, n_pages,
-                             splits=latent_splits(ctx, 1 if nh <= 16 else -(-nh // 32)), status=ctx.status)
+                             splits=latent_splits(ctx, 1 if nh <= 16 else -(-nh // 32), hd), status=ctx.status)
         return True
     group = next((g for g in range(min(nh, 128), 0, -1) if nh % g == 0))
     K.latent_attn_tc(q, out, ctx.slot, ctx.q_start, ctx.kv_len, ctx.B, nh, group, hd, v_dim, scale, pool, table, n_pages,

@@ -75,7 +75,8 @@ _SIGS = {
     "kb_latent_qrope": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
                         c_int, c_int, c_int, c_void_p, c_void_p, c_int],
     "kb_head_gemm": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                     c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int],
+                     c_int, c_void_p, c_int, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                     c_int, c_int, c_void_p, c_float, c_int, c_void_p],
     "kb_decay_chunked": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "kb_decay_scan": [c_void_p, c_int, c_int, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
@@ -552,12 +553,13 @@ def latent_qrope(q: torch.Tensor, dim: int, rot: int, freq: torch.Tensor, mult: 
 
 
 def head_gemm(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
-              gate: Optional[torch.Tensor] = None, tensor_cores: bool = True) -> None:
+              gate: Optional[torch.Tensor] = None, tensor_cores: bool = True, side=None) -> None:
     """per head h: out[t][h * out_head_stride + n] = sum_k a[t][h * a_head_stride + k] * w[h][n][k]; w [H, N, K].
     ``gate`` (rows or 32-bit planes [.., T, H * N], or [.., T, H] for one number a head): the result is multiplied by its
-    logistic function. bf16 operands
-    whose rows are 16-byte aligned (K, strides multiples of 8) run on the tensor cores unless ``tensor_cores`` is
-    False; everything else takes 32-bit multiply-adds in a fixed order"""
+    logistic function. bf16 operands whose rows are 16-byte aligned (K, strides multiples of 8) run on the tensor cores
+    unless ``tensor_cores`` is False; everything else takes 32-bit multiply-adds in a fixed order. ``side`` (only where
+    ``head_gemm_on_tensor_cores`` says yes): ``(q, dim, rot, at, head_dim, freq, mult, pairing, pos)``, the launch also does
+    ``latent_qrope`` of these arguments into ``out``"""
     _need_cuda(a, w, out, gate)
     H, N, Kd = w.shape
     M = a.shape[0]
@@ -566,10 +568,23 @@ def head_gemm(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.T
     n_planes, pstride, ldg = _planes_of(gate) if gate is not None else (1, 0, 0)
     if gate is not None:
         assert gate.shape[-2:] in ((M, H * N), (M, H))
+    more = (None, 0, 0, 0, 0, 0, None, 0.0, 0, None)
+    if side is not None:
+        q, dim, rot, at, head_dim, freq, mult, pairing, pos = side
+        _need_cuda(q, freq, pos)
+        assert q.dtype == torch.bfloat16 and q.shape == (M, H * (dim + rot)) and q.stride(1) == 1 and out_head_stride == head_dim
+        assert freq.dtype == torch.float32 and freq.numel() >= rot // 2 and tensor_cores
+        more = (_p(q), q.stride(0), dim, rot, at, head_dim, _p(freq), float(mult), PAIRING[pairing], _p(pos))
     _check(load().kb_head_gemm(_p(a), dt(a), a.stride(0), a_head_stride, _p(w), dt(w), _p(out), out.stride(0),
                                out_head_stride, M, N, Kd, H, _p(gate), dt(gate) if gate is not None else F32, n_planes,
                                pstride, ldg, _stream(), 1 if tensor_cores else 0,
-                               gate.shape[-1] // H if gate is not None else 1), "head_gemm")
+                               gate.shape[-1] // H if gate is not None else 1, *more), "head_gemm")
+
+
+def head_gemm_on_tensor_cores(a: torch.Tensor, a_head_stride: int, w: torch.Tensor) -> bool:
+    """whether ``head_gemm`` of these operands runs on the tensor cores"""
+    return (a.dtype == w.dtype == torch.bfloat16 and w.shape[2] % 8 == 0 and a.stride(0) % 8 == 0 and a_head_stride % 8 == 0
+            and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
 def decay_scan(a: torch.Tensor, B: int, H: int, d: int, dv: int, decay: torch.Tensor, q_start, slot,

@@ -124,8 +124,11 @@ class LatentAttention(Mixer):
                       cq, D, pool, table, n_pages, ctx.status, **turn)
         q = L.linear(ctx, cq, self.w_uq, self.dtype)
         qf = torch.empty((ctx.T, H * D), dtype=self.dtype, device=y.device)
-        K.head_gemm(q, d + r, self.w_uk_t, qf, D)
-        K.latent_qrope(q, d, r, pos.inv_freq, pos.mult, ctx.pos, qf, kr, D, H, **turn)
+        if K.head_gemm_on_tensor_cores(q, d + r, self.w_uk_t):
+            K.head_gemm(q, d + r, self.w_uk_t, qf, D, side=(q, d, r, kr, D, pos.inv_freq, pos.mult, pos.pairing, ctx.pos))
+        else:
+            K.head_gemm(q, d + r, self.w_uk_t, qf, D)
+            K.latent_qrope(q, d, r, pos.inv_freq, pos.mult, ctx.pos, qf, kr, D, H, **turn)
         att = torch.empty((ctx.T, H * self.vd), dtype=self.dtype, device=y.device)
         A.latent_attention(ctx, qf, att, H, D, self.vd, self.scale, pool, table, n_pages)
         o = torch.empty((ctx.T, H * dv), dtype=self.dtype, device=y.device)
