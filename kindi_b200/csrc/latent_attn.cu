@@ -12,6 +12,11 @@
 //                    scores 16 of a page's 64 positions, the scores meet in shared memory, and each warp then has the whole
 //                    page's weights for its quarter of the value columns.
 //   k_latent_merge   position splits of a decode step, merged in split order.
+//   k_latent_full    prompt-sized steps with every head's keys and values expanded from the latents (a product over all cached
+//                    positions of the step's sequences, gathered by k_latent_gather): fewer multiplications per query and key,
+//                    worth their making where a step brings a fair share of its sequences' positions. A CTA takes 128 tokens
+//                    of one head; its key tile is the head's plain part beside the rotated part that all heads share. The
+//                    queries' rotation happens on their way into shared memory, a gate per head on the way out.
 // bf16 in and out, 32-bit sums and softmax; every wait is bounded.
 #include "sm100.cuh"
 #include "mma_sync.cuh"
@@ -54,6 +59,80 @@ __device__ __forceinline__ uint64_t lt_desc_mn(uint32_t smem_addr, uint32_t lbo_
     d |= (uint64_t)1 << 46;
     d |= (uint64_t)2 << 61;
     return d;
+}
+
+// one tile of a softmax thread's row: scores from tensor memory (t_s, this warp's lanes), probabilities back over them as bf16,
+// O (t_o, n_cols columns) rescaled where the row's reference moved, then the tile handed over to the product with the values.
+// False: a wait ran out
+template <int KEYS>
+__device__ __forceinline__ bool lt_softmax_tile(uint32_t t_s, uint32_t t_o, int n_cols, int j, int key0, int p_row,
+        float scale_log2e, float& m_ref, float& l, uint32_t b_pv_done, uint32_t b_p_ready, int lane, int* status) {
+    tc_fence_after();
+    uint32_t sv[KEYS];
+#pragma unroll
+    for (int c = 0; c < KEYS; c += 32) tmem_ld_32x32(t_s + c, sv + c);
+    tmem_ld_wait();
+    tc_fence_before();
+    __syncwarp();
+    float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+    if (key0 + KEYS - 1 <= p_row) {
+#pragma unroll
+        for (int c = 0; c < KEYS; c++) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c]));
+    } else {
+#pragma unroll
+        for (int c = 0; c < KEYS; c++) {
+            const float s = key0 + c <= p_row ? __uint_as_float(sv[c]) : -INFINITY;
+            sv[c] = __float_as_uint(s);
+            mx4[c & 3] = fmaxf(mx4[c & 3], s);
+        }
+    }
+    const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2e;
+    const bool grow = mx > m_ref + LT_LAZY || (m_ref == -INFINITY && mx > -INFINITY);
+    float f = 1.0f;
+    if (grow) {
+        f = m_ref == -INFINITY ? 0.0f : lt_exp2(m_ref - mx);
+        m_ref = mx;
+        l *= f;
+    }
+    // P V of tile j - 1 done means: O holds tiles 0..j-1. A rescale of O waits for that here, otherwise the wait comes
+    // just before this tile's P is handed over (once per tile, in order)
+    const bool rescale = __any_sync(0xffffffffu, grow) && j > 0;
+    if (rescale) {
+        if (!mbar_wait(b_pv_done, (uint32_t)(j - 1) & 1u, status)) return false;
+        __syncwarp();
+        tc_fence_after();
+#pragma unroll 1
+        for (int c0 = 0; c0 < n_cols; c0 += 32) {
+            uint32_t ov[32];
+            tmem_ld_32x32(t_o + c0, ov);
+            tmem_ld_wait();
+#pragma unroll
+            for (int c = 0; c < 32; c++) ov[c] = __float_as_uint(__uint_as_float(ov[c]) * f);
+            lt_tmem_st32(t_o + c0, ov);
+        }
+        lt_tmem_st_wait();
+    }
+    const float nmr = m_ref == -INFINITY ? 0.0f : -m_ref;
+    float sum[4] = {0.f, 0.f, 0.f, 0.f};
+    uint32_t pv[KEYS / 2];
+#pragma unroll
+    for (int c = 0; c < KEYS; c += 2) {
+        const float p0 = lt_exp2(fmaf(__uint_as_float(sv[c]), scale_log2e, nmr));
+        const float p1 = lt_exp2(fmaf(__uint_as_float(sv[c + 1]), scale_log2e, nmr));
+        sum[(c >> 1) & 3] += p0 + p1;
+        pv[c >> 1] = pack_bf16(p0, p1);
+    }
+    l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
+    if (KEYS == 64) lt_tmem_st32(t_s, pv);
+    else lt_tmem_st16(t_s, pv);
+    lt_tmem_st_wait();
+    if (j > 0 && !rescale) {
+        if (!mbar_wait(b_pv_done, (uint32_t)(j - 1) & 1u, status)) return false;
+    }
+    tc_fence_before();
+    __syncwarp();
+    if (lane == 0) mbar_arrive(b_p_ready);
+    return true;
 }
 
 template <int HD, int KEYS, int STAGES>
@@ -215,72 +294,8 @@ __global__ void __launch_bounds__(LT_THREADS, 2 * LtSmem<HD, KEYS, STAGES>::TOTA
             const int bsel = j & 1;
             if (!(ok = mbar_wait(b_s_full + bsel * 8, (uint32_t)(j >> 1) & 1u, status))) break;
             __syncwarp();
-            tc_fence_after();
-            uint32_t sv[KEYS];
-#pragma unroll
-            for (int c = 0; c < KEYS; c += 32) tmem_ld_32x32(t_s + lane_base + bsel * KEYS + c, sv + c);
-            tmem_ld_wait();
-            tc_fence_before();
-            __syncwarp();
-            const int key0 = j * KEYS;
-            float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-            if (key0 + KEYS - 1 <= p_row) {
-#pragma unroll
-                for (int c = 0; c < KEYS; c++) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c]));
-            } else {
-#pragma unroll
-                for (int c = 0; c < KEYS; c++) {
-                    const float s = key0 + c <= p_row ? __uint_as_float(sv[c]) : -INFINITY;
-                    sv[c] = __float_as_uint(s);
-                    mx4[c & 3] = fmaxf(mx4[c & 3], s);
-                }
-            }
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2e;
-            const bool grow = mx > m_ref + LT_LAZY || (m_ref == -INFINITY && mx > -INFINITY);
-            float f = 1.0f;
-            if (grow) {
-                f = m_ref == -INFINITY ? 0.0f : lt_exp2(m_ref - mx);
-                m_ref = mx;
-                l *= f;
-            }
-            // P V of tile j - 1 done means: O holds tiles 0..j-1. A rescale of O waits for that here, otherwise the wait comes
-            // just before this tile's P is handed over (once per tile, in order)
-            const bool rescale = __any_sync(0xffffffffu, grow) && j > 0;
-            if (rescale) {
-                if (!(ok = mbar_wait(b_pv_done, (uint32_t)(j - 1) & 1u, status))) break;
-                __syncwarp();
-                tc_fence_after();
-#pragma unroll 1
-                for (int c0 = 0; c0 < n_cols; c0 += 32) {
-                    uint32_t ov[32];
-                    tmem_ld_32x32(t_o + lane_base + c0, ov);
-                    tmem_ld_wait();
-#pragma unroll
-                    for (int c = 0; c < 32; c++) ov[c] = __float_as_uint(__uint_as_float(ov[c]) * f);
-                    lt_tmem_st32(t_o + lane_base + c0, ov);
-                }
-                lt_tmem_st_wait();
-            }
-            const float nmr = m_ref == -INFINITY ? 0.0f : -m_ref;
-            float sum[4] = {0.f, 0.f, 0.f, 0.f};
-            uint32_t pv[KEYS / 2];
-#pragma unroll
-            for (int c = 0; c < KEYS; c += 2) {
-                const float p0 = lt_exp2(fmaf(__uint_as_float(sv[c]), scale_log2e, nmr));
-                const float p1 = lt_exp2(fmaf(__uint_as_float(sv[c + 1]), scale_log2e, nmr));
-                sum[(c >> 1) & 3] += p0 + p1;
-                pv[c >> 1] = pack_bf16(p0, p1);
-            }
-            l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
-            if (KEYS == 64) lt_tmem_st32(t_s + lane_base + bsel * KEYS, pv);
-            else lt_tmem_st16(t_s + lane_base + bsel * KEYS, pv);
-            lt_tmem_st_wait();
-            if (j > 0 && !rescale) {
-                if (!(ok = mbar_wait(b_pv_done, (uint32_t)(j - 1) & 1u, status))) break;
-            }
-            tc_fence_before();
-            __syncwarp();
-            if (lane == 0) mbar_arrive(b_p_ready);
+            ok = lt_softmax_tile<KEYS>(t_s + lane_base + bsel * KEYS, t_o + lane_base, n_cols, j, j * KEYS, p_row, scale_log2e, m_ref,
+                                       l, b_pv_done, b_p_ready, lane, status);
         }
         if (ok) ok = mbar_wait(b_pv_done, (uint32_t)(n_iter - 1) & 1u, status);
         ok = __all_sync(0xffffffffu, ok);
@@ -319,6 +334,284 @@ __global__ void __launch_bounds__(LT_THREADS, 2 * LtSmem<HD, KEYS, STAGES>::TOTA
     if (warp == 5) {
         tc_fence_after();
         tmem_dealloc(tmem, tmem_cols);
+    }
+}
+
+// ------------------------------------------------------------------------------------------------ expanded keys and values
+// the cached latents and rotated parts of the step's sequences, one after another: row sum(kv_len[0 .. b)) + p of lat [N][kr] and
+// rotk [N][rot]. A warp a row; 16-byte words
+__global__ void __launch_bounds__(256) k_latent_gather(const bf16* KB_STEP_DATA pool, int hd, int kr, int rot,
+        const int* __restrict__ slot, const int* __restrict__ kv_len, int B, const int* __restrict__ table, int table_stride,
+        int n_pages, bf16* __restrict__ lat, bf16* __restrict__ rotk, int N, int* status) {
+    kb_pdl_launch();
+    kb_pdl_wait();
+    const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (row >= N) return;
+    int b = 0, p = row;
+    while (b + 1 < B && p >= kv_len[b]) p -= kv_len[b++];
+    const int page = p < kv_len[b] ? table[(size_t)slot[b] * table_stride + p / KB_PAGE] : -1;
+    const bool ok = page >= 0 && page < n_pages;
+    if (!ok && lane == 0) atomicOr(status, KB_ST_BAD_PAGE);
+    const uint4* src = (const uint4*)(pool + ((size_t)(ok ? page : 0) * KB_PAGE + p % KB_PAGE) * hd);
+    for (int c = lane; c < (kr + rot) / 8; c += 32) {
+        const uint4 v = ok ? src[c] : make_uint4(0, 0, 0, 0);
+        if (c * 8 < kr) *(uint4*)(lat + (size_t)row * kr + c * 8) = v;
+        else *(uint4*)(rotk + (size_t)row * rot + c * 8 - kr) = v;
+    }
+}
+
+template <int KBX, int VBX>
+struct LfSmem {
+    static constexpr int QB = KBX + 1;
+    static constexpr int Q_BYTES = QB * 16384, K_BYTES = QB * 8192, V_BYTES = VBX * 8192;
+    static constexpr int V_OFF = Q_BYTES + 2 * K_BYTES, BARS = V_OFF + V_BYTES;
+    static constexpr int TOTAL = BARS + 96 + 896;      // (the base is 128-byte aligned and moves up to the next 1024)
+};
+struct LfArgs {
+    const bf16* q;              // rows [T][ldq]: heads of [d | rot]
+    int ldq, d, rot, dv, n_heads;
+    const float2* angles;       // [T][rot / 2]: cosine and sine of the row's angles
+    float mult;
+    int half;                   // pairs (i, i + rot / 2) instead of neighbours
+    const bf16* gate;           // rows [T][ldg], one number a head, or null
+    int ldg;
+    bf16* out;                  // rows [T][ldo]: heads of dv
+    int ldo;
+    const int* q_start;
+    const int* kv_len;
+    float scale_log2e;
+    int* status;
+};
+
+// kvmap: [N][n_heads d keys | n_heads dv values]; rotmap: [N][rot]. grid (heads, tiles of 128 tokens, sequences)
+template <int KBX, int VBX>
+__global__ void __launch_bounds__(LT_THREADS, 2) k_latent_full(const __grid_constant__ CUtensorMap kvmap,
+        const __grid_constant__ CUtensorMap rotmap, LfArgs a) {
+    using L = LfSmem<KBX, VBX>;
+    constexpr int QB = L::QB;
+    extern __shared__ __align__(128) uint8_t smem_raw[];
+    uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+    const uint32_t sbase = smem_u32(smem);
+    const uint32_t s_q = sbase, s_k = s_q + L::Q_BYTES, s_v = sbase + L::V_OFF;
+    const uint32_t b_k_full = sbase + L::BARS, b_k_empty = b_k_full + 16, b_v_full = b_k_empty + 16, b_v_empty = b_v_full + 8;
+    const uint32_t b_s_full = b_v_empty + 8, b_p_ready = b_s_full + 16, b_pv_done = b_p_ready + 8;
+    volatile uint32_t* tmem_slot = (volatile uint32_t*)(smem + L::BARS + 80);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int h = blockIdx.x, b = blockIdx.z;
+    const int n_cols = (a.dv + 15) / 16 * 16;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < 2; i++) {
+            mbar_init(b_k_full + i * 8, 1);
+            mbar_init(b_k_empty + i * 8, 1);
+            mbar_init(b_s_full + i * 8, 1);
+        }
+        mbar_init(b_v_full, 1);
+        mbar_init(b_v_empty, 1);
+        mbar_init(b_p_ready, 4);
+        mbar_init(b_pv_done, 1);
+        mbar_fence_init();
+        tma_prefetch_desc(&kvmap);
+        tma_prefetch_desc(&rotmap);
+    }
+    if (warp == 5) {
+        tmem_alloc(smem_u32((const void*)tmem_slot), 256);
+        tmem_relinquish();
+    }
+    kb_pdl_wait();
+    const int qs0 = a.q_start[b], qlen = a.q_start[b + 1] - qs0, kvl = a.kv_len[b];
+    int kv0 = 0;                                     // the sequence's first row among the expanded ones
+    for (int i = 0; i < b; i++) kv0 += a.kv_len[i];
+    const int pos0 = kvl - qlen;
+    const int n_tiles = (qlen + 127) / 128;
+    const bool active = (int)blockIdx.y < n_tiles;
+    const int tok0 = (n_tiles - 1 - (int)blockIdx.y) * 128;          // the longest tiles first
+    const int nrows = active ? min(128, qlen - tok0) : 0;
+    const int n_iter = active ? (pos0 + tok0 + nrows - 1) / 64 + 1 : 0;
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    const uint32_t t_s = tmem, t_o = tmem + 128;
+
+    if (warp != 4) {
+        if (active) {
+            constexpr int QT = LT_THREADS - 32, QV = 128 * QB * 8, QN = 8;
+            const int qt = warp < 4 ? (int)threadIdx.x : (int)threadIdx.x - 32;
+            const int rh = a.rot / 2;
+#pragma unroll 1
+            for (int e0 = 0; e0 < QV; e0 += QT * QN) {
+                uint4 v[QN], w[QN];
+#pragma unroll
+                for (int i = 0; i < QN; i++) {
+                    const int e = e0 + qt + i * QT, r = e / (QB * 8), c = e % (QB * 8);
+                    v[i] = w[i] = make_uint4(0, 0, 0, 0);
+                    if (e < QV && r < nrows) {
+                        const bf16* row = a.q + (size_t)(qs0 + tok0 + r) * a.ldq + (size_t)h * (a.d + a.rot);
+                        const int x = (c - KBX * 8) * 8;             // (rotated part)
+                        if (c < KBX * 8) {
+                            if (c * 8 < a.d) v[i] = *(const uint4*)(row + c * 8);
+                        } else if (x < a.rot) {
+                            v[i] = *(const uint4*)(row + a.d + x);
+                            if (a.half) w[i] = *(const uint4*)(row + a.d + (x < rh ? x + rh : x - rh));
+                        }
+                    }
+                }
+#pragma unroll
+                for (int i = 0; i < QN; i++) {
+                    const int e = e0 + qt + i * QT, r = e / (QB * 8), c = e % (QB * 8);
+                    if (e >= QV) continue;
+                    const int x = (c - KBX * 8) * 8;
+                    if (c >= KBX * 8 && x < a.rot && r < nrows) {
+                        const float2* an = a.angles + (size_t)(qs0 + tok0 + r) * rh;
+                        const bf16* vb = (const bf16*)&v[i], *wb = (const bf16*)&w[i];
+                        float y[8];
+                        if (a.half) {
+                            const bool lo = x < rh;
+#pragma unroll
+                            for (int k = 0; k < 8; k++) {
+                                const float2 cs = an[(lo ? x : x - rh) + k];
+                                const float m = __bfloat162float(vb[k]) * (cs.x * a.mult), o = __bfloat162float(wb[k]) * (cs.y * a.mult);
+                                y[k] = lo ? m - o : m + o;
+                            }
+                        } else {
+#pragma unroll
+                            for (int k = 0; k < 8; k += 2) {
+                                const float2 cs = an[(x + k) / 2];
+                                const float u0 = __bfloat162float(vb[k]), u1 = __bfloat162float(vb[k + 1]);
+                                const float cc = cs.x * a.mult, sn = cs.y * a.mult;
+                                y[k] = u0 * cc - u1 * sn;
+                                y[k + 1] = u1 * cc + u0 * sn;
+                            }
+                        }
+                        v[i] = make_uint4(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]), pack_bf16(y[4], y[5]), pack_bf16(y[6], y[7]));
+                    }
+                    *(uint4*)(smem + (c >> 3) * 16384 + r * 128 + (((c & 7) ^ (r & 7)) << 4)) = v[i];
+                }
+            }
+            asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        }
+        asm volatile("bar.sync 1, %0;" ::"n"(LT_THREADS - 32) : "memory");
+    }
+
+    if (warp == 4) {
+        // ------------------------------------------------------------ TMA producer: two streams, one thread polls both
+        if (lane == 0 && n_iter > 0) {
+            int ik = 0, iv = 0, spins = 0;
+            uint64_t t0 = 0;
+            while (iv < n_iter) {
+                bool moved = false;
+                if (ik < n_iter && mbar_poll(b_k_empty + (ik & 1) * 8, ((uint32_t)(ik >> 1) & 1u) ^ 1u)) {
+                    const uint32_t dst = s_k + (ik & 1) * L::K_BYTES, bar = b_k_full + (ik & 1) * 8;
+                    mbar_expect_tx(bar, L::K_BYTES);
+#pragma unroll
+                    for (int c = 0; c < KBX; c++) tma_load_2d(dst + c * 8192, &kvmap, h * a.d + c * 64, kv0 + ik * 64, bar);
+                    tma_load_2d(dst + KBX * 8192, &rotmap, 0, kv0 + ik * 64, bar);
+                    ik++;
+                    moved = true;
+                }
+                if (iv < ik && mbar_poll(b_v_empty, ((uint32_t)iv & 1u) ^ 1u)) {
+                    mbar_expect_tx(b_v_full, L::V_BYTES);
+#pragma unroll
+                    for (int c = 0; c < VBX; c++)
+                        tma_load_2d(s_v + c * 8192, &kvmap, a.n_heads * a.d + h * a.dv + c * 64, kv0 + iv * 64, b_v_full);
+                    iv++;
+                    moved = true;
+                }
+                if (moved) {
+                    spins = 0;
+                    continue;
+                }
+                __nanosleep(100);
+                if (++spins >= 256) {
+                    if (spins == 256) t0 = kb_globaltimer();
+                    else if ((spins & 255) == 0 && kb_globaltimer() - t0 > KB_WAIT_NS) {
+                        atomicOr(a.status, KB_ST_WAIT_TIMEOUT);
+                        break;
+                    }
+                }
+            }
+        }
+    } else if (warp == 5) {
+        // ------------------------------------------------------------ MMA issuer
+        if (lane == 0 && n_iter > 0) {
+            constexpr uint32_t idesc_s = umma_idesc_bf16(128, 64);
+            const uint32_t idesc_o = umma_idesc_bf16(128, n_cols) | (1u << 16);
+            bool ok = true;
+            auto issue_s = [&](int j) {
+                const uint32_t kt = s_k + (j & 1) * L::K_BYTES, d = t_s + (uint32_t)(j & 1) * 64;
+#pragma unroll
+                for (int k = 0; k < QB * 4; k++)
+                    umma_bf16(d, umma_desc_sw128(s_q + (k >> 2) * 16384 + (k & 3) * 32),
+                              umma_desc_sw128(kt + (k >> 2) * 8192 + (k & 3) * 32), idesc_s, k > 0 ? 1u : 0u);
+                umma_commit(b_s_full + (j & 1) * 8);
+                umma_commit(b_k_empty + (j & 1) * 8);
+            };
+            ok = mbar_wait(b_k_full, 0, a.status);
+            if (ok) {
+                tc_fence_after();
+                issue_s(0);
+            }
+            for (int j = 0; j < n_iter && ok; j++) {
+                if (j + 1 < n_iter) {
+                    if (!(ok = mbar_wait(b_k_full + ((j + 1) & 1) * 8, (uint32_t)((j + 1) >> 1) & 1u, a.status))) break;
+                    tc_fence_after();
+                    issue_s(j + 1);
+                }
+                if (!(ok = mbar_wait(b_p_ready, (uint32_t)j & 1u, a.status))) break;
+                if (!(ok = mbar_wait(b_v_full, (uint32_t)j & 1u, a.status))) break;
+                tc_fence_after();
+#pragma unroll
+                for (int k = 0; k < 4; k++)
+                    umma_bf16_ts(t_o, t_s + (uint32_t)(j & 1) * 64 + k * 8, lt_desc_mn(s_v + k * 2048, 8192), idesc_o,
+                                 (j > 0 || k > 0) ? 1u : 0u);
+                umma_commit(b_pv_done);
+                umma_commit(b_v_empty);
+            }
+        }
+    } else if (n_iter > 0) {
+        // ------------------------------------------------------------ softmax: thread = token = TMEM lane
+        const int r = warp * 32 + lane;
+        const bool row_ok = r < nrows;
+        const int p_row = row_ok ? pos0 + tok0 + r : 0x3fffffff;
+        const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
+        float m_ref = -INFINITY, l = 0.0f;
+        bool ok = true;
+        for (int j = 0; j < n_iter && ok; j++) {
+            if (!(ok = mbar_wait(b_s_full + (j & 1) * 8, (uint32_t)(j >> 1) & 1u, a.status))) break;
+            __syncwarp();
+            ok = lt_softmax_tile<64>(t_s + lane_base + (j & 1) * 64, t_o + lane_base, n_cols, j, j * 64, p_row, a.scale_log2e,
+                                     m_ref, l, b_pv_done, b_p_ready, lane, a.status);
+        }
+        if (ok) ok = mbar_wait(b_pv_done, (uint32_t)(n_iter - 1) & 1u, a.status);
+        ok = __all_sync(0xffffffffu, ok);
+        if (ok) {
+            tc_fence_after();
+            const size_t t = (size_t)(qs0 + tok0 + (row_ok ? r : 0));
+            float inv = l > 0.0f ? 1.0f / l : 0.0f;
+            if (a.gate != nullptr) inv *= 1.0f / (1.0f + expf(-__bfloat162float(a.gate[t * a.ldg + h])));
+            bf16* dst = a.out + t * a.ldo + (size_t)h * a.dv;
+#pragma unroll 1
+            for (int c0 = 0; c0 < n_cols; c0 += 32) {
+                uint32_t ov[32];
+                tmem_ld_32x32(t_o + lane_base + c0, ov);
+                tmem_ld_wait();
+                if (!row_ok) continue;
+#pragma unroll
+                for (int c = 0; c < 32; c += 8)
+                    if (c0 + c < a.dv)
+                        *(uint4*)(dst + c0 + c) =
+                            make_uint4(pack_bf16(__uint_as_float(ov[c]) * inv, __uint_as_float(ov[c + 1]) * inv),
+                                       pack_bf16(__uint_as_float(ov[c + 2]) * inv, __uint_as_float(ov[c + 3]) * inv),
+                                       pack_bf16(__uint_as_float(ov[c + 4]) * inv, __uint_as_float(ov[c + 5]) * inv),
+                                       pack_bf16(__uint_as_float(ov[c + 6]) * inv, __uint_as_float(ov[c + 7]) * inv));
+            }
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 5) {
+        tc_fence_after();
+        tmem_dealloc(tmem, 256);
     }
 }
 
@@ -654,6 +947,52 @@ extern "C" int kb_latent_tc(const void* q, int ldq, void* out, int ldo, int dv, 
         default: return (int)cudaErrorInvalidValue;
     }
 #undef LT_GO
+}
+
+extern "C" int kb_latent_gather(const void* pool, int hd, int kr, int rot, const int* slot, const int* kv_len, int B,
+                                const int* table, int table_stride, int n_pages, void* lat, void* rotk, int N, int* status,
+                                cudaStream_t st) {
+    if (N <= 0) return 0;
+    if (hd % 8 || kr % 8 || rot % 8 || kr + rot > hd || B < 1) return (int)cudaErrorInvalidValue;
+    kb_launch(k_latent_gather, (N + 7) / 8, 256, 0, st, (const bf16*)pool, hd, kr, rot, slot, kv_len, B, table, table_stride,
+              n_pages, (bf16*)lat, (bf16*)rotk, N, status);
+    KB_LAUNCH_RET();
+}
+
+template <int KBX, int VBX>
+static int launch_latent_full(const CUtensorMap& kv, const CUtensorMap& rot, const LfArgs& a, int grid_x, int B, cudaStream_t st) {
+    using L = LfSmem<KBX, VBX>;
+    static char once_tag;
+    if (kb_first_use(&once_tag)) {
+        cudaError_t e = cudaFuncSetAttribute(k_latent_full<KBX, VBX>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+        if (e != cudaSuccess) return (int)e;
+    }
+    return (int)kb_launch(k_latent_full<KBX, VBX>, dim3(a.n_heads, grid_x, B), LT_THREADS, L::TOTAL, st, kv, rot, a);
+}
+
+// q rows of nh heads [d | rot]; kv rows [N][nh d keys | nh dv values] and rotk rows [N][rot] of the step's sequences one after
+// another (kv_len[b] rows each); angles [T][rot / 2] (cosine, sine); gate: rows of one number a head, or null. d, rot, dv
+// multiples of 8 (half pairing: rot of 16), d and dv at most 128, rot at most 64; grid_x = ceil(longest q_len / 128)
+extern "C" int kb_latent_full(const void* q, int ldq, int d, int rot, int dv, int nh, const void* kv, int ldkv, const void* rotk,
+                              int N, const float* angles, float mult, int half, const void* gate, int ldg, void* out, int ldo,
+                              const int* q_start, const int* kv_len, int B, float scale, int grid_x, int* status,
+                              cudaStream_t st) {
+    if (B <= 0 || grid_x <= 0) return 0;
+    if (d < 8 || d % 8 || d > 128 || dv < 8 || dv % 8 || dv > 128 || rot < 8 || rot % 8 || rot > 64 || (half && rot % 16) ||
+        ldq % 8 || ldkv % 8 || ldo % 8 || (((uintptr_t)q | (uintptr_t)out) & 15) || N < 1 || grid_x > 65535 || B > 65535 ||
+        !(scale > 0.0f) || ((uintptr_t)angles & 7))
+        return (int)cudaErrorInvalidValue;
+    CUtensorMap kvm, rm;
+    int rc = kb_make_map_bf16(&kvm, kv, N, (uint64_t)nh * (d + dv), ldkv, 64);
+    if (!rc) rc = kb_make_map_bf16(&rm, rotk, N, rot, rot, 64);
+    if (rc) return rc;
+    LfArgs a;
+    a.q = (const bf16*)q; a.ldq = ldq; a.d = d; a.rot = rot; a.dv = dv; a.n_heads = nh;
+    a.angles = (const float2*)angles; a.mult = mult; a.half = half; a.gate = (const bf16*)gate; a.ldg = ldg;
+    a.out = (bf16*)out; a.ldo = ldo; a.q_start = q_start; a.kv_len = kv_len; a.scale_log2e = scale * 1.4426950408889634f;
+    a.status = status;
+    if (d <= 64) return dv <= 64 ? launch_latent_full<1, 1>(kvm, rm, a, grid_x, B, st) : launch_latent_full<1, 2>(kvm, rm, a, grid_x, B, st);
+    return dv <= 64 ? launch_latent_full<2, 1>(kvm, rm, a, grid_x, B, st) : launch_latent_full<2, 2>(kvm, rm, a, grid_x, B, st);
 }
 
 template <int HD, int MT, int STAGES>

@@ -167,13 +167,13 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_prep(const TIN* KB_STEP_D
     kb_pdl_wait();
     if (p < 0) {                                       // a padding row of a recorded step: a defined query latent, no store
         if (is_q)
-            for (int i = threadIdx.x; i < q_rank; i += LP_THREADS) cqr[i] = kb_from_f<T>(0.0f);
+            for (int i = threadIdx.x; i < q_rank; i += blockDim.x) cqr[i] = kb_from_f<T>(0.0f);
         return;
     }
     const TIN* src = in + (size_t)t * ld_in + (is_q ? 0 : q_rank);
     const int n = is_q ? q_rank : kv_rank, n_all = is_q ? n : n + rot;
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < n_all; i += LP_THREADS) {
+    for (int i = threadIdx.x; i < n_all; i += blockDim.x) {
         const float v = mx_rd8<TIN>(src, n_planes, plane_stride, i);
         sv[i] = v;
         if (i < n) ss = fmaf(v, v, ss);
@@ -181,7 +181,7 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_prep(const TIN* KB_STEP_D
     const float tot = mx_block_sum(ss, red);           // (its barriers also cover sv)
     const float scale = 1.0f / sqrtf(tot / (float)n + eps);
     if (is_q) {
-        for (int i = threadIdx.x; i < n; i += LP_THREADS)
+        for (int i = threadIdx.x; i < n; i += blockDim.x)
             cqr[i] = kb_from_f<T>(__fmul_rn(__fmul_rn(scale, sv[i]), kb_to_f<TW>(wq[i])));
         return;
     }
@@ -193,12 +193,12 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_prep(const TIN* KB_STEP_D
     }
     T* kd = (T*)cv.pool + kb_kv_offset(cv, page, 0, 0, p % KB_PAGE);
     T* vd = (T*)cv.pool + kb_kv_offset(cv, page, 1, 0, p % KB_PAGE);
-    for (int i = threadIdx.x; i < n; i += LP_THREADS) {
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
         const T c = kb_from_f<T>(__fmul_rn(__fmul_rn(scale, sv[i]), kb_to_f<TW>(wkv[i])));
         kd[i] = c;
         if (!cv.one_plane) vd[i] = c;
     }
-    for (int i = threadIdx.x; i < rot / 2; i += LP_THREADS) {
+    for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
         float c, sn;
         int ia, ib;
         mx_angle<sizeof(T) == 4>(rr, p, i, c, sn);
@@ -207,9 +207,9 @@ __global__ void __launch_bounds__(LP_THREADS) k_latent_prep(const TIN* KB_STEP_D
         kd[n + ia] = kb_from_f<T>(__fsub_rn(__fmul_rn(x, c), __fmul_rn(y, sn)));
         kd[n + ib] = kb_from_f<T>(__fadd_rn(__fmul_rn(y, c), __fmul_rn(x, sn)));
     }
-    for (int i = n_all + threadIdx.x; i < cv.head_dim; i += LP_THREADS) kd[i] = kb_from_f<T>(0.0f);
+    for (int i = n_all + threadIdx.x; i < cv.head_dim; i += blockDim.x) kd[i] = kb_from_f<T>(0.0f);
     if (cv.one_plane) return;
-    for (int i = n + threadIdx.x; i < cv.head_dim; i += LP_THREADS) vd[i] = kb_from_f<T>(0.0f);
+    for (int i = n + threadIdx.x; i < cv.head_dim; i += blockDim.x) vd[i] = kb_from_f<T>(0.0f);
 }
 
 extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long long plane_stride, int ld_in, int q_rank,
@@ -224,7 +224,7 @@ extern "C" int kb_latent_prep(const void* in, int in_dtype, int n_planes, long l
     const size_t sm = (size_t)(q_rank > kv_rank + rot ? q_rank : kv_rank + rot) * sizeof(float);
     if (sm > 46 * 1024) return (int)cudaErrorInvalidValue;
 #define KB_LP(TIN, TW, T_)                                                                                       \
-    kb_launch(k_latent_prep<TIN, TW, T_>, dim3(T, 2), LP_THREADS, sm, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in,  \
+    kb_launch(k_latent_prep<TIN, TW, T_>, dim3(T, 2), T >= 256 ? 128 : LP_THREADS, sm, st, (const TIN*)in, n_planes, (size_t)plane_stride, ld_in,  \
               q_rank, kv_rank, rot, (const TW*)wq, (const TW*)wkv, eps, rr, pos, seq, slot, (T_*)cq, ldcq, \
               cv, status)
     if (in_dtype == KB_F32 && dtype == KB_F32 && wdtype == KB_F32) KB_LP(float, float, float);

@@ -74,6 +74,12 @@ def attention(ctx, q, out, nh, nkv, hd, scale, window, pool, table, n_pages, kee
     return rows_gate is not None
 
 
+def latent_full_pays(ctx, *shape) -> bool:
+    """see ``fast.latent_full_pays``"""
+    from . import fast
+    return fast.latent_full_pays(ctx, *shape)
+
+
 def latent_attention(ctx, q, out, nh: int, hd: int, v_dim: int, scale: float, pool, table, n_pages) -> None:
     """``out`` ``[T, nh v_dim]`` = causal attention of the query rows ``q`` ``[T, nh hd]`` over their sequences' cached vectors
     (``pool`` ``[pages, 1, 1, 64, hd]``, this step's included): one per position, the key of every head, whose first ``v_dim``

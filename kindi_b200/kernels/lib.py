@@ -72,6 +72,10 @@ _SIGS = {
                      c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "kb_latent_decode": [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                          c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+    "kb_latent_gather": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                         c_int, c_void_p, c_void_p],
+    "kb_latent_full": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_float, c_int,
+                       c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p],
     "kb_latent_qrope": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int,
                         c_int, c_int, c_int, c_void_p, c_void_p, c_int],
     "kb_head_gemm": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
@@ -839,6 +843,38 @@ def latent_attn_tc(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B:
     _check(load().kb_latent_tc(_p(q), q.stride(0), _p(out), out.stride(0), v_dim, _p(slot), _p(q_start), _p(kv_len), B, nh, group,
                                hd, float(scale), _p(pool), _p(table), table.stride(0), n_pages, -(-max_q // (128 // group)),
                                _p(status), _stream()), "latent_tc")
+
+
+def latent_gather(pool: torch.Tensor, kr: int, rot: int, slot, kv_len, B: int, table: torch.Tensor, n_pages: int,
+                  lat: torch.Tensor, rotk: torch.Tensor, status: torch.Tensor) -> None:
+    """the cached latents ``lat`` [N, kr] and rotated parts ``rotk`` [N, rot] of ``B`` sequences, one after another (``kv_len``
+    rows each, N their sum), from a pool of one plane (bf16; kr and rot multiples of 8)"""
+    _need_cuda(pool, table, lat, rotk)
+    N, hd = lat.shape[0], pool.shape[-1]
+    assert pool.dtype == lat.dtype == rotk.dtype == torch.bfloat16 and pool.is_contiguous() and pool.shape[1:] == (1, 1, PAGE, hd)
+    assert lat.shape == (N, kr) and rotk.shape == (N, rot) and lat.is_contiguous() and rotk.is_contiguous()
+    _check(load().kb_latent_gather(_p(pool), hd, kr, rot, _p(slot), _p(kv_len), B, _p(table), table.stride(0), n_pages, _p(lat),
+                                   _p(rotk), N, _p(status), _stream()), "latent_gather")
+
+
+def latent_attn_full(q: torch.Tensor, nh: int, d: int, rot: int, dv: int, kv: torch.Tensor, rotk: torch.Tensor,
+                     angles: torch.Tensor, mult: float, pairing: str, gate: Optional[torch.Tensor], out: torch.Tensor, q_start,
+                     kv_len, B: int, scale: float, *, max_q: int, status: torch.Tensor) -> None:
+    """tcgen05 attention of prompt-sized steps over expanded keys and values: ``kv`` rows [N, nh d | nh dv] and ``rotk`` [N, rot] of
+    the step's sequences one after another (the rotated part every head shares), queries ``q`` [T, nh (d + rot)] not yet
+    rotated (``angles``: what ``rope_table`` made for the step's rows; cosines and sines times ``mult``), out [T, nh dv].
+    ``gate`` (bf16 rows, one number a head): out *= sigmoid(gate). Sizes multiples of 8, d and dv up to 128, rot up to 64"""
+    _need_cuda(q, kv, rotk, angles, gate, out)
+    T, N = q.shape[0], kv.shape[0]
+    assert q.dtype == kv.dtype == rotk.dtype == out.dtype == torch.bfloat16
+    assert q.shape == (T, nh * (d + rot)) and kv.shape == (N, nh * (d + dv)) and rotk.shape == (N, rot) and out.shape == (T, nh * dv)
+    assert q.stride(1) == kv.stride(1) == out.stride(1) == 1 and rotk.is_contiguous()
+    assert angles.dtype == torch.float32 and angles.shape == (T, rot // 2, 2) and angles.is_contiguous()
+    assert gate is None or (gate.dtype == torch.bfloat16 and gate.shape == (T, nh) and gate.stride(1) == 1)
+    _check(load().kb_latent_full(_p(q), q.stride(0), d, rot, dv, nh, _p(kv), kv.stride(0), _p(rotk), N, _p(angles), float(mult),
+                                 PAIRING[pairing], _p(gate), gate.stride(0) if gate is not None else 0, _p(out), out.stride(0),
+                                 _p(q_start), _p(kv_len), B, float(scale), -(-max_q // 128), _p(status), _stream()),
+           "latent_full")
 
 
 def latent_attn_decode(q: torch.Tensor, out: torch.Tensor, slot, q_start, kv_len, B: int, nh: int, hd: int, v_dim: int,

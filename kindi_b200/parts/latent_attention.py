@@ -20,6 +20,9 @@ in its epilogue). Prompts, single tokens and cut prompts
 are the same code, and nothing is expanded per cached position. The rotation is the mixer's position part (its
 frequencies, pairing and factor on cosines and sines: see ``parts/rope.py``), applied by the latent kernels.
 
+Long prompts of the serving path may take the other form: keys and values of all heads expanded from the latents of the
+step's sequences by one product, fewer multiplications per query and key (``fast.latent_full_pays``). The cache is the same.
+
 Parameters: ``n_heads``, ``head_dim`` (plain), ``rot_dim``, ``v_head_dim``, ``q_rank``, ``kv_rank``, ``scale``, ``eps``,
 ``position`` (a rotation of ``rot_dim`` dimensions, either pairing), ``names`` (tensor suffixes: ``dq``, ``dq_norm``, ``uq``, ``dkv``,
 ``dkv_norm``, ``uk``, ``uv``, ``o``, and ``gate`` or None), ``head_gate`` (the gate has a row per head).
@@ -112,6 +115,31 @@ class LatentAttention(Mixer):
         w_uv = weights(n["uv"]).view(self.H, self.dv, self.kr)
         self.w_uv = torch.nn.functional.pad(w_uv, (0, self.vd - self.kr)).contiguous()
         self.w_o = weights(n["o"])
+        # every head's plain keys, then every head's values: what the expanded form multiplies the latents with
+        same = weights(n["uk"]).dtype == weights(n["uv"]).dtype == torch.bfloat16
+        self.w_kv = torch.cat([weights(n["uk"]), weights(n["uv"])], dim=0).contiguous() if same and dtype == torch.bfloat16 else None
+
+    def _full(self, ctx: StepContext, q: torch.Tensor, gate, pool, table, n_pages) -> torch.Tensor:
+        """the heads' outputs ``[T, H v_dim]`` over expanded keys and values, a gate per head applied"""
+        H, d, r, dv, kr, pos = self.H, self.d, self.r, self.dv, self.kr, self.position
+        N = sum(ctx.h_kv_len)
+        lat, rotk = (torch.empty((N, n), dtype=self.dtype, device=q.device) for n in (kr, r))
+        K.latent_gather(pool, kr, r, ctx.slot, ctx.kv_len, ctx.B, table, n_pages, lat, rotk, ctx.status)
+        kv = L.linear(ctx, lat, self.w_kv, self.dtype)
+        key = ("angles of", pos.angles_key or id(pos))
+        angles = ctx.scratch.get(key)
+        if angles is None:
+            angles = ctx.scratch[key] = K.rope_table(ctx.pos, pos.inv_freq, r)
+        o = torch.empty((ctx.T, H * dv), dtype=self.dtype, device=q.device)
+        in_kernel = gate is not None and self.gate_rows == H and gate.dim() == 2
+        K.latent_attn_full(q, H, d, r, dv, kv, rotk, angles, pos.mult, pos.pairing, gate if in_kernel else None, o, ctx.q_start,
+                           ctx.kv_len, ctx.B, self.scale, max_q=ctx.max_q, status=ctx.status)
+        if gate is not None and not in_kernel:
+            if self.gate_rows == H:
+                K.head_gate_mul(o, gate, o, dv)
+            else:
+                K.gate_mul(o, gate, o)
+        return o
 
     def forward(self, ctx: StepContext, y: torch.Tensor) -> Branch:
         H, d, r, dv, qr, kr, D = self.H, self.d, self.r, self.dv, self.qr, self.kr, self.D
@@ -123,6 +151,10 @@ class LatentAttention(Mixer):
         K.latent_prep(a, qr, kr, r, self.g_q, self.g_kv, self.eps, pos.inv_freq, pos.mult, ctx.pos, ctx.seq, ctx.slot,
                       cq, D, pool, table, n_pages, ctx.status, **turn)
         q = L.linear(ctx, cq, self.w_uq, self.dtype)
+        at = qr + kr + r
+        gate = a[..., at:at + self.gate_rows] if self.gate_rows else None
+        if ctx.fast and self.w_kv is not None and A.latent_full_pays(ctx, H, d, r, dv, kr, D, self.vd, pos.pairing):
+            return Branch(L.planes(ctx, self._full(ctx, q, gate, pool, table, n_pages), self.w_o))
         qf = torch.empty((ctx.T, H * D), dtype=self.dtype, device=y.device)
         if K.head_gemm_on_tensor_cores(q, d + r, self.w_uk_t):
             K.head_gemm(q, d + r, self.w_uk_t, qf, D, side=(q, d, r, kr, D, pos.inv_freq, pos.mult, pos.pairing, ctx.pos))
@@ -132,8 +164,7 @@ class LatentAttention(Mixer):
         att = torch.empty((ctx.T, H * self.vd), dtype=self.dtype, device=y.device)
         A.latent_attention(ctx, qf, att, H, D, self.vd, self.scale, pool, table, n_pages)
         o = torch.empty((ctx.T, H * dv), dtype=self.dtype, device=y.device)
-        at = qr + kr + r
-        K.head_gemm(att, self.vd, self.w_uv, o, dv, gate=a[..., at:at + self.gate_rows] if self.gate_rows else None)
+        K.head_gemm(att, self.vd, self.w_uv, o, dv, gate=gate)
         return Branch(L.planes(ctx, o, self.w_o))
 
     def bytes_read(self) -> int:

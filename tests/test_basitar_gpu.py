@@ -304,6 +304,70 @@ def test_attention_over_latents(K, nh, hd, v_dim, step, dtype):
             assert _rel(out, want) < 1e-2, splits
 
 
+@pytest.mark.parametrize("pairing", ["half", "interleaved"])
+@pytest.mark.parametrize("nh,d,rot,dv,gated", [(3, 64, 32, 64, True), (5, 128, 64, 128, False), (2, 48, 16, 72, True), (4, 8, 16, 8, False),
+                                               (1, 120, 48, 40, True), (6, 64, 16, 128, False)])
+@pytest.mark.parametrize("new", [[1, 65, 130, 333], [1, 3, 70, 200]])
+def test_attention_over_expanded_keys(K, nh, d, rot, dv, gated, new, pairing):
+    """cached latents and rotated parts gathered from scattered pages; keys far away, at tile borders and the row's own carry the
+    largest scores; queries rotated on the way in, heads gated on the way out"""
+    from kindi_b200.parts.rope import yarn_frequencies
+    g = torch.Generator().manual_seed(nh * 1000 + d + rot)
+    lens, kr, hd = [1, 65, 130, 333], 40, 128
+    rng, bf = random.Random(d), torch.bfloat16
+    n_blocks = [-(-n // 64) for n in lens]
+    order = list(range(sum(n_blocks) + 3))
+    rng.shuffle(order)
+    table = torch.full((6, max(n_blocks) + 1), -1, dtype=torch.int32)
+    pool = torch.full((len(order), 1, 1, 64, hd), float("nan"), dtype=bf)
+    slots, at, N = [4, 0, 5, 2], 0, sum(lens)
+    cached = torch.randn(N, kr + rot, generator=g).to(bf)
+    k0 = [sum(lens[:i]) for i in range(4)]
+    for s, n in enumerate(lens):
+        for b in range(n_blocks[s]):
+            table[slots[s], b] = order[at]
+            m = min(64, n - b * 64)
+            pool[order[at], 0, 0, :m, :kr + rot] = cached[k0[s] + b * 64:k0[s] + b * 64 + m]
+            at += 1
+    lat, rotk = (torch.full((N, n), float("nan"), dtype=bf, device="cuda") for n in (kr, rot))
+    st, kv_len = _status(), _i32(lens)
+    K.latent_gather(pool.cuda(), kr, rot, _i32(slots), kv_len, 4, table.cuda(), len(order), lat, rotk, st)
+    assert torch.equal(torch.cat([lat, rotk], dim=1).cpu(), cached)
+    kv = torch.randn(N, nh * (d + dv), generator=g).to(bf)
+    rspec = {"base": 100.0, "dims": rot, "scaling": {"factor": 4.0, "original": 64, "fast": 32.0, "slow": 1.0}}
+    f, m = yarn_frequencies(100.0, rot, rspec["scaling"])
+    scale, qs, want, pos = 1.2 * (d + rot) ** -0.5, [], [], []
+    gates = torch.randn(sum(new), nh + 2, generator=g).to(bf)
+    for s, n in enumerate(lens):
+        k = kv[k0[s]:k0[s] + n, :nh * d].view(n, nh, d)
+        v = kv[k0[s]:k0[s] + n, nh * d:].view(n, nh, dv).double()
+        q = torch.randn(n, nh, d + rot, generator=g)
+        for i in range(0, n, 3):
+            for h in range(nh):
+                q[i, h, :d] = k[max(0, (i, 0, i // 64 * 64, i // 64 * 64 - 1)[h % 4]), h].float() * 1.5
+        q = q.to(bf)
+        qr = torch.cat([q[:, :, :d].double(), PB.rotate(q[:, :, d:].double(), rspec, pairing == "interleaved")], dim=2)
+        kr_ = cached[k0[s]:k0[s] + n, kr:].double()
+        o = torch.zeros(new[s], nh, dv, dtype=F64)
+        for j, i in enumerate(range(n - new[s], n)):
+            for h in range(nh):
+                sc = (k[:i + 1, h].double() @ qr[i, h, :d] + kr_[:i + 1] @ qr[i, h, d:]) * scale
+                o[j, h] = torch.softmax(sc, dim=0) @ v[:i + 1, h]
+        qs.append(q[n - new[s]:])
+        want.append(o)
+        pos += list(range(n - new[s], n))
+    q, want = torch.cat(qs).reshape(-1, nh * (d + rot)).cuda(), torch.cat(want)
+    if gated:
+        want = want * torch.sigmoid(gates[:, 1:1 + nh].double())[:, :, None]
+    q_start = [sum(new[:i]) for i in range(5)]
+    angles = K.rope_table(_i32(pos), f.float().cuda(), rot)
+    out = torch.full((len(pos), nh * dv), float("nan"), dtype=bf, device="cuda")
+    K.latent_attn_full(q, nh, d, rot, dv, kv.cuda(), rotk, angles, m, pairing, gates.cuda()[:, 1:1 + nh] if gated else None, out,
+                       _i32(q_start), kv_len, 4, scale, max_q=max(new), status=st)
+    assert int(st.item()) == 0
+    assert _rel(out, want.reshape(len(pos), -1)) < 1.2e-2, _rel(out, want.reshape(len(pos), -1))
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("M,H,N,Kd,planes", [(1, 2, 5, 7, 1), (70, 4, 20, 16, 2), (130, 8, 48, 32, 1), (9, 1, 100, 136, 2), (5, 3, 1, 8, 1)])
 def test_products_per_head_with_a_gate_per_head(K, dtype, M, H, N, Kd, planes):
@@ -516,6 +580,39 @@ def test_long_decoding_in_a_batch(tmp_path, dtype):
     assert eng.graph_replays > 150
     _nothing_held(eng)
     _compare(tiny.collect(out, steps, raw["vocab"]), reqs, want, TOL[dtype], "long %s" % dtype)
+
+
+def test_long_prompts_in_both_forms_of_latent_attention(tmp_path, monkeypatch):
+    """a long prompt whole, in long portions and beside another: once with the keys expanded wherever the kernel takes the shape,
+    once never; the expanded form does run"""
+    from kindi_b200.kernels import fast
+    from kindi_b200.kernels import lib
+    raw = TB.TINY["B"][0]
+    folder = TB.make_model(tmp_path, "B", "bfloat16")
+    rng = random.Random(5)
+    reqs = {"a": TB.needle_request(raw["vocab"], 620, 2, list(range(60, 620, 7)), rng),
+            "b": TB.needle_request(raw["vocab"], 410, 300, list(range(301, 410, 3)), rng)}
+    want = _plain(folder, reqs)
+    whole = tiny.trace_whole(reqs)
+    cut = [(0, 0), (300, 100), (330, 101), (620, 410)]
+    steps = [{"step": len(whole) + i, "entries": [{"id": r, "tokens": reqs[r][u[k]:v[k]], "want": list(range(v[k] - u[k]))}
+                                                  for k, r in enumerate("ab")], "end": ["a", "b"] if i == 2 else []}
+             for i, (u, v) in enumerate(zip(cut, cut[1:]))]
+    real, calls = fast.latent_full_pays, []
+    count = lib.latent_attn_full
+    monkeypatch.setattr(lib, "latent_attn_full", lambda *x, **kw: (calls.append(1), count(*x, **kw)))
+    for rows in (1, 10 ** 9):
+        monkeypatch.setattr(fast, "LATENT_FULL_MIN_ROWS", rows)
+        monkeypatch.setattr(fast, "latent_full_pays", lambda ctx, *s: real(ctx, *s[:5], 10 ** 6, *s[6:]) if rows == 1 else False)
+        eng = _engine(folder, whole + steps, "bfloat16", cuda_graphs=False)
+        out = str(tmp_path / ("out%d" % rows))
+        del calls[:]
+        tiny.run_replay(eng, whole, out)
+        _compare(tiny.collect(out, whole, raw["vocab"]), reqs, want, TOL["bfloat16"], "rows from %d whole" % rows)
+        tiny.run_replay(eng, steps, out)
+        _compare(tiny.collect(out, steps, raw["vocab"]), reqs, want, TOL["bfloat16"], "rows from %d portions" % rows)
+        _nothing_held(eng)
+        assert bool(calls) == (rows == 1)
 
 
 @pytest.mark.parametrize("dtype,tie", [("float32", 1e-5), ("bfloat16", 8e-2)])
