@@ -695,11 +695,23 @@ __global__ void __launch_bounds__(LD_THREADS, 2 * LdSmem<HD, MT, STAGES>::TOTAL 
     }
     // -------------------------------------------------------------------- products and softmax
     kb_pdl_wait();
-    for (int e = threadIdx.x; e < MT * 16 * (HD / 8); e += 128) {
-        const int r = e / (HD / 8), c = e % (HD / 8);
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (h0 + r < nh) v = *(const uint4*)(q + (size_t)qs0 * ldq + (size_t)(h0 + r) * HD + c * 8);
-        *(uint4*)(qs + r * L::QLD + c * 8) = v;
+    {
+        constexpr int QV = MT * 16 * (HD / 8), QN = QV / 128 < 6 ? QV / 128 : 6;         // (loads in flight a thread)
+#pragma unroll 1
+        for (int e0 = 0; e0 < QV; e0 += 128 * QN) {
+            uint4 v[QN];
+#pragma unroll
+            for (int i = 0; i < QN; i++) {
+                const int e = e0 + threadIdx.x + i * 128, r = e / (HD / 8), c = e % (HD / 8);
+                v[i] = make_uint4(0, 0, 0, 0);
+                if (e < QV && h0 + r < nh) v[i] = *(const uint4*)(q + (size_t)qs0 * ldq + (size_t)(h0 + r) * HD + c * 8);
+            }
+#pragma unroll
+            for (int i = 0; i < QN; i++) {
+                const int e = e0 + threadIdx.x + i * 128, r = e / (HD / 8), c = e % (HD / 8);
+                if (e < QV) *(uint4*)(qs + r * L::QLD + c * 8) = v[i];
+            }
+        }
     }
     asm volatile("bar.sync 1, 128;" ::: "memory");
     float o[MT][TPW][2][4];

@@ -460,6 +460,14 @@ __global__ void __launch_bounds__(128) k_head_gemm_mma(const bf16* KB_STEP_DATA 
         }
     }
     cp_async_wait_all();
+    float gh[2] = {1.0f, 1.0f};                        // a gate per head: one number for each of this thread's two rows
+    if (gate != nullptr && gph == 1) {
+#pragma unroll
+        for (int half = 0; half < 2; half++) {
+            const int m = m0 + warp * 16 + g + half * 8;
+            if (m < M) gh[half] = mx_sigmoid(mx_rd8<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, h));
+        }
+    }
     const bool pairs = N % 2 == 0 && ldc % 2 == 0 && ldch % 2 == 0 && ((uintptr_t)C & 3) == 0;
 #pragma unroll
     for (int j = 0; j < 8; j++)
@@ -467,13 +475,11 @@ __global__ void __launch_bounds__(128) k_head_gemm_mma(const bf16* KB_STEP_DATA 
         for (int half = 0; half < 2; half++) {
             const int m = m0 + warp * 16 + g + half * 8, n = n0 + j * 8 + 2 * t;
             if (m >= M || n >= N) continue;
-            float v[2] = {acc[j][2 * half], acc[j][2 * half + 1]};
-            if (gate != nullptr)
+            float v[2] = {acc[j][2 * half] * gh[half], acc[j][2 * half + 1] * gh[half]};
+            if (gate != nullptr && gph > 1)
 #pragma unroll
                 for (int i = 0; i < 2; i++)
-                    if (n + i < N)
-                        v[i] *= mx_sigmoid(mx_rd<TG>(gate + (size_t)m * ldg, n_planes, plane_stride,
-                                                     (size_t)h * gph + (gph > 1 ? n + i : 0)));
+                    if (n + i < N) v[i] *= mx_sigmoid(mx_rd8<TG>(gate + (size_t)m * ldg, n_planes, plane_stride, (size_t)h * gph + n + i));
             bf16* dst = C + (size_t)m * ldc + (size_t)h * ldch + n;
             if (pairs) *(__nv_bfloat162*)dst = __floats2bfloat162_rn(v[0], v[1]);
             else {

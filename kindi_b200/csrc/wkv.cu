@@ -585,6 +585,17 @@ __global__ void __launch_bounds__(WR_THREADS, DP <= 64 ? 2 : 1) k_wkv_out(WkvArg
         for (int i = 0; i < WR_P; i++)
             rr[i] = wr_pair(rg + (size_t)(pc * WR_P + i) * a.ld, j, d, pc * WR_P + i < r.n, vec & 1);
     }
+    // (and r as it is, with the bonuses, for the sums inside a piece further down)
+    constexpr int NP = DP / 8;
+    const int pa = warp >> 1, hf = warp & 1, t0 = pa * WR_P;
+    const int ti = lane & 15, jl = hf * (DP / 2) + (lane >> 4) * 2;
+    float2 p[NP], bonus[NP];
+#pragma unroll
+    for (int q = 0; q < NP; q++) {
+        const int j = jl + 4 * q;
+        p[q] = wr_pair(rg + (size_t)(t0 + ti) * a.ld, j, d, t0 + ti < r.n, vec & 1);
+        bonus[q] = make_float2(j < d ? __ldg(a.u + (size_t)h * d + j) : 0.0f, j + 1 < d ? __ldg(a.u + (size_t)h * d + j + 1) : 0.0f);
+    }
     cp_async_wait_all();
     __syncthreads();
 #pragma unroll
@@ -633,22 +644,17 @@ __global__ void __launch_bounds__(WR_THREADS, DP <= 64 ? 2 : 1) k_wkv_out(WkvArg
         tab[6 * DP + j] = wr_ex2(d1 + d2);
     }
     __syncthreads();
-    const int pa = warp >> 1, hf = warp & 1, t0 = pa * WR_P;
     // ---- scores inside the piece: lane = (token, half of this warp's channel pairs); the decay is carried along as a product
     {
-        constexpr int NP = DP / 8;
-        const int ti = lane & 15, t = t0 + ti, jl = hf * (DP / 2) + (lane >> 4) * 2;
+        const int t = t0 + ti;
         const bool first = lane < 16;
-        float2 p[NP];
         float own = 0.0f;
 #pragma unroll
         for (int q = 0; q < NP; q++) {
             const int j = jl + 4 * q;
-            p[q] = wr_pair(rg + (size_t)t * a.ld, j, d, t < r.n, vec & 1);
             const float2 k2 = __bfloat1622float2(*(const __nv_bfloat162*)(ks + t * S::KLD + j));
-            const float ux = j < d ? __ldg(a.u + (size_t)h * d + j) : 0.0f, uy = j + 1 < d ? __ldg(a.u + (size_t)h * d + j + 1) : 0.0f;
-            own = fmaf(p[q].x * ux, k2.x, own);
-            own = fmaf(p[q].y * uy, k2.y, own);
+            own = fmaf(p[q].x * bonus[q].x, k2.x, own);
+            own = fmaf(p[q].y * bonus[q].y, k2.y, own);
         }
         own += __shfl_xor_sync(0xffffffffu, own, 16);
         float* dst = hf ? sc2 + t * (WR_P + 2) : sc + t * WR_SLD + t0;
