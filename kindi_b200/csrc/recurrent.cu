@@ -451,12 +451,105 @@ __global__ void __launch_bounds__(128) k_head_norm_gate(const float* KB_STEP_DAT
     }
 }
 
+// The same with four neighbours a lane and G lanes a head (heads of up to 16 G elements, everything aligned): the head in
+// registers, every load in flight before the first use
+template <typename TG, typename TO, int G>
+__global__ void __launch_bounds__(128) k_head_norm_gate4(const float* KB_STEP_DATA x, int ldx, int T, int H, int n,
+        const float* __restrict__ w, float eps, const TG* KB_STEP_DATA g, int n_planes, size_t plane_stride, int ldg,
+        int og, int gate_kind, TO* __restrict__ out, int ldo, int w_head) {
+    constexpr int NI = 4;
+    kb_pdl_launch();
+    const int gl = threadIdx.x % G;
+    const long long item0 = (long long)blockIdx.x * (128 / G) + threadIdx.x / G;
+    const bool live = item0 < (long long)T * H;
+    const long long item = live ? item0 : 0;
+    const size_t t = (size_t)(item / H);
+    const int h = (int)(item % H);
+    kb_pdl_wait();
+    const float* xr = x + t * ldx + (size_t)h * n;
+    float v[NI][4], z[NI][4], gw[NI][4];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NI; i++) {
+        const int e = (gl + i * G) * 4;
+        float4 q = make_float4(0.f, 0.f, 0.f, 0.f), ww = q;
+#pragma unroll
+        for (int k = 0; k < 4; k++) z[i][k] = 0.0f;
+        if (e < n) {
+            q = *(const float4*)(xr + e);
+            ww = *(const float4*)(w + (size_t)h * w_head + e);
+            if (g != nullptr) {
+                const TG* gp = g + t * ldg + og + (size_t)h * n + e;
+                for (int s = 0; s < n_planes; s++) {
+                    if (sizeof(TG) == 4) {
+                        const float4 u = *(const float4*)(gp + (size_t)s * plane_stride);
+                        z[i][0] += u.x; z[i][1] += u.y; z[i][2] += u.z; z[i][3] += u.w;
+                    } else {
+                        const uint2 u = *(const uint2*)(gp + (size_t)s * plane_stride);
+                        const bf16* ub = (const bf16*)&u;
+#pragma unroll
+                        for (int k = 0; k < 4; k++) z[i][k] += __bfloat162float(ub[k]);
+                    }
+                }
+            }
+        }
+        v[i][0] = q.x; v[i][1] = q.y; v[i][2] = q.z; v[i][3] = q.w;
+        gw[i][0] = ww.x; gw[i][1] = ww.y; gw[i][2] = ww.z; gw[i][3] = ww.w;
+#pragma unroll
+        for (int k = 0; k < 4; k++) ss = fmaf(v[i][k], v[i][k], ss);
+    }
+#pragma unroll
+    for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float f = 1.0f / sqrtf(ss / (float)n + eps);
+    if (!live) return;
+#pragma unroll
+    for (int i = 0; i < NI; i++) {
+        const int e = (gl + i * G) * 4;
+        if (e >= n) continue;
+        float y[4];
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+            y[k] = __fmul_rn(__fmul_rn(f, v[i][k]), gw[i][k]);
+            if (g != nullptr) y[k] *= rc_gate(z[i][k], gate_kind);
+        }
+        TO* dst = out + t * ldo + (size_t)h * n + e;
+        if (sizeof(TO) == 4) *(float4*)dst = make_float4(y[0], y[1], y[2], y[3]);
+        else {
+            __nv_bfloat162 p[2] = {__floats2bfloat162_rn(y[0], y[1]), __floats2bfloat162_rn(y[2], y[3])};
+            *(uint2*)dst = *(uint2*)p;
+        }
+    }
+}
+
 extern "C" int kb_head_norm_gate(const float* x, int ldx, int T, int H, int n, const float* w, float eps,
                                  const void* g, int gdtype, int n_planes, long long plane_stride, int ldg, int og,
                                  int gate_kind, void* out, int odtype, int ldo, cudaStream_t st, int w_head) {
     // w_head: elements between two heads' gains (0: all heads share them)
     if (T <= 0 || H <= 0) return 0;
     const int grid = (int)(((long long)T * H + 3) / 4);
+    const int gel = gdtype == KB_F32 ? 4 : 2, oel = odtype == KB_F32 ? 4 : 2;
+    if (n % 4 == 0 && n <= 512 && ldx % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 && w_head % 4 == 0 &&
+        (g == nullptr || (ldg % 4 == 0 && og % 4 == 0 && plane_stride % 4 == 0 && (uintptr_t)g % (4 * gel) == 0)) &&
+        ldo % 4 == 0 && (uintptr_t)out % (4 * oel) == 0 && (long long)T * H < 0x7fffffffLL) {
+        // (16 lanes a head of up to 64 elements: one word of four a lane; else a warp)
+#define KB_HN4(TG, TO)                                                                                             \
+    do {                                                                                                           \
+        const int lanes = n <= 64 ? 16 : 32, per = 128 / lanes;                                                    \
+        const unsigned gr = (unsigned)(((long long)T * H + per - 1) / per);                                        \
+        if (lanes == 16)                                                                                           \
+            kb_launch(k_head_norm_gate4<TG, TO, 16>, gr, 128, 0, st, x, ldx, T, H, n, w, eps, (const TG*)g, n_planes, \
+                      (size_t)plane_stride, ldg, og, gate_kind, (TO*)out, ldo, w_head);                            \
+        else                                                                                                       \
+            kb_launch(k_head_norm_gate4<TG, TO, 32>, gr, 128, 0, st, x, ldx, T, H, n, w, eps, (const TG*)g, n_planes, \
+                      (size_t)plane_stride, ldg, og, gate_kind, (TO*)out, ldo, w_head);                            \
+    } while (0)
+        if (gdtype == KB_F32 && odtype == KB_F32) KB_HN4(float, float);
+        else if (gdtype == KB_F32 && odtype == KB_BF16) KB_HN4(float, bf16);
+        else if (gdtype == KB_BF16 && odtype == KB_BF16) KB_HN4(bf16, bf16);
+        else return (int)cudaErrorInvalidValue;
+#undef KB_HN4
+        KB_LAUNCH_RET();
+    }
 #define KB_HN(TG, TO)                                                                                              \
     kb_launch(k_head_norm_gate<TG, TO>, grid, 128, 0, st, x, ldx, T, H, n, w, eps, (const TG*)g, n_planes,        \
               (size_t)plane_stride, ldg, og, gate_kind, (TO*)out, ldo, w_head)

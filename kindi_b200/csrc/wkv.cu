@@ -74,8 +74,16 @@ __global__ void __launch_bounds__(256) k_token_mix(const T* KB_STEP_DATA y, int 
             d[i] = kb_to_f<T>(pv.v[i]) - x[i];
         }
     }
+#pragma unroll 5
     for (int s = 0; s < n; s++) {
-        const float* m = mu + (size_t)s * E + c;
+        float m[V];
+        if (V % 4 == 0) {
+#pragma unroll
+            for (int i = 0; i < V; i += 4) *(float4*)(m + i) = __ldg((const float4*)(mu + (size_t)s * E + c + i));
+        } else {
+#pragma unroll
+            for (int i = 0; i < V; i++) m[i] = mu[(size_t)s * E + c + i];
+        }
 #pragma unroll
         for (int i = 0; i < V; i++) o.v[i] = kb_from_f<T>(fmaf(d[i], m[i], x[i]));
         *(Pack*)(dst + (size_t)s * E) = o;
@@ -89,7 +97,8 @@ extern "C" int kb_token_mix(const void* y, int dtype, int E, const float* mu, in
     if (T <= 0 || n <= 0) return 0;
     const int el = dtype == KB_F32 ? 4 : 2;
     const int v = dtype == KB_F32 ? 4 : 8;
-    const bool vec = E % v == 0 && ldo % v == 0 && (uintptr_t)y % (v * el) == 0 && (uintptr_t)out % (v * el) == 0;
+    const bool vec = E % v == 0 && ldo % v == 0 && (uintptr_t)y % (v * el) == 0 && (uintptr_t)out % (v * el) == 0 &&
+                     (uintptr_t)mu % 16 == 0;
 #define TM_GO(TT, V)                                                                                                   \
     kb_launch(k_token_mix<TT, V>, dim3(T, (E + 256 * V - 1) / (256 * V)), 256, 0, st, \
               (const TT*)y, E, mu, n, pos, seq, slot, q_start, last, (size_t)last_stride, (TT*)out, ldo)
