@@ -20,6 +20,9 @@ from typing import Dict, IO
 from .batch import StepEntry
 
 
+MANY = 64           # live requests whose partly filled last pages the program's cache has room for beside the tokens
+
+
 def replay(engine, lines: IO[str], out_dir: str, out: IO[str] = sys.stdout) -> int:
     os.makedirs(out_dir, exist_ok=True)
     slots: Dict[str, int] = {}
@@ -64,11 +67,13 @@ def main(argv=None) -> int:
     p.add_argument("--dtype", required=True, choices=("bfloat16", "float32"))
     p.add_argument("--out", required=True, help="folder for <step>.f32 files")
     p.add_argument("--max-tokens", type=int, required=True, dest="max_tokens",
-                   help="most tokens live requests hold at any time (each rounded up to 64)")
+                   help="most tokens live requests hold at any time")
     a = p.parse_args(argv)
     from .engine import Engine
-    from ..cache.pages import pages_for
-    engine = Engine(a.model, ctx=a.max_tokens, dtype=a.dtype, max_batch=min(max(1, pages_for(a.max_tokens)), 1024))
+    from ..cache.pages import PAGE, pages_for
+    # (every live request's last page may be partly filled: a page more for each of up to MANY of them)
+    engine = Engine(a.model, ctx=a.max_tokens + MANY * PAGE, dtype=a.dtype,
+                    max_batch=min(max(MANY, pages_for(a.max_tokens)), 1024))
     replay(engine, sys.stdin, a.out)
     return 0
 

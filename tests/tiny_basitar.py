@@ -70,6 +70,7 @@ BA_D = _config(131, 72, 1e-5, (7, 0, -3), _again([
 # E: cached vectors of 304 (kept as 320) and of 576 exactly (values of 512 elements), 48 heads, heads of 64 channels
 BA_E = _config(401, 160, 1e-5, (1009, 127, 3), [
     _lat(1, 48, 16, 48, 16, 64, 256, 64), _wkv(2, 64, (8, 2, 24)), _lat(2, 4, 32, 64, 40, 96, 512, (5, 3, 40), 500000.0)])
+RANKS = {"B": 40, "C": 24, "D": 5}                    # the decay's projection (16 elsewhere): sizes that come from the tensors alone
 TINY = {"A": (BA_A, 51), "B": (BA_B, 52), "C": (BA_C, 53), "D": (BA_D, 54), "E": (BA_E, 55)}
 
 
@@ -162,7 +163,13 @@ def make_model(tmp_path, name: str, dtype: str = "bfloat16") -> str:
         return d
     os.makedirs(d, exist_ok=True)
     _, spec = model_from_config(cfg)
-    t = random_tensors(expected_tensors(spec), seed, dtype=torch.float32, inits=tensor_inits(spec))
+    shapes = expected_tensors(spec)
+    for n, s in shapes.items():
+        if n.endswith(".mix.w1") and name in RANKS:
+            shapes[n] = (RANKS[name], s[1])
+        elif n.endswith(".mix.w2") and name in RANKS:
+            shapes[n] = (s[0], RANKS[name])
+    t = random_tensors(shapes, seed, dtype=torch.float32, inits=tensor_inits(spec))
     plant(cfg, t, seed)
     tdt = {"bfloat16": torch.bfloat16, "float32": torch.float32}[dtype]
     t = {n: v.to(tdt).contiguous() for n, v in t.items()}
